@@ -41,6 +41,12 @@ constexpr int TILE = 64;                // keys per tile = cache page size
 constexpr int CHUNKS = D / 8;           // 16-byte chunks per row
 constexpr int THREADS = 128;
 constexpr float LOG2E = 1.4426950408889634f;
+// With -DKIDI_SIGMOID_WEIGHTS=1 the weight of a key is sigmoid(score + weight_bias[head]), normalised over nothing,
+// instead of its share of a softmax: no running maximum, no denominator, no rescaling of what is summed.
+#ifndef KIDI_SIGMOID_WEIGHTS
+#define KIDI_SIGMOID_WEIGHTS 0
+#endif
+constexpr bool SIGMOID = KIDI_SIGMOID_WEIGHTS != 0;
 // Shared memory of a decode block: the query rows and two key and two value tiles (or, once
 // they are consumed, the warps' partial results).
 constexpr size_t DECODE_TILES = (size_t)(16 + 4 * TILE) * PITCH * sizeof(bf16);
@@ -142,6 +148,9 @@ struct Args {
     const bf16* gate;         // [rows, ldg] or null: head h of a row is multiplied by sigmoid(gate[row, h])
     long long ldg;
     float softcap;            // > 0: a scaled score s becomes softcap * tanh(s / softcap)
+    const float* weight_bias; // [heads], sigmoid build only: a key's weight is sigmoid(score + weight_bias[h])
+    int chunk;                // > 0: only keys of the query's own run of `chunk` positions are seen
+    float out_scale;          // the result is multiplied by it
 };
 
 // How a raw dot product becomes a score in base-2 exponent units: times scale * log2(e), or, bounded,
@@ -174,10 +183,18 @@ __device__ __forceinline__ float shaped(float raw, const ScoreShape& shape) {
 // What the weighted sum of a finished (row, head) is multiplied by: 1 / (denominator, with the head's sink in
 // it), times the row's gate. `top` is the maximum that the denominator `total` is relative to, in log2 units.
 __device__ __forceinline__ float finish_factor(const Args& a, long long row, int head, float top, float total) {
+    if (SIGMOID) return a.out_scale;
     if (a.sinks) total += exp2f(a.sinks[head] * 1.4426950408889634f - top);
     float factor = total > 0.f ? 1.0f / total : 0.f;
     if (a.gate) factor *= 1.0f / (1.0f + expf(-__bfloat162float(a.gate[row * a.ldg + head])));
-    return factor;
+    return factor * a.out_scale;
+}
+
+// sigmoid(score + bias) from both in base-2 exponent units; a score of -infinity (a key that is not seen) gives 0.
+__device__ __forceinline__ float sigmoid_log2(float score, float bias) {
+    float power;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(power) : "f"(fminf(-(score + bias), 126.f)));
+    return score == -INFINITY ? 0.f : __fdividef(1.f, 1.f + power);
 }
 
 // Loads one 64 x D tile of keys (or values) for absolute key positions [tile*64, tile*64+64)
@@ -208,7 +225,14 @@ __device__ __forceinline__ void load_tile(bf16* shared, const bf16* step, long l
 template <int NT>
 __device__ __forceinline__ void softmax_and_weighted_sum(float (&s)[NT][4], float (&best)[2], float (&denom)[2],
                                                         float (&o)[D / 8][4], const bf16* v_tile, int first_key,
-                                                        int lane) {
+                                                        int lane, const float (&bias)[2]) {
+    if constexpr (SIGMOID) {
+#pragma unroll
+        for (int j = 0; j < NT; ++j)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) s[j][i] = sigmoid_log2(s[j][i], bias[i >> 1]);
+        best[0] = best[1] = 0.f;               // partial results are added as they are
+    } else {
     float top[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
@@ -250,6 +274,7 @@ __device__ __forceinline__ void softmax_and_weighted_sum(float (&s)[NT][4], floa
         o[n][1] *= keep[0];
         o[n][2] *= keep[1];
         o[n][3] *= keep[1];
+    }
     }
     // P (bf16) times V: 16 keys per k-step = two score tiles.
     const int matrix = lane >> 3, within = lane & 7;
@@ -314,7 +339,7 @@ __global__ void __launch_bounds__(THREADS) attention_prefill_kernel(Args a) {
     const int last = start + count - 1;                     // last key position that exists
     const int step_from = a.k_step ? start : 0x7fffffff;
     const int high = start + q0 + q_rows - 1;               // largest query position of the block
-    const int low = a.window > 0 ? max(0, start + q0 - a.window + 1) : 0;
+    const int low = first_visible(start + q0, a.window, a.chunk);
     const int tile_low = low / TILE, tile_high = high / TILE;
 
     for (int chunk = threadIdx.x; chunk < TILE * CHUNKS; chunk += THREADS) {
@@ -335,6 +360,9 @@ __global__ void __launch_bounds__(THREADS) attention_prefill_kernel(Args a) {
         for (int i = 0; i < 4; ++i) o[n][i] = 0.f;
     const ScoreShape shape = score_shape(a.scale, a.softcap);
     const int position0 = start + q0 + warp * 16 + g;       // query position of accumulator rows 0,1 (and +8 for 2,3)
+    const int first_seen[2] = {first_visible(position0, a.window, a.chunk), first_visible(position0 + 8, a.window, a.chunk)};
+    float bias[2] = {0.f, 0.f};
+    if (SIGMOID) bias[0] = bias[1] = a.weight_bias[head] * LOG2E;
 
     for (int tile = tile_low; tile <= tile_high; ++tile) {
         const int buffer = (tile - tile_low) & 1;
@@ -360,10 +388,10 @@ __global__ void __launch_bounds__(THREADS) attention_prefill_kernel(Args a) {
                 for (int i = 0; i < 4; ++i) {
                     const int u = tile * TILE + j * 8 + 2 * t + (i & 1);
                     const int p = position0 + (i >> 1) * 8;
-                    const bool visible = u <= p && (a.window <= 0 || u > p - a.window);
+                    const bool visible = u <= p && u >= first_seen[i >> 1];
                     if (!visible) s[j][i] = -INFINITY;
                 }
-            softmax_and_weighted_sum<8>(s, best, denom, o, v_tiles + buffer * TILE * PITCH, 0, lane);
+            softmax_and_weighted_sum<8>(s, best, denom, o, v_tiles + buffer * TILE * PITCH, 0, lane, bias);
         }
         __syncthreads();
     }
@@ -408,7 +436,7 @@ __global__ void __launch_bounds__(THREADS) attention_decode_kernel(Args a) {
     if (seq >= 0) {
         position = a.row_pos[row];
         slot = a.seq_slot[seq];
-        low = a.window > 0 ? max(0, position - a.window + 1) : 0;
+        low = first_visible(position, a.window, a.chunk);
         const int tile_low = low / TILE, tile_high = position / TILE;
         const int all = tile_high - tile_low + 1;
         const int per_split = (all + a.splits - 1) / a.splits;
@@ -438,6 +466,11 @@ __global__ void __launch_bounds__(THREADS) attention_decode_kernel(Args a) {
         load_tile(v_tiles, nullptr, 0, 0, 0x7fffffff, a.v_cache, a.cache, slot, kv_head, tile_first, position);
         copy_async_commit();
         const ScoreShape shape = score_shape(a.scale, a.softcap);
+        float bias[2] = {0.f, 0.f};
+        if (SIGMOID) {
+            if (g < group) bias[0] = a.weight_bias[head0 + g] * LOG2E;
+            if (g + 8 < group) bias[1] = a.weight_bias[head0 + g + 8] * LOG2E;
+        }
         for (int index = 0; index < tiles; ++index) {
             const int tile = tile_first + index, buffer = index & 1;
             if (index + 1 < tiles) {
@@ -462,7 +495,7 @@ __global__ void __launch_bounds__(THREADS) attention_decode_kernel(Args a) {
                         const int u = tile * TILE + first_key + j * 8 + 2 * t + (i & 1);
                         if (u > position || u < low) s[j][i] = -INFINITY;
                     }
-                softmax_and_weighted_sum<2>(s, best, denom, o, v_tiles + buffer * TILE * PITCH, first_key, lane);
+                softmax_and_weighted_sum<2>(s, best, denom, o, v_tiles + buffer * TILE * PITCH, first_key, lane, bias);
             }
             __syncthreads();
         }
@@ -697,7 +730,7 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
     if (seq >= 0) {
         position = position_ahead;
         slot = seq == guess ? slot_ahead : a.seq_slot[seq];
-        low = a.window > 0 ? max(0, position - a.window + 1) : 0;
+        low = first_visible(position, a.window, a.chunk);
         const int tile_low = low / TILE, tile_high = position / TILE;
         const int all = tile_high - tile_low + 1;
         const int per_split = (all + a.splits - 1) / a.splits;
@@ -805,6 +838,12 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
         copy_async_commit();
         const ScoreShape shape = score_shape(a.scale, a.softcap);
         unsigned q_frag[D / 16][2];                         // Q^T as B operand: (dims, head g)
+        float bias[2] = {0.f, 0.f};
+        if (SIGMOID) {
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+                if (2 * t + i < group) bias[i] = a.weight_bias[head0 + 2 * t + i] * LOG2E;
+        }
         for (int index = 0; index < tiles; ++index) {
             const int tile = tile_first + index, buffer = index & 1;
             const int k_load = 2 * index, v_load = 2 * index + 1;                 // the ring's loads of this tile
@@ -897,6 +936,11 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
                 s[1] = see0 ? shaped(s[1], shape) : -INFINITY;
                 s[2] = see1 ? shaped(s[2], shape) : -INFINITY;
                 s[3] = see1 ? shaped(s[3], shape) : -INFINITY;
+                if constexpr (SIGMOID) {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) s[i] = sigmoid_log2(s[i], bias[i & 1]);
+                    best[0] = best[1] = 0.f;                // partial results are added as they are
+                } else {
                 float top[2] = {fmaxf(s[0], s[2]), fmaxf(s[1], s[3])};
 #pragma unroll
                 for (int i = 0; i < 2; ++i) {               // over the eight lanes that share t
@@ -921,6 +965,7 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
 #pragma unroll
                 for (int n = 0; n < D / 16; ++n) {
                     o[n][0] *= keep[0]; o[n][1] *= keep[1]; o[n][2] *= keep[0]; o[n][3] *= keep[1];
+                }
                 }
                 p0 = transpose_8x8(pack_bf16(s[0], s[1]));   // keys 2t, 2t+1 of head g
                 p1 = transpose_8x8(pack_bf16(s[2], s[3]));   // keys 2t+8, 2t+9
@@ -1216,7 +1261,7 @@ KIDI_API int kidi_attention_prefill(const Args* args, int max_new, cudaStream_t 
     const Args& a = *args;
     if (a.rows <= 0 || a.seqs <= 0 || max_new <= 0) return 0;
     if (a.cache.head_dim != D || a.heads % a.kv_heads || a.heads > 65535 || a.seqs > 65535 || !aligned(a) ||
-        (a.cache.table && a.cache.page_shift != 6))
+        (a.cache.table && a.cache.page_shift != 6) || a.chunk < 0 || (SIGMOID && (!a.weight_bias || a.sinks || a.gate)))
         return KIDI_REFUSED_SIZE;
     static std::atomic<bool> configured{false};      // setting the attribute twice is harmless
     if (!configured.load(std::memory_order_acquire)) {
@@ -1236,7 +1281,8 @@ KIDI_API int kidi_attention_decode(const Args* args, cudaStream_t stream) {
     if (a.rows <= 0) return 0;
     const int group = a.kv_heads > 0 ? a.heads / a.kv_heads : 0;
     if (a.cache.head_dim != D || a.heads % a.kv_heads || group > 16 || a.kv_heads > 65535 || a.rows > 65535 ||
-        !aligned(a) || a.cache.page_shift != 6 || a.splits < 1 || a.splits > 65535 || (a.counters && a.splits > 32))
+        !aligned(a) || a.chunk < 0 || (SIGMOID && (!a.weight_bias || a.sinks || a.gate)) ||
+        a.cache.page_shift != 6 || a.splits < 1 || a.splits > 65535 || (a.counters && a.splits > 32))
         return KIDI_REFUSED_SIZE;
     if (a.fuse) {   // the rotation inside the kernel: the narrow kernel, vectors of eight elements
         if (group > 8 || !a.k_step || !a.v_step || (a.ldkv & 7) || (a.rotary_dim & 15) || a.rotary_dim > D ||
@@ -1308,7 +1354,7 @@ KIDI_API int kidi_attention_decode(const Args* args, cudaStream_t stream) {
 static __device__ __align__(256) float kidi_static_scratch[KIDI_STATIC_SCRATCH_FLOATS];
 
 // The published argument block is the kernels' own, field for field.
-static_assert(sizeof(KidiAttentionArgs) == sizeof(Args) && sizeof(KidiCacheGeometry) == sizeof(CacheGeometry) &&
+static_assert(sizeof(KidiAttentionArgs) == offsetof(Args, weight_bias) && sizeof(KidiCacheGeometry) == sizeof(CacheGeometry) &&
                   offsetof(KidiAttentionArgs, out) == offsetof(Args, out) &&
                   offsetof(KidiAttentionArgs, splits) == offsetof(Args, splits) &&
                   offsetof(KidiAttentionArgs, cache_rows) == offsetof(Args, cache_rows),
@@ -1326,8 +1372,10 @@ KIDI_API long long kidi_attention_decode_static_need(int rows, int heads, int sp
 KIDI_API int kidi_attention_decode_static(const KidiAttentionArgs* args, cudaStream_t stream) {
     constexpr int MAX_DEVICES = 64;
     static std::atomic<float*> scratch_of_device[MAX_DEVICES];      // zero-initialised
-    Args a = {};           // the public block ends before the sinks and the gate: they stay null
+    if (SIGMOID) return KIDI_REFUSED_SIZE;      // the published block has no weight bias
+    Args a = {};           // (the public block ends before the weight bias: it stays null, and there are no chunks)
     memcpy(&a, args, sizeof(KidiAttentionArgs));
+    a.out_scale = 1.f;
     if (a.rows <= 0) return 0;
     const long long need = kidi_attention_decode_static_need(a.rows, a.heads, a.splits);
     if (need < 0 || a.heads <= 0) return KIDI_REFUSED_SIZE;

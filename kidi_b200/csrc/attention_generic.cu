@@ -13,7 +13,8 @@
 //    (src/kidi/layers/qwen3.cpp:53-54, src/kidi/runtime/vulkan/attention.comp:32-101)
 //  * the causal rule is the generic causal path's: key u is visible to the query at
 //    position p when u <= p (src/kidi/model/gemma4.cpp:736-740); with a window W,
-//    when also u > p - W.
+//    when also u > p - W; with chunks of C positions, when also floor(u / C) = floor(p / C).
+//  * instead of the softmax a key's weight can be sigmoid(s + b_h), b_h a number per head, normalised over nothing.
 // Norm sums, rotation, scores, softmax and the weighted sum are 32-bit.
 #include "common.cuh"
 
@@ -270,6 +271,153 @@ KIDI_API int kidi_rope_store(const RopeStoreArgs* args, int dtype, int norm_dtyp
 }
 
 // ---------------------------------------------------------------------------
+// A norm of a row's whole query (and key) projection, before it is split into heads: all query entries of a row divided by
+// their one root mean square and multiplied by a weight of that size, the keys likewise, in place; the keys and the values
+// (as they are) also go to the cache where one is given. A block a row; a thread takes V consecutive entries at a time.
+struct WideNormArgs {
+    void* qkv;                 // [rows, ld]: q heads, k heads, v heads
+    long long ld;
+    const float* q_norm;       // [heads * head_dim]
+    const float* k_norm;       // [kv_heads * head_dim]
+    const int* row_seq;        // [rows] (-1: padding row, skipped)
+    const int* row_pos;
+    const int* seq_slot;
+    const int* seq_start;
+    const int* seq_len;
+    void* k_cache;             // storage of this schedule entry, or null (no write)
+    void* v_cache;
+    CacheGeometry cache;
+    int heads, kv_heads, head_dim, value_dim;
+    float eps;
+};
+
+constexpr int WIDE_THREADS = 256;
+
+template <typename T, int V> struct Piece;
+template <> struct Piece<float, 1> {
+    static __device__ __forceinline__ void load(const float* p, float (&v)[1]) { v[0] = *p; }
+    static __device__ __forceinline__ void store(float* p, const float (&v)[1]) { *p = v[0]; }
+    static __device__ __forceinline__ void copy(float* to, const float* from) { *to = *from; }
+};
+template <> struct Piece<bf16, 1> {
+    static __device__ __forceinline__ void load(const bf16* p, float (&v)[1]) { v[0] = to_float(*p); }
+    static __device__ __forceinline__ void store(bf16* p, const float (&v)[1]) { *p = from_float<bf16>(v[0]); }
+    static __device__ __forceinline__ void copy(bf16* to, const bf16* from) { *to = *from; }
+};
+template <> struct Piece<bf16, 8> {
+    static __device__ __forceinline__ void load(const bf16* p, float (&v)[8]) { load8(p, v); }
+    static __device__ __forceinline__ void store(bf16* p, const float (&v)[8]) {
+        uint4 packed;
+        __nv_bfloat162* out = reinterpret_cast<__nv_bfloat162*>(&packed);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) out[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+        *reinterpret_cast<uint4*>(p) = packed;
+    }
+    static __device__ __forceinline__ void copy(bf16* to, const bf16* from) {
+        *reinterpret_cast<uint4*>(to) = *reinterpret_cast<const uint4*>(from);
+    }
+};
+
+template <typename T, int V>
+__global__ void __launch_bounds__(WIDE_THREADS) wide_norm_store_kernel(WideNormArgs a) {
+    __shared__ float scratch[2][32];
+    constexpr int WARPS = WIDE_THREADS / 32;
+    constexpr int HELD = V == 8 ? 2 : 1;          // pieces of q that stay in registers between the two passes
+    const int row = blockIdx.x;
+    const int seq = a.row_seq[row];
+    if (seq < 0) return;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    T* q = (T*)a.qkv + row * a.ld;
+    const int q_width = a.heads * a.head_dim, k_width = a.kv_heads * a.head_dim, v_width = a.kv_heads * a.value_dim;
+    T* k = q + q_width;
+    const T* v = k + k_width;
+    const int position = a.row_pos[row];
+    bool keep = a.k_cache != nullptr;
+    if (keep && a.cache.ring_pages)   // a ring keeps the last ring_tokens tokens of the step only
+        keep = position >= a.seq_start[seq] + a.seq_len[seq] - (a.cache.ring_pages << a.cache.page_shift);
+    const long long offset = keep ? cache_row_offset(a.cache, a.seq_slot[seq], position, 0) : 0;
+    const long long key_stride = (long long)a.head_dim << a.cache.page_shift;      // from one head's row to the next head's
+    const long long value_stride = (long long)a.value_dim << a.cache.page_shift;
+    T* k_cached = (T*)a.k_cache + offset;
+    T* v_cached = (T*)a.v_cache + offset / a.head_dim * a.value_dim;
+
+    float held[HELD][V], held_k[V], piece[V];
+    float q_square = 0.f, k_square = 0.f;
+    int index = 0;
+    for (int c = threadIdx.x * V; c < q_width; c += WIDE_THREADS * V, ++index) {
+        Piece<T, V>::load(q + c, piece);
+#pragma unroll
+        for (int i = 0; i < V; ++i) q_square = fmaf(piece[i], piece[i], q_square);
+#pragma unroll
+        for (int slot = 0; slot < HELD; ++slot)
+            if (slot == index) {
+#pragma unroll
+                for (int i = 0; i < V; ++i) held[slot][i] = piece[i];
+            }
+    }
+    for (int c = threadIdx.x * V; c < k_width; c += WIDE_THREADS * V) {
+        Piece<T, V>::load(k + c, piece);
+        if (c < WIDE_THREADS * V) {
+#pragma unroll
+            for (int i = 0; i < V; ++i) held_k[i] = piece[i];
+        }
+#pragma unroll
+        for (int i = 0; i < V; ++i) k_square = fmaf(piece[i], piece[i], k_square);
+    }
+    if (keep)
+        for (int c = threadIdx.x * V; c < v_width; c += WIDE_THREADS * V) {
+            const int head = c / a.value_dim;
+            Piece<T, V>::copy(v_cached + head * value_stride + (c - head * a.value_dim), v + c);
+        }
+    q_square = warp_sum(q_square);
+    k_square = warp_sum(k_square);
+    if (lane == 0) { scratch[0][warp] = q_square; scratch[1][warp] = k_square; }
+    __syncthreads();
+    float q_total = 0.f, k_total = 0.f;
+#pragma unroll
+    for (int w = 0; w < WARPS; ++w) { q_total += scratch[0][w]; k_total += scratch[1][w]; }
+    const float q_inv = 1.0f / sqrtf(q_total / (float)q_width + a.eps);
+    const float k_inv = 1.0f / sqrtf(k_total / (float)k_width + a.eps);
+    index = 0;
+    for (int c = threadIdx.x * V; c < q_width; c += WIDE_THREADS * V, ++index) {
+        if (index >= HELD) Piece<T, V>::load(q + c, piece);
+#pragma unroll
+        for (int slot = 0; slot < HELD; ++slot)
+            if (slot == index) {
+#pragma unroll
+                for (int i = 0; i < V; ++i) piece[i] = held[slot][i];
+            }
+#pragma unroll
+        for (int i = 0; i < V; ++i) piece[i] = piece[i] * q_inv * a.q_norm[c + i];
+        Piece<T, V>::store(q + c, piece);
+    }
+    for (int c = threadIdx.x * V; c < k_width; c += WIDE_THREADS * V) {
+        if (c >= WIDE_THREADS * V) Piece<T, V>::load(k + c, held_k);
+#pragma unroll
+        for (int i = 0; i < V; ++i) piece[i] = held_k[i] * k_inv * a.k_norm[c + i];
+        Piece<T, V>::store(k + c, piece);
+        if (keep) {
+            const int head = c / a.head_dim;
+            Piece<T, V>::store(k_cached + head * key_stride + (c - head * a.head_dim), piece);
+        }
+    }
+}
+
+KIDI_API int kidi_wide_norm_store(const WideNormArgs* args, int rows, int dtype, cudaStream_t stream) {
+    const WideNormArgs& a = *args;
+    if (rows <= 0) return 0;
+    if (a.heads <= 0 || a.kv_heads <= 0 || a.head_dim <= 0 || a.value_dim <= 0 || !a.q_norm || !a.k_norm ||
+        (a.k_cache != nullptr) != (a.v_cache != nullptr))
+        return KIDI_REFUSED_SIZE;
+    const bool vectors = !(a.head_dim & 7) && !(a.value_dim & 7) && !(a.ld & 7) && !((uintptr_t)a.qkv & 15) &&
+                         !((uintptr_t)a.k_cache & 15) && !((uintptr_t)a.v_cache & 15);
+    if (dtype == KIDI_F32) return kidi_launch(wide_norm_store_kernel<float, 1>, rows, WIDE_THREADS, 0, stream, a);
+    if (dtype == KIDI_BF16 && vectors) return kidi_launch(wide_norm_store_kernel<bf16, 8>, rows, WIDE_THREADS, 0, stream, a);
+    if (dtype == KIDI_BF16) return kidi_launch(wide_norm_store_kernel<bf16, 1>, rows, WIDE_THREADS, 0, stream, a);
+    return KIDI_REFUSED_DTYPE;
+}
+
+// ---------------------------------------------------------------------------
 struct AttentionArgs {
     const void* q;        // [rows, ldq], head h at h*head_dim
     long long ldq;
@@ -295,6 +443,10 @@ struct AttentionArgs {
                           // every row sees, with that score as it is, unscaled, and no value)
     const void* gate;     // [rows, ldg] or null: head h of a row is multiplied by sigmoid(gate[row, h])
     long long ldg;
+    const float* weight_bias;  // [heads] or null: the weight of a key is sigmoid(score + weight_bias[h]) instead of its
+                               // share of a softmax (nothing is normalised over the keys)
+    int chunk;                 // > 0: only keys of the query's own run of `chunk` positions are seen
+    float out_scale;           // the result is multiplied by it
 };
 
 // One block of 4 warps per (row, head). Warp w takes keys lo+w, lo+w+4, ... in
@@ -317,7 +469,7 @@ __global__ void __launch_bounds__(128) attention_generic_kernel(AttentionArgs a)
         return;
     }
     const int position = a.row_pos[row];
-    const int first = a.window > 0 ? max(0, position - a.window + 1) : 0;
+    const int first = first_visible(position, a.window, a.chunk);
     const int kv_head = head / (a.heads / a.kv_heads);
     const int slot = a.seq_slot[seq];
     const int start = a.k_step ? a.seq_start[seq] : 0x7fffffff;  // keys >= start come from the step
@@ -350,6 +502,15 @@ __global__ void __launch_bounds__(128) attention_generic_kernel(AttentionArgs a)
         float score = warp_sum(dot) * a.scale;
         if (a.softcap > 0.f) score = a.softcap * tanhf(score / a.softcap);
         if (a.slopes) score += a.slopes[head] * (float)(u - position);
+        if (a.weight_bias) {             // a weight of its own for every key: nothing to rescale
+            const float weight = 1.0f / (1.0f + expf(-(score + a.weight_bias[head])));
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const int c = lane + 32 * i;
+                if (c < vd) acc[i] = fmaf(weight, to_float(value[c]), acc[i]);
+            }
+            continue;
+        }
         const float next = fmaxf(best, score);
         const float keep = expf(best - next);  // 0 on the first key (best = -inf)
         const float weight = expf(score - next);
@@ -379,6 +540,11 @@ __global__ void __launch_bounds__(128) attention_generic_kernel(AttentionArgs a)
         factor[w] = part_max[w] == -INFINITY ? 0.f : expf(part_max[w] - top);
         total += part_sum[w] * factor[w];
     }
+    if (a.weight_bias) {
+        total = 1.f;
+#pragma unroll
+        for (int w = 0; w < 4; ++w) factor[w] = 1.f;
+    }
     float gate = 1.f;
     if (a.gate) gate = 1.0f / (1.0f + expf(-to_float(((const T*)a.gate)[row * a.ldg + head])));
     for (int c = threadIdx.x; c < vd; c += 128) {
@@ -386,7 +552,8 @@ __global__ void __launch_bounds__(128) attention_generic_kernel(AttentionArgs a)
 #pragma unroll
         for (int w = 0; w < 4; ++w) value += part_acc[w][c] * factor[w];
         value /= total;
-        out[c] = from_float<T>(a.gate ? value * gate : value);
+        if (a.gate) value *= gate;
+        out[c] = from_float<T>(value * a.out_scale);
     }
 }
 
@@ -394,7 +561,7 @@ KIDI_API int kidi_attention_generic(const AttentionArgs* args, int dtype, cudaSt
     const AttentionArgs& a = *args;
     if (a.rows <= 0) return 0;
     if (a.head_dim > 256 || a.head_dim <= 0 || a.heads % a.kv_heads || a.heads > 65535 || a.value_dim < 0 ||
-        a.value_dim > 256)
+        a.value_dim > 256 || a.chunk < 0 || (a.weight_bias && a.sinks))
         return KIDI_REFUSED_SIZE;
     dim3 grid(a.rows, a.heads);
     if (dtype == KIDI_F32) return kidi_launch(attention_generic_kernel<float>, grid, 128, 0, stream, a);

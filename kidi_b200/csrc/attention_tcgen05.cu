@@ -64,6 +64,12 @@ constexpr int CONTROL_REGISTERS = 32, SOFTMAX_REGISTERS = 112;
 constexpr unsigned SPIN_LIMIT = 1u << 24;
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr float RAISE_AFTER = 8.0f;               // the reference maximum follows after a growth of 2^8
+// With -DKIDI_SIGMOID_WEIGHTS=1 the weight of a key is sigmoid(score + weight_bias[head]), normalised over nothing: P is
+// computed from a row's scores alone, O is never rescaled and the warps of a row have nothing to exchange.
+#ifndef KIDI_SIGMOID_WEIGHTS
+#define KIDI_SIGMOID_WEIGHTS 0
+#endif
+constexpr bool SIGMOID = KIDI_SIGMOID_WEIGHTS != 0;
 constexpr int TMEM_COLUMNS = 512;                 // S of head h: columns 128 h ..; O of head h: 256 + 128 h ..
 
 __device__ int kidi_attention_timeout = 0;
@@ -227,6 +233,9 @@ struct Params {
     const bf16* gate;       // [rows, ldg] or null: head h of a row is multiplied by sigmoid(gate[row, h])
     long long ldg;
     float softcap;          // > 0: a scaled score s becomes softcap * tanh(s / softcap)
+    const float* weight_bias;   // [heads], sigmoid build only: a key's weight is sigmoid(score + weight_bias[h])
+    int chunk;              // > 0: only keys of the query's own run of `chunk` positions are seen
+    float out_scale;        // the result is multiplied by it
 };
 
 // Where a block works: its sequence, query rows, heads and key tiles.
@@ -249,7 +258,7 @@ struct Place {
         slot = p.from_cache ? p.seq_slot[seq] : 0;
         q_rows = min(BM, count - q0);
         const int high = start + q0 + q_rows - 1;                          // last query position of the block
-        const int low = p.window > 0 ? max(0, start + q0 - p.window + 1) : 0;   // first key any of its queries sees
+        const int low = first_visible(start + q0, p.window, p.chunk);      // first key any of its queries sees
         tile_low = low / BN;
         tiles = high / BN - tile_low + 1;
     }
@@ -292,6 +301,74 @@ __device__ __forceinline__ float probabilities(const float (&s)[SHARE], float sc
         packed[i >> 1] = *reinterpret_cast<unsigned*>(&pair);
     }
     return sum;
+}
+
+// Bounded scores for the sigmoid: tanh(x) = x T(x^2) on |x| <= TANH_REACH, T the polynomial that interpolates
+// tanh(sqrt(y)) / sqrt(y) at the six Chebyshev nodes of [0, TANH_REACH^2] (error below 2e-8): multiply-adds instead
+// of an exponential and a division for every score while a thread's scores all lie within the reach.
+constexpr float TANH_REACH = 0.75f;
+__device__ __forceinline__ float tanh_ratio(float y) {
+    float t = fmaf(y, -0.004711522234108173f, 0.019576216423628997f);
+    t = fmaf(y, t, -0.053341115327886254f);
+    t = fmaf(y, t, 0.13325338848115112f);
+    t = fmaf(y, t, -0.3333295409840258f);
+    return fmaf(y, t, 0.9999999704657839f);
+}
+
+__device__ __forceinline__ float reciprocal_approx(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+// P = sigmoid(score + bias), rounded to bfloat16 and packed in pairs. Two weights share one reciprocal:
+// 1 / a = b / (a b) with a, b = 1 + exp(-z); z is held above -41.6 (2^-60), so that the product stays finite.
+// FORM 0: scores as they are; 1: bounded, all within the reach of the polynomial; 2: bounded, any.
+template <bool MASKED, int FORM>
+__device__ __forceinline__ void sigmoid_share(const float (&s)[SHARE], float inner, float outer, float bias_log2, int first,
+                                              int last, unsigned (&packed)[SHARE / 2]) {
+#pragma unroll
+    for (int i = 0; i < SHARE; i += 2) {
+        float z[2];
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            float x = s[i + e];
+            if (FORM == 1) {
+                x *= inner;
+                x *= tanh_ratio(x * x);
+            } else if (FORM == 2) {
+                x = tanh_near(x * inner);
+            }
+            z[e] = fmaf(outer, x, bias_log2);
+        }
+        const float a = 1.f + exp2_approx(fminf(z[0], 60.f)), b = 1.f + exp2_approx(fminf(z[1], 60.f));
+        const float both = reciprocal_approx(a * b);
+        float p0 = b * both, p1 = a * both;
+        if (MASKED) {
+            if (i < first || i > last) p0 = 0.f;
+            if (i + 1 < first || i + 1 > last) p1 = 0.f;
+        }
+        __nv_bfloat162 pair = __floats2bfloat162_rn(p0, p1);
+        packed[i >> 1] = *reinterpret_cast<unsigned*>(&pair);
+    }
+}
+
+template <bool MASKED>
+__device__ __forceinline__ void sigmoid_weights(const float (&s)[SHARE], float scale, float softcap, float bias, int first,
+                                                int last, unsigned (&packed)[SHARE / 2]) {
+    const float bias_log2 = -bias * LOG2E;
+    if (softcap <= 0.f) {
+        sigmoid_share<MASKED, 0>(s, 0.f, -scale * LOG2E, bias_log2, first, last, packed);
+        return;
+    }
+    const float inner = scale / softcap, outer = -softcap * LOG2E;
+    float most[2] = {0.f, 0.f};
+#pragma unroll
+    for (int i = 0; i < SHARE; ++i) most[i & 1] = fmaxf(most[i & 1], fabsf(s[i]));
+    if (fmaxf(most[0], most[1]) * inner <= TANH_REACH)
+        sigmoid_share<MASKED, 1>(s, inner, outer, bias_log2, first, last, packed);
+    else
+        sigmoid_share<MASKED, 2>(s, inner, outer, bias_log2, first, last, packed);
 }
 
 // Writes a thread's packed P into the swizzled K-major tile. `p_row` is the shared-memory
@@ -486,7 +563,11 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map, const 
             const unsigned tmem_s = tmem + h * 128 + lane_bits + key, tmem_o = tmem + 256 + h * 128 + lane_bits;
             unsigned char* p_tile = p_tiles + h * P_TILE;
             const unsigned p_row = smem_u32(p_tile) + r * 128;
+            // The first key this row sees, and the first that the block's last row sees.
+            const int first_seen = first_visible(position, p.window, p.chunk);
+            const int last_first_seen = first_visible(at.start + q0 + BM - 1, p.window, p.chunk);
             const float scale_log2 = p.scale * LOG2E;
+            const float weight_bias = SIGMOID ? p.weight_bias[head0 + h] : 0.f;
             float reference = -INFINITY;                            // what the exponentials are taken against
             float denom = 0.f;                                      // this thread's part of the row sum
             unsigned exchanges = 0;                                 // uses of row_shared so far
@@ -503,9 +584,8 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map, const 
                 // tile needs a mask at all is the same for the whole block.
                 const int key0 = (tile_low + j) * BN;
                 const int last = position - key0 - key;
-                const int first = p.window > 0 ? position - p.window + 1 - key0 - key : 0;
-                const bool masked =
-                    key0 + BN - 1 > at.start + q0 || (p.window > 0 && at.start + q0 + BM - p.window > key0);
+                const int first = first_seen - key0 - key;
+                const bool masked = key0 + BN - 1 > at.start + q0 || last_first_seen > key0;
                 ok = mbarrier_wait(&ctl.s_ready[h], j & 1, abort_flag);
                 if (!ok) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -515,6 +595,20 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map, const 
                 tmem_load_wait();
                 asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
                 mbarrier_arrive(&ctl.s_free[h]);
+                if constexpr (SIGMOID) {
+                    unsigned packed[SHARE / 2];
+                    if (masked) sigmoid_weights<true>(s, p.scale, p.softcap, weight_bias, first, last, packed);
+                    else sigmoid_weights<false>(s, p.scale, p.softcap, weight_bias, first, last, packed);
+                    if (j > 0) {                     // the product of the tile before has read its P
+                        ok = mbarrier_wait(&ctl.pv_done[h], (j - 1) & 1, abort_flag);
+                        if (!ok) break;
+                    }
+                    store_probabilities(packed, p_row, r, key);
+                    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+                    asm volatile("fence.proxy.async.shared::cta;" ::: "memory");   // P is read by the tensor core
+                    mbarrier_arrive(&ctl.p_ready[h]);
+                    continue;
+                }
                 if (p.softcap > 0.f) {      // bounded scores: the raw scores take the form that `scale` then restores
                     const float inner = p.scale / p.softcap, outer = p.softcap / p.scale;
 #pragma unroll
@@ -574,6 +668,8 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map, const 
             if (ok) ok = mbarrier_wait(&ctl.pv_done[h], (tiles - 1) & 1, abort_flag);
             if (ok) {
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                float inverse = p.out_scale;
+                if constexpr (!SIGMOID) {
                 // The head's products are done: its P tile holds the parts of the row sums.
                 float* parts = reinterpret_cast<float*>(p_tile) + r * GROUPS;
                 parts[group] = denom;
@@ -583,9 +679,10 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map, const 
                 for (int g = 1; g < GROUPS; ++g) total += parts[g];
                 // The reference is the same in all warps of a row; the sink's exponential is taken against it.
                 if (p.sinks) total += exp2f(p.sinks[head0 + h] * LOG2E - (reference == -INFINITY ? 0.f : reference));
-                float inverse = 1.0f / total;
+                inverse *= 1.0f / total;
                 if (p.gate && r < q_rows)
                     inverse *= 1.0f / (1.0f + expf(-__bfloat162float(p.gate[(long long)(row0 + q0 + r) * p.ldg + head0 + h])));
+                }
                 bf16* out = p.out + (long long)(row0 + q0 + r) * p.ldo + (long long)(head0 + h) * D;
 #pragma unroll 1
                 for (int c = 32 * group; c < D && ok; c += 32 * GROUPS) {
@@ -675,6 +772,9 @@ struct KidiHeadExtras {      // what a head's result passes beside the plain sof
     const void* gate;        // [rows, ldg] bfloat16: head h of a row is multiplied by sigmoid(gate[row, h])
     long long ldg;
     float softcap;           // > 0: a scaled score s becomes softcap * tanh(s / softcap)
+    const float* weight_bias;   // [heads] float32, sigmoid build only (and there needed): a number added to a head's scores
+    int chunk;               // > 0: only keys of the query's own run of `chunk` positions are seen
+    float out_scale;         // the result is multiplied by it
 };
 
 // `cache` null: every sequence starts at position 0 and its keys are rows of qkv. Else every
@@ -745,12 +845,17 @@ KIDI_API int kidi_attention_prefill_tcgen05(const void* qkv, long long ld, int r
     p.kv_heads = kv_heads;
     p.window = window;
     p.scale = scale;
+    p.out_scale = 1.f;
     if (extras) {
         p.sinks = extras->sinks;
         p.gate = (const bf16*)extras->gate;
         p.ldg = extras->ldg;
         p.softcap = extras->softcap;
+        p.weight_bias = extras->weight_bias;
+        p.chunk = extras->chunk;
+        p.out_scale = extras->out_scale;
     }
+    if (p.chunk < 0 || (SIGMOID && (!p.weight_bias || p.sinks || p.gate))) return KIDI_REFUSED_SIZE;
     const int group_size = heads / kv_heads;
     dim3 grid(kv_heads * ((group_size + HEADS - 1) / HEADS), seqs, (max_new + BM - 1) / BM);
     attention_prefill_tcgen05_kernel<<<grid, THREADS, SHARED_BYTES, stream>>>(map, k_map, v_map, p);

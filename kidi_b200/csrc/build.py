@@ -47,6 +47,7 @@ LIBRARIES: Dict[str, Tuple[str, ...]] = {
     "differential_attention": ("differential_attention.cu",),
     "routed": ("routed.cu",),
     "scalar_recurrence": ("scalar_recurrence.cu",),
+    "linear_attention": ("linear_attention.cu",),
 }
 
 _loaded: Dict[str, ctypes.CDLL] = {}

@@ -74,6 +74,15 @@ __device__ __forceinline__ long long cache_row_offset(const CacheGeometry& g, in
     return ((((long long)page * g.kv_heads + kv_head) << g.page_shift) + within) * g.head_dim;
 }
 
+// The first key a query at `position` sees: every earlier one, or those of its window (the last `window` positions,
+// itself included), or those of its chunk (runs of `chunk` positions counted from the sequence's position 0).
+// It never decreases with the position.
+__host__ __device__ __forceinline__ int first_visible(int position, int window, int chunk) {
+    int first = window > 0 ? position - window + 1 : 0;
+    if (chunk > 0) first = max(first, position - position % chunk);
+    return max(first, 0);
+}
+
 static inline int kidi_launch_status() { return (int)cudaGetLastError(); }
 
 __device__ __forceinline__ void prefetch_l2(const void* pointer) {

@@ -1,6 +1,6 @@
 // A feed-forward made of many small experts, of which each token uses a few.
 //
-//   z = W_router h (32-bit), s = score(z), a sigmoid of each logit or a softmax over all of them; the `top`
+//   z = W_router h (+ a bias per expert) (32-bit), s = score(z), a sigmoid of each logit or a softmax over all of them; the `top`
 //   experts with the largest scores are taken (ties: the lower index) with weights w = s (optionally divided
 //   by their sum plus a small number). With groups, the experts form equal runs of neighbours, a group's
 //   score is its largest, and only experts of the `keep` best groups (ties: the lower index) can be taken;
@@ -59,13 +59,14 @@ template <typename T, typename TW>
 __global__ void __launch_bounds__(512) route_kernel(const T* __restrict__ x, const TW* __restrict__ router,
                                                     int* __restrict__ chosen, float* __restrict__ weight, int hidden,
                                                     int experts, int top, int renormalise, int softmax, int groups,
-                                                    int keep, float renormalise_eps) {
+                                                    int keep, float renormalise_eps, const float* __restrict__ bias) {
     extern __shared__ float score[];       // [experts] scores, then [experts] what may still be chosen
     float* open = score + experts;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long row = blockIdx.x;
     for (int e = warp; e < experts; e += 16) {
-        const float z = warp_sum(dot1<T, TW>(router + (long long)e * hidden, x + row * hidden, hidden, lane));
+        float z = warp_sum(dot1<T, TW>(router + (long long)e * hidden, x + row * hidden, hidden, lane));
+        if (bias) z += bias[e];
         if (lane == 0) score[e] = softmax ? z : 1.0f / (1.0f + expf(-z));
     }
     __syncthreads();
@@ -146,7 +147,7 @@ __global__ void __launch_bounds__(512) route_kernel(const T* __restrict__ x, con
 
 KIDI_API int kidi_route(const void* x, int dtype, const void* router, int weight_dtype, int* chosen, float* weight,
                         int rows, int hidden, int experts, int top, int renormalise, int softmax, int groups, int keep,
-                        float renormalise_eps, cudaStream_t stream) {
+                        float renormalise_eps, const float* bias, cudaStream_t stream) {
     if (rows <= 0) return 0;
     if (experts <= 0 || experts > 1024 || top <= 0 || top > experts || top > 32) return KIDI_REFUSED_SIZE;
     if (groups < 1 || experts % groups || keep < 1 || keep > groups || groups > 2048 ||
@@ -156,7 +157,8 @@ KIDI_API int kidi_route(const void* x, int dtype, const void* router, int weight
 #define KIDI_CASE(D, T, W, TW)                                                                                        \
     if (dtype == D && weight_dtype == W)                                                                              \
         return kidi_launch(route_kernel<T, TW>, (unsigned)rows, 512, shared, stream, (const T*)x, (const TW*)router,  \
-                           chosen, weight, hidden, experts, top, renormalise, softmax, groups, keep, renormalise_eps);
+                           chosen, weight, hidden, experts, top, renormalise, softmax, groups, keep, renormalise_eps, \
+                           bias);
     KIDI_CASE(KIDI_F32, float, KIDI_F32, float)
     KIDI_CASE(KIDI_F32, float, KIDI_BF16, bf16)
     KIDI_CASE(KIDI_BF16, bf16, KIDI_BF16, bf16)

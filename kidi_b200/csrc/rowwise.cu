@@ -72,6 +72,207 @@ add_layernorm_kernel(float* __restrict__ residual, const TD* __restrict__ delta,
         out[c] = from_float<TY>((staged[c] - mean) * inv * weight[c] + (bias ? bias[c] : 0.f));
 }
 
+// ---------------------------------------------------------------- residual add + RMS norm in equal parts
+// One block per output row r; source row s = row_index ? row_index[r] : r.
+//   d = delta[s], or with delta_weight the delta's own RMS norm in `delta_groups` equal parts:
+//       d = delta[s] / sqrt(mean of its part's squares + delta_eps) * delta_weight
+//   v = residual[s] + d (delta optional); if write_residual: residual[s] = v
+//   y[r] = v / sqrt(mean of its part's squares + eps) * weight, in `groups` equal parts, or without a weight v
+//   itself (a copy of the stream in y's type); y optional.
+// The row is staged in shared memory. A part's squares are added by WARPS / groups warps (at least one), each over a
+// run of the part, and the runs' sums in order.
+struct PartsNorm {
+    float* residual;
+    const void* delta;
+    const float* delta_weight;
+    const float* weight;
+    void* y;
+    const int* row_index;
+    int hidden, groups, delta_groups, write_residual;
+    float eps, delta_eps;
+};
+
+__device__ __forceinline__ void part_factors(const float* row, float* runs, float* factors, int hidden, int groups, float eps) {
+    constexpr int WARPS = ROW_THREADS / 32;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int width = hidden / groups;
+    const int split = groups >= WARPS ? 1 : WARPS / groups;          // runs of a part
+    const int run = (width + split - 1) / split;
+    for (int item = warp; item < groups * split; item += WARPS) {
+        const int part = item / split, which = item - part * split;
+        const int begin = part * width + which * run, end = min((part + 1) * width, begin + run);
+        float square = 0.f;
+        for (int c = begin + lane; c < end; c += 32) square = fmaf(row[c], row[c], square);
+        square = warp_sum(square);
+        if (lane == 0) runs[item] = square;
+    }
+    __syncthreads();
+    for (int part = threadIdx.x; part < groups; part += ROW_THREADS) {
+        float total = 0.f;
+        for (int which = 0; which < split; ++which) total += runs[part * split + which];
+        factors[part] = 1.0f / sqrtf(total / (float)width + eps);
+    }
+    __syncthreads();
+}
+
+template <typename TD, typename TY>
+__global__ void __launch_bounds__(ROW_THREADS) add_parts_norm_kernel(PartsNorm a) {
+    extern __shared__ float staged[];            // [hidden], then the runs' sums and the parts' factors
+    const int hidden = a.hidden, most = max(max(a.groups, a.delta_groups), ROW_THREADS / 32);
+    float* runs = staged + hidden;
+    float* factors = runs + most;
+    const int r = blockIdx.x;
+    const long long s = a.row_index ? a.row_index[r] : r;
+    float* h = a.residual + s * hidden;
+    const TD* delta = a.delta ? (const TD*)a.delta + s * hidden : nullptr;
+    if (delta && a.delta_weight) {
+        for (int c = threadIdx.x; c < hidden; c += ROW_THREADS) staged[c] = to_float(delta[c]);
+        __syncthreads();
+        part_factors(staged, runs, factors, hidden, a.delta_groups, a.delta_eps);
+        const int width = hidden / a.delta_groups;
+        for (int c = threadIdx.x; c < hidden; c += ROW_THREADS)
+            staged[c] = h[c] + staged[c] * factors[c / width] * a.delta_weight[c];
+    } else {
+        for (int c = threadIdx.x; c < hidden; c += ROW_THREADS) staged[c] = h[c] + (delta ? to_float(delta[c]) : 0.f);
+    }
+    if (a.write_residual)
+        for (int c = threadIdx.x; c < hidden; c += ROW_THREADS) h[c] = staged[c];
+    if (!a.y) return;
+    TY* out = (TY*)a.y + (long long)r * hidden;
+    if (!a.weight) {
+        for (int c = threadIdx.x; c < hidden; c += ROW_THREADS) out[c] = from_float<TY>(staged[c]);
+        return;
+    }
+    __syncthreads();
+    part_factors(staged, runs, factors, hidden, a.groups, a.eps);
+    const int width = hidden / a.groups;
+    for (int c = threadIdx.x; c < hidden; c += ROW_THREADS) out[c] = from_float<TY>(staged[c] * factors[c / width] * a.weight[c]);
+}
+
+// The same for rows of exactly ROW_THREADS * 4 * CHUNKS elements whose parts are whole multiples of 128 elements: a
+// thread keeps its CHUNKS groups of four elements in registers, and a warp's 128 elements of a chunk lie in one part
+// (segment i * WARPS + warp of the row; a part's segments are added in order).
+__device__ __forceinline__ float4 row_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 row_load4(const bf16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void row_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void row_store4(bf16* p, float4 v) {
+    uint2 raw;
+    *reinterpret_cast<__nv_bfloat162*>(&raw.x) = __floats2bfloat162_rn(v.x, v.y);
+    *reinterpret_cast<__nv_bfloat162*>(&raw.y) = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = raw;
+}
+
+template <int CHUNKS>
+__device__ __forceinline__ void segment_factors(const float4 (&v)[CHUNKS], float (&factor)[CHUNKS], float* segments,
+                                                int width, float eps) {
+    constexpr int WARPS = ROW_THREADS / 32;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+#pragma unroll
+    for (int i = 0; i < CHUNKS; ++i) {
+        float square = v[i].x * v[i].x;
+        square = fmaf(v[i].y, v[i].y, square);
+        square = fmaf(v[i].z, v[i].z, square);
+        square = warp_sum(fmaf(v[i].w, v[i].w, square));
+        if (lane == 0) segments[i * WARPS + warp] = square;
+    }
+    __syncthreads();
+    const int per = width >> 7;                               // segments of a part
+    int last = -1;
+    float value = 0.f;
+#pragma unroll
+    for (int i = 0; i < CHUNKS; ++i) {
+        const int part = (i * WARPS + warp) / per;
+        if (part != last) {
+            float total = 0.f;
+            for (int k = 0; k < per; ++k) total += segments[part * per + k];
+            value = 1.0f / sqrtf(total / (float)width + eps);
+            last = part;
+        }
+        factor[i] = value;
+    }
+}
+
+template <typename TD, typename TY, int CHUNKS>
+__global__ void __launch_bounds__(ROW_THREADS) add_parts_norm_vector_kernel(PartsNorm a) {
+    constexpr int hidden = ROW_THREADS * 4 * CHUNKS;
+    __shared__ float segments[2][CHUNKS * (ROW_THREADS / 32)];
+    const int r = blockIdx.x;
+    const long long s = a.row_index ? a.row_index[r] : r;
+    float* h = a.residual + s * hidden;
+    float4 v[CHUNKS], d[CHUNKS];
+    float factor[CHUNKS];
+    if (a.delta) {
+#pragma unroll
+        for (int i = 0; i < CHUNKS; ++i) d[i] = row_load4((const TD*)a.delta + s * hidden + 4 * (threadIdx.x + ROW_THREADS * i));
+    }
+#pragma unroll
+    for (int i = 0; i < CHUNKS; ++i) v[i] = row_load4(h + 4 * (threadIdx.x + ROW_THREADS * i));
+    if (a.delta && a.delta_weight) {
+        segment_factors<CHUNKS>(d, factor, segments[0], hidden / a.delta_groups, a.delta_eps);
+#pragma unroll
+        for (int i = 0; i < CHUNKS; ++i) {
+            const float4 w = row_load4(a.delta_weight + 4 * (threadIdx.x + ROW_THREADS * i));
+            v[i].x = fmaf(d[i].x * factor[i], w.x, v[i].x);
+            v[i].y = fmaf(d[i].y * factor[i], w.y, v[i].y);
+            v[i].z = fmaf(d[i].z * factor[i], w.z, v[i].z);
+            v[i].w = fmaf(d[i].w * factor[i], w.w, v[i].w);
+        }
+    } else if (a.delta) {
+#pragma unroll
+        for (int i = 0; i < CHUNKS; ++i) {
+            v[i].x += d[i].x; v[i].y += d[i].y; v[i].z += d[i].z; v[i].w += d[i].w;
+        }
+    }
+    if (a.write_residual) {
+#pragma unroll
+        for (int i = 0; i < CHUNKS; ++i) row_store4(h + 4 * (threadIdx.x + ROW_THREADS * i), v[i]);
+    }
+    if (!a.y) return;
+    TY* out = (TY*)a.y + (long long)r * hidden;
+    if (a.weight) {
+        segment_factors<CHUNKS>(v, factor, segments[1], hidden / a.groups, a.eps);
+#pragma unroll
+        for (int i = 0; i < CHUNKS; ++i) {
+            const float4 w = row_load4(a.weight + 4 * (threadIdx.x + ROW_THREADS * i));
+            v[i].x *= factor[i] * w.x; v[i].y *= factor[i] * w.y; v[i].z *= factor[i] * w.z; v[i].w *= factor[i] * w.w;
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < CHUNKS; ++i) row_store4(out + 4 * (threadIdx.x + ROW_THREADS * i), v[i]);
+}
+
+template <typename TD, typename TY>
+int launch_parts_norm(const PartsNorm& a, int rows, cudaStream_t stream) {
+    const bool vectors = a.hidden % (ROW_THREADS * 4) == 0 && (a.hidden / a.groups) % 128 == 0 &&
+                         (a.hidden / a.delta_groups) % 128 == 0 && !((uintptr_t)a.residual & 15) && !((uintptr_t)a.delta & 15) &&
+                         !((uintptr_t)a.y & 15) && !((uintptr_t)a.weight & 15) && !((uintptr_t)a.delta_weight & 15);
+    if (vectors) {
+        switch (a.hidden / (ROW_THREADS * 4)) {
+            case 1: return kidi_launch(add_parts_norm_vector_kernel<TD, TY, 1>, rows, ROW_THREADS, 0, stream, a);
+            case 2: return kidi_launch(add_parts_norm_vector_kernel<TD, TY, 2>, rows, ROW_THREADS, 0, stream, a);
+            case 3: return kidi_launch(add_parts_norm_vector_kernel<TD, TY, 3>, rows, ROW_THREADS, 0, stream, a);
+            case 4: return kidi_launch(add_parts_norm_vector_kernel<TD, TY, 4>, rows, ROW_THREADS, 0, stream, a);
+            case 6: return kidi_launch(add_parts_norm_vector_kernel<TD, TY, 6>, rows, ROW_THREADS, 0, stream, a);
+            case 8: return kidi_launch(add_parts_norm_vector_kernel<TD, TY, 8>, rows, ROW_THREADS, 0, stream, a);
+            default: break;
+        }
+    }
+    const int most = max(max(a.groups, a.delta_groups), ROW_THREADS / 32);
+    const size_t shared = ((size_t)a.hidden + 2 * (size_t)most) * sizeof(float);
+    if (shared > 200 * 1024) return KIDI_REFUSED_SIZE;
+    auto kernel = add_parts_norm_kernel<TD, TY>;
+    if (shared > 48 * 1024) {
+        cudaError_t status = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
+        if (status != cudaSuccess) return (int)status;
+    }
+    return kidi_launch(kernel, rows, ROW_THREADS, shared, stream, a);
+}
+
 // ---------------------------------------------------------------- a gate per head; an activation; a vector on every row
 // x[r, h, :] *= sigmoid(gate[r, h]) for x [rows, heads, width] and gate logits [rows, heads] (row stride ldg);
 // the sigmoid and the product are 32-bit.
@@ -313,6 +514,26 @@ KIDI_API int kidi_add_layernorm(float* residual, const void* delta, int delta_dt
     KIDI_CASE(KIDI_BF16, bf16, KIDI_F32, float)
     KIDI_CASE(KIDI_BF16, bf16, KIDI_BF16, bf16)
 #undef KIDI_CASE
+    return KIDI_REFUSED_DTYPE;
+}
+
+KIDI_API int kidi_add_parts_norm(float* residual, const void* delta, int delta_dtype, const float* delta_weight,
+                                 int delta_groups, float delta_eps, const float* weight, int groups, float eps, void* y,
+                                 int y_dtype, const int* row_index, int rows, int hidden, int write_residual,
+                                 cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (delta_dtype == KIDI_NONE) { delta = nullptr; delta_dtype = KIDI_F32; }
+    if (y_dtype == KIDI_NONE) { y = nullptr; y_dtype = KIDI_F32; }
+    if (!delta) delta_weight = nullptr;
+    if (!delta_weight) delta_groups = 1;
+    if (!weight) groups = 1;
+    if (hidden <= 0 || groups <= 0 || delta_groups <= 0 || hidden % groups || hidden % delta_groups) return KIDI_REFUSED_SIZE;
+    const PartsNorm a = {residual, delta, delta_weight, weight, y, row_index, hidden, groups, delta_groups, write_residual,
+                         eps, delta_eps};
+    if (delta_dtype == KIDI_F32 && y_dtype == KIDI_F32) return launch_parts_norm<float, float>(a, rows, stream);
+    if (delta_dtype == KIDI_F32 && y_dtype == KIDI_BF16) return launch_parts_norm<float, bf16>(a, rows, stream);
+    if (delta_dtype == KIDI_BF16 && y_dtype == KIDI_F32) return launch_parts_norm<bf16, float>(a, rows, stream);
+    if (delta_dtype == KIDI_BF16 && y_dtype == KIDI_BF16) return launch_parts_norm<bf16, bf16>(a, rows, stream);
     return KIDI_REFUSED_DTYPE;
 }
 

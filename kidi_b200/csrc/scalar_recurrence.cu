@@ -3,7 +3,7 @@
 //     S_t = a_t S_(t-1) + b_t k_t v_t^T            S: [dim, vdim] (+ one column whose "value" is 1, if asked for)
 //     o_t = S_t^T q_t
 //
-// a_t (decay) and b_t (write strength) come computed, in 32-bit, from a gate kernel of the mixer that owns the
+// a_t (decay) and b_t (write strength; or one fixed decay a head and a write strength of 1) come computed, in 32-bit, from a gate kernel of the mixer that owns the
 // recurrence; k, q (per head, or per group of heads) and v are columns of the mixer's projections. Two mixers
 // are served, each with its gate kernel and its finishing kernel:
 //
@@ -36,6 +36,7 @@ struct ScalarRecurrenceArgs {
     const int* seq_len;    // [seqs]
     int seqs, heads, k_heads, q_heads, dim, vdim, extra, coef_width;
     float q_scale;         // q is multiplied by it
+    const float* decay;    // [heads] or null: a_t is this number for every token and b_t is 1 (`coef` is not read)
 };
 
 struct ShortConvArgs {
@@ -142,7 +143,7 @@ __global__ void __launch_bounds__(THREADS + 32) scalar_recurrence_kernel(ScalarR
                 const long long row = row0 + t0 + t;
                 raw_k[i] = Raw<T>::load((const T*)a.k + row * a.ldk + (long long)k_head * dim + d);
                 raw_q[i] = Raw<T>::load((const T*)a.q + row * a.ldq + (long long)q_head * dim + d);
-                raw_write[i] = Raw<float>::load(a.coef + (row * a.heads + head) * a.coef_width + 1);
+                raw_write[i] = a.decay ? 1.f : Raw<float>::load(a.coef + (row * a.heads + head) * a.coef_width + 1);
             }
         }
 #pragma unroll
@@ -154,7 +155,8 @@ __global__ void __launch_bounds__(THREADS + 32) scalar_recurrence_kernel(ScalarR
                 raw_v[i] = Raw<T>::load((const T*)a.v + (long long)(row0 + t0 + t) * a.ldv + (long long)head * vdim + col);
         }
         if (threadIdx.x < tokens)
-            raw_keep = Raw<float>::load(a.coef + ((long long)(row0 + t0 + threadIdx.x) * a.heads + head) * a.coef_width);
+            raw_keep = a.decay ? a.decay[head]
+                               : Raw<float>::load(a.coef + ((long long)(row0 + t0 + threadIdx.x) * a.heads + head) * a.coef_width);
     };
     auto put = [&](float* target) {
         if (!walker) return;
@@ -493,7 +495,7 @@ KIDI_API int kidi_scalar_recurrence(const ScalarRecurrenceArgs* args, int dtype,
     const ScalarRecurrenceArgs& a = *args;
     if (a.seqs <= 0) return 0;
     if (a.heads <= 0 || a.heads > 65535 || a.dim <= 0 || a.vdim <= 0 || a.extra < 0 || a.extra > 1 || a.k_heads <= 0 ||
-        a.q_heads <= 0 || a.heads % a.k_heads || a.heads % a.q_heads || a.coef_width < 2 ||
+        a.q_heads <= 0 || a.heads % a.k_heads || a.heads % a.q_heads || (!a.decay && (!a.coef || a.coef_width < 2)) ||
         (a.vdim + 15) / 16 > 65535)
         return KIDI_REFUSED_SIZE;
     if (dtype == KIDI_F32) return dispatch_recurrence<float>(a, stream);

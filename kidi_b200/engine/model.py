@@ -33,6 +33,7 @@ from ..parts import routed as _routed  # noqa: F401
 from ..parts import state_space as _state_space  # noqa: F401
 from ..parts import matrix_memory as _matrix_memory  # noqa: F401
 from ..parts import parallel_mixers as _parallel_mixers  # noqa: F401
+from ..parts import linear_attention as _linear_attention  # noqa: F401
 
 
 class CausalLM:

@@ -45,42 +45,59 @@ class FastAttentionArgs(ctypes.Structure):
                 ("counters", c_void_p), ("fuse", c_int), ("norm_is_float", c_int), ("q_norm", c_void_p),
                 ("k_norm", c_void_p), ("cos_table", c_void_p), ("sin_table", c_void_p), ("rotary_dim", c_int),
                 ("eps", c_float), ("cache_rows", c_longlong), ("sinks", c_void_p), ("gate", c_void_p),
-                ("ldg", c_longlong), ("softcap", c_float)]
+                ("ldg", c_longlong), ("softcap", c_float), ("weight_bias", c_void_p), ("chunk", c_int),
+                ("out_scale", c_float)]
+
+    def __init__(self, *values, **named):
+        named.setdefault("out_scale", 1.0)
+        super().__init__(*values, **named)
 
 
-_libraries: Dict[int, ctypes.CDLL] = {}
-_tensor_memory_libraries: Dict[int, ctypes.CDLL] = {}
+# The libraries by (head width, whether they weigh keys by a sigmoid instead of a softmax).
+_libraries: Dict[tuple, ctypes.CDLL] = {}
+_tensor_memory_libraries: Dict[tuple, ctypes.CDLL] = {}
 _sm_count: Dict[int, int] = {}
-_ring_set: Dict[int, bool] = {}      # the decode form each library was last switched to
+_ring_set: Dict[tuple, bool] = {}      # the decode form each library was last switched to
 
 
-def library(head_dim: int) -> ctypes.CDLL:
-    """The tensor-core attention kernels compiled for one head width."""
-    lib = _libraries.get(head_dim)
+def library_request(stem: str, source: str, head_dim: int, sigmoid: bool):
+    """(name, sources, definitions) of an attention library: what `load_library` and an ahead-of-time build take."""
+    defines = {"KIDI_HEAD_DIM": head_dim}
+    if sigmoid:
+        defines["KIDI_SIGMOID_WEIGHTS"] = 1
+    return f"{stem}_d{head_dim}" + ("_sigmoid" if sigmoid else ""), (source,), defines
+
+
+def library(head_dim: int, sigmoid: bool = False) -> ctypes.CDLL:
+    """The tensor-core attention kernels compiled for one head width (`sigmoid`: their form whose weights are a sigmoid
+    of each score)."""
+    key = (head_dim, bool(sigmoid))
+    lib = _libraries.get(key)
     if lib is None:
-        lib = load_library(f"attention_d{head_dim}", ("attention_bf16.cu",), {"KIDI_HEAD_DIM": head_dim})
+        lib = load_library(*library_request("attention", "attention_bf16.cu", head_dim, sigmoid))
         lib.kidi_attention_prefill.argtypes = [c_void_p, c_int, c_void_p]
         lib.kidi_attention_decode.argtypes = [c_void_p, c_void_p]
         lib.kidi_attention_prefill.restype = lib.kidi_attention_decode.restype = c_int
         lib.kidi_attention_decode_ring.argtypes = [c_int]
         lib.kidi_attention_decode_ring.restype = None
         lib.kidi_attention_decode_ring(0)
-        _ring_set[head_dim] = False
-        _libraries[head_dim] = lib
+        _ring_set[key] = False
+        _libraries[key] = lib
     return lib
 
 
-def tensor_memory_library(head_dim: int) -> ctypes.CDLL:
+def tensor_memory_library(head_dim: int, sigmoid: bool = False) -> ctypes.CDLL:
     """The tcgen05 prompt-attention kernel compiled for one head width (64 or 128)."""
-    lib = _tensor_memory_libraries.get(head_dim)
+    key = (head_dim, bool(sigmoid))
+    lib = _tensor_memory_libraries.get(key)
     if lib is None:
-        lib = load_library(f"attention_tcgen05_d{head_dim}", ("attention_tcgen05.cu",), {"KIDI_HEAD_DIM": head_dim})
+        lib = load_library(*library_request("attention_tcgen05", "attention_tcgen05.cu", head_dim, sigmoid))
         lib.kidi_attention_prefill_tcgen05.argtypes = [
             c_void_p, c_longlong, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
             c_float, c_void_p, c_void_p, c_void_p]
         lib.kidi_attention_prefill_tcgen05.restype = c_int
         lib.kidi_attention_tcgen05_timeout_flag.restype = c_int
-        _tensor_memory_libraries[head_dim] = lib
+        _tensor_memory_libraries[key] = lib
     return lib
 
 
@@ -100,8 +117,10 @@ class PromptCache(ctypes.Structure):
 
 
 class HeadExtras(ctypes.Structure):
-    """A number per head in the softmax denominator and a sigmoid gate per row and head (KidiHeadExtras)."""
-    _fields_ = [("sinks", c_void_p), ("gate", c_void_p), ("ldg", c_longlong), ("softcap", c_float)]
+    """What a layer adds to plain causal softmax attention (KidiHeadExtras): a number per head in the denominator, a
+    sigmoid gate per row and head, a bound on the scores, sigmoid weights, chunks, a factor on the result."""
+    _fields_ = [("sinks", c_void_p), ("gate", c_void_p), ("ldg", c_longlong), ("softcap", c_float),
+                ("weight_bias", c_void_p), ("chunk", c_int), ("out_scale", c_float)]
 
 
 def extras_fit(sinks: Optional[torch.Tensor], gate: Optional[torch.Tensor], heads: int) -> bool:
@@ -115,17 +134,19 @@ def prefill_tensor_memory(qkv: torch.Tensor, out: torch.Tensor, seq_len: torch.T
                           seqs: int, max_new: int, *, heads: int, kv_heads: int, head_dim: int, scale: float,
                           window: int, kv_view=None, seq_start: Optional[torch.Tensor] = None,
                           seq_slot: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None,
-                          gate: Optional[torch.Tensor] = None, q_only: bool = False, softcap: float = 0.0) -> None:
+                          gate: Optional[torch.Tensor] = None, q_only: bool = False, softcap: float = 0.0,
+                          weight_bias: Optional[torch.Tensor] = None, chunk: int = 0, out_scale: float = 1.0) -> None:
     """Causal attention of packed prompts. Without `kv_view` the prompts start at position 0
     and every key is a row of qkv; with it (a cache of 64-token pages without a ring, into
     which the step's rows have been written) every key and value is read from the cache,
     so the prompts may continue sequences of `seq_start` tokens. `sinks`, `gate`: see `run`. `q_only` (with
     `kv_view`): the rows of qkv hold the query heads only."""
-    lib = tensor_memory_library(head_dim)
+    lib = tensor_memory_library(head_dim, weight_bias is not None)
     cache = extras = None
-    if sinks is not None or gate is not None or softcap:
+    if sinks is not None or gate is not None or softcap or weight_bias is not None or chunk or out_scale != 1.0:
         extras = HeadExtras(sinks.data_ptr() if sinks is not None else 0, gate.data_ptr() if gate is not None else 0,
-                            gate.stride(0) if gate is not None else 0, float(softcap or 0.0))
+                            gate.stride(0) if gate is not None else 0, float(softcap or 0.0),
+                            weight_bias.data_ptr() if weight_bias is not None else 0, int(chunk or 0), float(out_scale))
     if kv_view is not None:
         cache = PromptCache(kv_view.keys.data_ptr(), kv_view.values.data_ptr(), kv_view.keys.numel() // head_dim,
                             kv_view.table.data_ptr(), kv_view.table.shape[1], seq_start.data_ptr(), seq_slot.data_ptr(),
@@ -244,7 +265,8 @@ def fuses_rotation(plan, qkv: torch.Tensor, *, heads: int, kv_heads: int, head_d
 def run(ctx, qkv, out, *, heads, kv_heads, head_dim, scale, window, kv_view, keys_in_step, rotation=None,
         step_rows_cached: bool = False, splits: Optional[int] = None, ring: Optional[bool] = None,
         softcap: float = 0.0, slopes: Optional[torch.Tensor] = None, value_dim: Optional[int] = None,
-        sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, q_only: bool = False) -> None:
+        sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, q_only: bool = False,
+        weight_bias: Optional[torch.Tensor] = None, chunk: Optional[int] = None, out_scale: float = 1.0) -> None:
     """`ctx` gives the step's `plan`, its device `tables` and `workspace(name, count, zero)`.
     `keys_in_step`: the step's own keys and values are read from qkv (else from the
     cache, like the earlier ones). `step_rows_cached`: they are in the cache as well (a cache
@@ -255,23 +277,26 @@ def run(ctx, qkv, out, *, heads, kv_heads, head_dim, scale, window, kv_view, key
     override the launcher's own choice of the decode kernel's form (tests of each form).
     `value_dim`, `sinks`, `gate`: value heads of another width than the keys, a number per head in the softmax
     denominator, a sigmoid gate per row and head (see `ops.attention_generic`). `q_only`: the rows of qkv hold the
-    query heads only (every key and value comes from the cache)."""
+    query heads only (every key and value comes from the cache). `weight_bias`, `chunk`, `out_scale`: sigmoid weights,
+    chunks of positions and a factor on the result (see `ops.attention_generic`)."""
     plan, tables = ctx.plan, ctx.tables
     decode = plan.is_decode and not keys_in_step
     # Scores that are shifted by position run on the general kernel (the tensor-core kernels compute scaled
     # scores, bounded by a tanh where a layer asks for it).
     reshaped = slopes is not None
     uneven = value_dim is not None and value_dim != head_dim
-    if (reshaped or uneven or not extras_fit(sinks, gate, heads)
+    sigmoid = weight_bias is not None
+    if (reshaped or uneven or (sigmoid and (sinks is not None or gate is not None)) or not extras_fit(sinks, gate, heads)
             or not fast_fits(qkv.dtype, heads, kv_heads, head_dim, decode)
             or (kv_view is not None and kv_view.page_size != 64)):
         ops.attention_generic(qkv, out, heads=heads, kv_heads=kv_heads, head_dim=head_dim, scale=scale,
                               window=window, tables=tables, kv_view=kv_view, keys_in_step=keys_in_step,
-                              softcap=softcap, slopes=slopes, value_dim=value_dim, sinks=sinks, gate=gate)
+                              softcap=softcap, slopes=slopes, value_dim=value_dim, sinks=sinks, gate=gate,
+                              weight_bias=weight_bias, chunk=chunk, out_scale=out_scale)
         return
     if not decode and tensor_memory_fits(qkv, out, head_dim, heads, kv_heads, scale):
         common = dict(heads=heads, kv_heads=kv_heads, head_dim=head_dim, scale=scale, window=window, sinks=sinks,
-                      gate=gate, softcap=softcap)
+                      gate=gate, softcap=softcap, weight_bias=weight_bias, chunk=int(chunk or 0), out_scale=out_scale)
         if keys_in_step and int(plan.seq_start.max()) == 0:      # every key is a row of this step
             prefill_tensor_memory(qkv, out, tables.seq_len, tables.seq_row0, plan.n_seqs, plan.max_new, **common)
             return
@@ -297,16 +322,20 @@ def run(ctx, qkv, out, *, heads, kv_heads, head_dim, scale, window, kv_view, key
     if gate is not None:
         args.gate, args.ldg = gate.data_ptr(), gate.stride(0)
     args.softcap = float(softcap or 0.0)
-    lib = library(head_dim)
+    if sigmoid:
+        args.weight_bias = weight_bias.data_ptr()
+    args.chunk, args.out_scale = int(chunk or 0), float(out_scale)
+    lib = library(head_dim, sigmoid)
+    form_key = (head_dim, sigmoid)
     stream = ops._stream()
     if not decode:
         _check(lib.kidi_attention_prefill(ctypes.byref(args), plan.max_new, stream), "attention_prefill[mma.sync]")
         return
     rows = qkv.shape[0]
-    splits, ring = decode_form(rows, kv_heads, head_dim, plan.max_total, window, qkv.device, splits, ring)
-    if _ring_set.get(head_dim) != ring:                # the form is a switch of the library, not of a launch
+    splits, ring = decode_form(rows, kv_heads, head_dim, plan.max_total, reach_of(window, chunk), qkv.device, splits, ring)
+    if _ring_set.get(form_key) != ring:                # the form is a switch of the library, not of a launch
         lib.kidi_attention_decode_ring(1 if ring else 0)
-        _ring_set[head_dim] = ring
+        _ring_set[form_key] = ring
     # One wave of blocks and few splits: the blocks of a (row, key/value head) form a thread-block
     # cluster and merge through distributed shared memory. Clusters that must wait for several
     # free slots of one GPC at once lose that again when the grid takes more than a wave.
@@ -342,6 +371,12 @@ def run(ctx, qkv, out, *, heads, kv_heads, head_dim, scale, window, kv_view, key
            2 if form == "combine kernel" else 1)
 
 
+def reach_of(window, chunk) -> Optional[int]:
+    """The most keys a query may see: the smaller of window and chunk (None: no bound)."""
+    bounds = [int(bound) for bound in (window, chunk) if bound]
+    return min(bounds) if bounds else None
+
+
 def decode_form(rows: int, kv_heads: int, head_dim: int, longest: int, window, device: torch.device,
                 splits: Optional[int] = None, ring: Optional[bool] = None):
     """(key splits, ring form) of decode attention for `rows` sequences of at most `longest`
@@ -360,7 +395,9 @@ class AttentionLauncher:
     form of its decode kernel itself, from the rows of the step and the longest sequence."""
 
     def __init__(self, *, heads: int, kv_heads: int, head_dim: int, scale: float, window=None,
-                 softcap: float = 0.0, slopes: Optional[torch.Tensor] = None):
+                 softcap: float = 0.0, slopes: Optional[torch.Tensor] = None, chunk: Optional[int] = None,
+                 out_scale: float = 1.0):
+        self.chunk, self.out_scale = chunk, float(out_scale)
         self.geometry = dict(heads=heads, kv_heads=kv_heads, head_dim=head_dim)
         self.scale, self.window = scale, window
         # Scores bounded by softcap * tanh(s / softcap) run on every kernel; scores shifted by slopes[head] *
@@ -374,7 +411,7 @@ class AttentionLauncher:
 
     def run(self, ctx, qkv, out, **arguments) -> None:
         run(ctx, qkv, out, scale=self.scale, window=self.window, softcap=self.softcap, slopes=self.slopes,
-            **self.geometry, **arguments)
+            chunk=self.chunk, out_scale=self.out_scale, **self.geometry, **arguments)
 
     def launch_signature(self, dtype: torch.dtype, rows: int, longest: int, device: torch.device) -> tuple:
         """What a captured decode step freezes of this launcher's choices: the form of the
@@ -382,4 +419,5 @@ class AttentionLauncher:
         geometry = self.geometry
         if self.reshaped or not fast_fits(dtype, geometry["heads"], geometry["kv_heads"], geometry["head_dim"], True):
             return ()
-        return decode_form(rows, geometry["kv_heads"], geometry["head_dim"], longest, self.window, device)
+        return decode_form(rows, geometry["kv_heads"], geometry["head_dim"], longest, reach_of(self.window, self.chunk),
+                           device)

@@ -1,0 +1,92 @@
+"""Python faces of the kernels of linear attention with one fixed decay per head (csrc/linear_attention.cu), compiled
+when a model with such a layer first runs."""
+from __future__ import annotations
+
+import ctypes
+
+import torch
+
+from ..csrc.build import load_library
+from ..errors import invalid_argument
+from . import ops, scalar_recurrence
+from .ops import _check, c_float, c_int, c_longlong, c_void_p, dtype_code
+from .scalar_recurrence import MAX_DIM, _float_tensor, _rows_view
+
+
+class LinearStepArgs(ctypes.Structure):
+    _fields_ = [("q", c_void_p), ("ldq", c_longlong), ("k", c_void_p), ("ldk", c_longlong), ("v", c_void_p),
+                ("ldv", c_longlong), ("decay", c_void_p), ("state", c_void_p), ("out", c_void_p), ("row_seq", c_void_p),
+                ("seq_slot", c_void_p), ("seq_row0", c_void_p), ("seqs", c_int), ("heads", c_int), ("dim", c_int),
+                ("vdim", c_int)]
+
+
+_library = None
+
+
+def library():
+    global _library
+    if _library is None:
+        lib = load_library("linear_attention")
+        lib.kidi_linear_step.argtypes = [c_void_p, c_int, c_void_p]
+        lib.kidi_normed_gate.argtypes = [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_longlong, c_int, c_int,
+                                         c_float, c_float, c_void_p]
+        lib.kidi_silu_columns.argtypes = [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_void_p]
+        for name in ("kidi_linear_step", "kidi_normed_gate", "kidi_silu_columns"):
+            getattr(lib, name).restype = c_int
+        _library = lib
+    return _library
+
+
+def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, *,
+                     heads: int, dim: int, vdim: int, tables, seqs: int, one_token: bool) -> torch.Tensor:
+    """S_t = decay_h S_(t-1) + k_t v_t^T and o_t = S_t^T q_t for every sequence's rows of the step, from and into `state`
+    [slots + 1, heads, dim, vdim] (float32). q, k [rows, heads * dim] and v [rows, heads * vdim] are views of the step's
+    element type; decay float32 [heads]. `one_token`: every sequence of the step brings one token (decoding). Returns the
+    read-out, float32 [rows, heads * vdim]."""
+    if not one_token:
+        return scalar_recurrence.scalar_recurrence(k, q, v, None, state, heads=heads, k_heads=heads, q_heads=heads, dim=dim,
+                                                   vdim=vdim, tables=tables, seqs=seqs, decay=decay)
+    ops._need_cuda(q, k, v, decay, state)
+    rows = v.shape[0]
+    for tensor, width, what in ((k, heads * dim, "keys"), (q, heads * dim, "queries"), (v, heads * vdim, "values")):
+        _rows_view(tensor, "linear attention")
+        if tensor.shape != (rows, width) or tensor.dtype != v.dtype:
+            raise invalid_argument(f"linear attention: the {what} have the wrong shape or type")
+    _float_tensor(decay, (heads,), "the decays")
+    if state.dtype != torch.float32 or tuple(state.shape[1:]) != (heads, dim, vdim) or not state.is_contiguous():
+        raise invalid_argument("linear attention: the state is float32 [slots, heads, dim, vdim]")
+    out = torch.empty((rows, heads * vdim), dtype=torch.float32, device=v.device)
+    args = LinearStepArgs(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), decay.data_ptr(),
+                          state.data_ptr(), out.data_ptr(), tables.row_seq.data_ptr(), tables.seq_slot.data_ptr(),
+                          tables.seq_row0.data_ptr(), seqs, heads, dim, vdim)
+    _check(library().kidi_linear_step(ctypes.byref(args), dtype_code(v.dtype), ops._stream()), "linear_attention[one token]")
+    return out
+
+
+def normed_gate(read: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, eps: float, factor: float,
+                out: torch.Tensor) -> torch.Tensor:
+    """out = read / rms(read) * weight * sigmoid(gate) * factor over each row; read float32 [rows, width], gate and out
+    views of the step's element type whose rows are contiguous."""
+    ops._need_cuda(read, weight, gate, out)
+    rows, width = read.shape
+    _float_tensor(read, (rows, width), "the read-out")
+    _float_tensor(weight, (width,), "the norm weight")
+    _rows_view(gate, "normed gate")
+    _rows_view(out, "normed gate")
+    if gate.shape != (rows, width) or out.shape != (rows, width) or gate.dtype != out.dtype:
+        raise invalid_argument("normed gate: the gate or the result has the wrong shape or type")
+    _check(library().kidi_normed_gate(read.data_ptr(), weight.data_ptr(), gate.data_ptr(), gate.stride(0),
+                                      dtype_code(gate.dtype), out.data_ptr(), out.stride(0), rows, width, float(eps),
+                                      float(factor), ops._stream()), "normed_gate")
+    return out
+
+
+def silu_columns(x: torch.Tensor, begin: int, end: int) -> torch.Tensor:
+    """x[:, begin:end] <- silu of itself, in place (32-bit arithmetic)."""
+    ops._need_cuda(x)
+    _rows_view(x, "silu columns")
+    if not 0 <= begin <= end <= x.shape[1]:
+        raise invalid_argument("silu columns: the range lies outside the matrix")
+    _check(library().kidi_silu_columns(x.data_ptr(), x.stride(0), dtype_code(x.dtype), x.shape[0], int(begin),
+                                       int(end - begin), ops._stream()), "silu_columns")
+    return x

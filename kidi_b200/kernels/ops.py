@@ -158,6 +158,11 @@ def core():
                                             c_void_p]
         lib.kidi_add_layernorm.argtypes = [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                            c_int, c_int, c_float, c_int, c_void_p, c_float, c_void_p]
+        lib.kidi_add_parts_norm.argtypes = [c_void_p, c_void_p, c_int, c_void_p, c_int, c_float, c_void_p, c_int, c_float,
+                                            c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p]
+        lib.kidi_wide_norm_store.argtypes = [c_void_p, c_int, c_int, c_void_p]
+        for name in ("kidi_add_parts_norm", "kidi_wide_norm_store"):
+            getattr(lib, name).restype = c_int
         lib.kidi_head_gate.argtypes = [c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_void_p]
         lib.kidi_gelu.argtypes = [c_void_p, c_void_p, c_int, c_longlong, c_void_p]
         lib.kidi_add_vector.argtypes = [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
@@ -232,7 +237,15 @@ class AttentionArgs(ctypes.Structure):
                 ("seq_slot", c_void_p), ("seq_start", c_void_p), ("seq_row0", c_void_p), ("rows", c_int),
                 ("heads", c_int), ("kv_heads", c_int), ("head_dim", c_int), ("window", c_int), ("scale", c_float),
                 ("softcap", c_float), ("slopes", c_void_p), ("value_dim", c_int), ("sinks", c_void_p),
-                ("gate", c_void_p), ("ldg", c_longlong)]
+                ("gate", c_void_p), ("ldg", c_longlong), ("weight_bias", c_void_p), ("chunk", c_int),
+                ("out_scale", c_float)]
+
+
+class WideNormArgs(ctypes.Structure):
+    _fields_ = [("qkv", c_void_p), ("ld", c_longlong), ("q_norm", c_void_p), ("k_norm", c_void_p),
+                ("row_seq", c_void_p), ("row_pos", c_void_p), ("seq_slot", c_void_p), ("seq_start", c_void_p),
+                ("seq_len", c_void_p), ("k_cache", c_void_p), ("v_cache", c_void_p), ("cache", CacheGeometry),
+                ("heads", c_int), ("kv_heads", c_int), ("head_dim", c_int), ("value_dim", c_int), ("eps", c_float)]
 
 
 def cache_geometry(view, kv_heads: int, head_dim: int) -> CacheGeometry:
@@ -322,6 +335,34 @@ def add_layernorm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight:
         _ptr(residual), _ptr(delta), dtype_code(delta.dtype) if delta is not None else NONE, _ptr(weight), _ptr(bias),
         _ptr(out), dtype_code(out.dtype) if out is not None else NONE, _ptr(row_index), rows, hidden, float(eps),
         0 if row_index is not None else 1, _ptr(delta_weight), float(delta_eps), _stream()), "add_layernorm")
+    return out
+
+
+def add_parts_norm(residual: torch.Tensor, delta: Optional[torch.Tensor], out_dtype: Optional[torch.dtype], *,
+                   weight: Optional[torch.Tensor] = None, groups: int = 1, eps: float = 0.0,
+                   delta_weight: Optional[torch.Tensor] = None, delta_groups: int = 1, delta_eps: float = 0.0,
+                   row_index: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """residual += delta (in place, float32); with `delta_weight` the delta passes an RMS norm in `delta_groups` equal
+    parts first. Returns (in `out_dtype`; None: nothing) the new rows' RMS norm in `groups` equal parts, or without
+    `weight` a copy of the rows. With `row_index`, row r of the result comes from row row_index[r] and the residual is
+    left as it is. A part is divided by the root of its own mean square plus eps; the weights are float32 [hidden]."""
+    _need_cuda(residual, delta, weight, delta_weight, row_index)
+    if residual.dtype != torch.float32 or residual.dim() != 2 or not residual.is_contiguous():
+        raise invalid_argument("the residual stream is a contiguous float32 matrix")
+    hidden = residual.shape[1]
+    if delta is not None and (delta.shape != residual.shape or not delta.is_contiguous()):
+        raise invalid_argument("the residual delta must match the residual stream")
+    _float_vector(weight, hidden, "the norm weight")
+    _float_vector(delta_weight, hidden, "the weight of the delta's norm")
+    if row_index is not None and (row_index.dtype != torch.int32 or row_index.dim() != 1):
+        raise invalid_argument("row_index must be an int32 vector")
+    rows = row_index.shape[0] if row_index is not None else residual.shape[0]
+    out = torch.empty((rows, hidden), dtype=out_dtype, device=residual.device) if out_dtype is not None else None
+    _check(core().kidi_add_parts_norm(
+        _ptr(residual), _ptr(delta), dtype_code(delta.dtype) if delta is not None else NONE, _ptr(delta_weight),
+        int(delta_groups), float(delta_eps), _ptr(weight), int(groups), float(eps), _ptr(out),
+        dtype_code(out.dtype) if out is not None else NONE, _ptr(row_index), rows, hidden,
+        0 if row_index is not None else 1, _stream()), "add_parts_norm")
     return out
 
 
@@ -729,17 +770,43 @@ def rope_store(qkv: torch.Tensor, *, heads: int, kv_heads: int, head_dim: int, q
            "rope_store")
 
 
+def wide_norm_store(qkv: torch.Tensor, *, heads: int, kv_heads: int, head_dim: int, value_dim: int, q_norm: torch.Tensor,
+                    k_norm: torch.Tensor, eps: float, tables, kv_view, store: bool) -> None:
+    """In place on qkv (as for `rope_store`): all query entries of a row divided by their one root mean square and
+    multiplied by q_norm (float32 [heads * head_dim]), the key entries likewise with k_norm; with `store` the keys and
+    the values also go to the cache."""
+    _need_cuda(qkv, q_norm, k_norm)
+    if qkv.dim() != 2 or qkv.stride(1) != 1 or qkv.shape[1] < (heads + kv_heads) * head_dim + kv_heads * value_dim:
+        raise invalid_argument("wide_norm_store: qkv has the wrong shape")
+    _float_vector(q_norm, heads * head_dim, "the query norm's weight")
+    _float_vector(k_norm, kv_heads * head_dim, "the key norm's weight")
+    view = kv_view if store else None
+    if view is not None and view.keys.dtype != qkv.dtype:
+        raise invalid_argument("wide_norm_store: the cache and the activations differ in element type")
+    args = WideNormArgs(
+        qkv.data_ptr(), qkv.stride(0), q_norm.data_ptr(), k_norm.data_ptr(), tables.row_seq.data_ptr(),
+        tables.row_pos.data_ptr(), tables.seq_slot.data_ptr(), tables.seq_start.data_ptr(), tables.seq_len.data_ptr(),
+        view.keys.data_ptr() if view is not None else 0, view.values.data_ptr() if view is not None else 0,
+        cache_geometry(view, kv_heads, head_dim), heads, kv_heads, head_dim, value_dim, float(eps))
+    _check(core().kidi_wide_norm_store(ctypes.byref(args), qkv.shape[0], dtype_code(qkv.dtype), _stream()),
+           "wide_norm_store")
+
+
 def attention_generic(qkv: torch.Tensor, out: torch.Tensor, *, heads: int, kv_heads: int, head_dim: int,
                       scale: float, window: Optional[int], tables, kv_view, keys_in_step: bool,
                       softcap: float = 0.0, slopes: Optional[torch.Tensor] = None, value_dim: Optional[int] = None,
-                      sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
+                      sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                      weight_bias: Optional[torch.Tensor] = None, chunk: Optional[int] = None,
+                      out_scale: float = 1.0) -> None:
     """Causal attention of every row of the step over its sequence's keys. Keys of the
     step's own rows are read from `qkv` when `keys_in_step` is set, earlier ones (or
     all of them) from the cache. `softcap` > 0 bounds a score s to softcap * tanh(s / softcap);
     `slopes` (float32 [heads]) adds slopes[h] * (key position - query position) to head h's scores.
     `value_dim` (default head_dim): the width of a value head and of a head of `out`. `sinks` (float32
     [heads]): exp(sinks[h]) joins head h's softmax denominator. `gate` ([rows, heads], a view of the step's
-    element type): head h of a row is multiplied by sigmoid(gate[row, h])."""
+    element type): head h of a row is multiplied by sigmoid(gate[row, h]). `weight_bias` (float32 [heads]): a key's
+    weight is sigmoid(score + weight_bias[h]), normalised over nothing, instead of its share of a softmax. `chunk`: only
+    keys of the query's own run of `chunk` positions (counted from 0) are seen. `out_scale`: a factor on the result."""
     value_dim = head_dim if value_dim is None else int(value_dim)
     if sinks is not None and (sinks.dtype != torch.float32 or sinks.shape != (heads,) or not sinks.is_contiguous()
                               or sinks.device != qkv.device):
@@ -749,6 +816,9 @@ def attention_generic(qkv: torch.Tensor, out: torch.Tensor, *, heads: int, kv_he
     if slopes is not None and (slopes.dtype != torch.float32 or slopes.shape != (heads,) or not slopes.is_contiguous()
                                or slopes.device != qkv.device):
         raise invalid_argument("attention: the score slopes must be a float32 vector with one entry per head")
+    _float_vector(weight_bias, heads, "attention: the bias of the sigmoid weights")
+    if weight_bias is not None and sinks is not None:
+        raise invalid_argument("attention: sigmoid weights have no denominator that a sink could join")
     _need_cuda(qkv, out)
     rows = qkv.shape[0]
     if out.shape != (rows, heads * value_dim) or out.dtype != qkv.dtype or out.stride(1) != 1:
@@ -765,7 +835,8 @@ def attention_generic(qkv: torch.Tensor, out: torch.Tensor, *, heads: int, kv_he
         tables.row_seq.data_ptr(), tables.row_pos.data_ptr(), tables.seq_slot.data_ptr(),
         tables.seq_start.data_ptr(), tables.seq_row0.data_ptr(), rows, heads, kv_heads, head_dim,
         int(window or 0), float(scale), float(softcap or 0.0), slopes.data_ptr() if slopes is not None else 0,
-        value_dim, _ptr(sinks), _ptr(gate), gate.stride(0) if gate is not None else 0)
+        value_dim, _ptr(sinks), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(weight_bias), int(chunk or 0),
+        float(out_scale))
     _check(core().kidi_attention_generic(ctypes.byref(args), dtype_code(qkv.dtype), _stream()), "attention")
 
 

@@ -19,7 +19,7 @@ def library():
     if _library is None:
         lib = load_library("routed")
         lib.kidi_route.argtypes = [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                   c_int, c_int, c_int, c_float, c_void_p]
+                                   c_int, c_int, c_int, c_float, c_void_p, c_void_p]
         lib.kidi_expert_slots.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                                           c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p]
         lib.kidi_gather_slots.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
@@ -39,13 +39,15 @@ def _check_addend(addend, like: torch.Tensor, rows: int, hidden: int) -> None:
 
 
 def route(x: torch.Tensor, router: torch.Tensor, top: int, renormalise: bool, score: str = "sigmoid", groups: int = 1,
-          keep: int = 1, renormalise_eps: float = 0.0):
+          keep: int = 1, renormalise_eps: float = 0.0, bias: Optional[torch.Tensor] = None):
     """(chosen int32 [rows, top], weight float32 [rows, top]) for rows x [rows, hidden] and a router
     [experts, hidden]: logits in 32-bit, scores (a sigmoid of each logit, or with `score` "softmax" a softmax over
     all experts), the `top` largest (ties: the lower index), their scores as weights (with `renormalise` divided by
     their sum plus `renormalise_eps`). With `groups` > 1 the experts form that many equal runs of neighbours and
-    only experts of the `keep` groups with the largest best score can be chosen."""
-    ops._need_cuda(x, router)
+    only experts of the `keep` groups with the largest best score can be chosen. `bias` (float32 [experts]) is added
+    to the logits."""
+    ops._need_cuda(x, router, bias)
+    ops._float_vector(bias, router.shape[0], "the router's bias")
     if x.dim() != 2 or not x.is_contiguous() or router.dim() != 2 or not router.is_contiguous() \
             or router.shape[1] != x.shape[1]:
         raise invalid_argument("the router takes contiguous rows and a contiguous [experts, hidden] matrix")
@@ -55,7 +57,8 @@ def route(x: torch.Tensor, router: torch.Tensor, top: int, renormalise: bool, sc
     _check(library().kidi_route(x.data_ptr(), dtype_code(x.dtype), router.data_ptr(), dtype_code(router.dtype),
                                 chosen.data_ptr(), weight.data_ptr(), rows, hidden, router.shape[0], top,
                                 1 if renormalise else 0, 1 if score == "softmax" else 0, int(groups), int(keep),
-                                float(renormalise_eps), ops._stream()), "route")
+                                float(renormalise_eps), bias.data_ptr() if bias is not None else 0, ops._stream()),
+           "route")
     return chosen, weight
 
 

@@ -22,7 +22,7 @@ class ScalarRecurrenceArgs(ctypes.Structure):
                 ("ldv", c_longlong), ("coef", c_void_p), ("state", c_void_p), ("out", c_void_p), ("row_seq", c_void_p),
                 ("seq_slot", c_void_p), ("seq_row0", c_void_p), ("seq_len", c_void_p), ("seqs", c_int), ("heads", c_int),
                 ("k_heads", c_int), ("q_heads", c_int), ("dim", c_int), ("vdim", c_int), ("extra", c_int),
-                ("coef_width", c_int), ("q_scale", c_float)]
+                ("coef_width", c_int), ("q_scale", c_float), ("decay", c_void_p)]
 
 
 class ShortConvArgs(ctypes.Structure):
@@ -70,21 +70,27 @@ def _float_tensor(x: torch.Tensor, shape, what: str) -> None:
         raise invalid_argument(f"{what} must be a contiguous float32 tensor of shape {tuple(shape)}")
 
 
-def scalar_recurrence(k: torch.Tensor, q: torch.Tensor, v: torch.Tensor, coef: torch.Tensor, state: torch.Tensor, *,
-                      heads: int, k_heads: int, q_heads: int, dim: int, vdim: int, extra: int = 0,
-                      q_scale: float = 1.0, tables, seqs: int) -> torch.Tensor:
+def scalar_recurrence(k: torch.Tensor, q: torch.Tensor, v: torch.Tensor, coef: Optional[torch.Tensor],
+                      state: torch.Tensor, *, heads: int, k_heads: int, q_heads: int, dim: int, vdim: int,
+                      extra: int = 0, q_scale: float = 1.0, tables, seqs: int,
+                      decay: Optional[torch.Tensor] = None) -> torch.Tensor:
     """S_t = a_t S_(t-1) + b_t k_t (v_t, 1 if `extra`)^T and o_t = S_t^T (q_scale q_t) for every sequence's rows of
     the step, from and into `state` [slots + 1, heads, dim, vdim + extra] (float32). k [rows, k_heads * dim],
     q [rows, q_heads * dim], v [rows, heads * vdim] are views of the step's element type (head h reads key head
-    h // (heads / k_heads), likewise q); coef float32 [rows, heads, >= 2] holds (a_t, b_t). Returns the read-out,
-    float32 [rows, heads * (vdim + extra)]."""
+    h // (heads / k_heads), likewise q); coef float32 [rows, heads, >= 2] holds (a_t, b_t), or `decay`
+    (float32 [heads], coef None) holds a_t for every token and b_t is 1. Returns the read-out, float32
+    [rows, heads * (vdim + extra)]."""
     ops._need_cuda(k, q, v, coef, state)
     rows = v.shape[0]
     for tensor, width, what in ((k, k_heads * dim, "keys"), (q, q_heads * dim, "queries"), (v, heads * vdim, "values")):
         _rows_view(tensor, "scalar recurrence")
         if tensor.shape != (rows, width) or tensor.dtype != v.dtype:
             raise invalid_argument(f"scalar recurrence: the {what} have the wrong shape or type")
-    if coef.dtype != torch.float32 or coef.dim() != 3 or coef.shape[:2] != (rows, heads) or coef.shape[2] < 2 \
+    if (coef is None) == (decay is None):
+        raise invalid_argument("scalar recurrence: the decays come per token (coef) or per head (decay)")
+    if decay is not None:
+        _float_tensor(decay, (heads,), "the decays")
+    elif coef.dtype != torch.float32 or coef.dim() != 3 or coef.shape[:2] != (rows, heads) or coef.shape[2] < 2 \
             or not coef.is_contiguous():
         raise invalid_argument("scalar recurrence: the coefficients are float32 [rows, heads, >= 2]")
     if state.dtype != torch.float32 or tuple(state.shape[1:]) != (heads, dim, vdim + extra) or not state.is_contiguous():
@@ -93,9 +99,11 @@ def scalar_recurrence(k: torch.Tensor, q: torch.Tensor, v: torch.Tensor, coef: t
         raise invalid_argument(f"scalar recurrence: the kernel takes up to {MAX_DIM} state rows a head")
     out = torch.empty((rows, heads * (vdim + extra)), dtype=torch.float32, device=v.device)
     args = ScalarRecurrenceArgs(k.data_ptr(), k.stride(0), q.data_ptr(), q.stride(0), v.data_ptr(), v.stride(0),
-                                coef.data_ptr(), state.data_ptr(), out.data_ptr(), tables.row_seq.data_ptr(),
+                                coef.data_ptr() if coef is not None else 0, state.data_ptr(), out.data_ptr(), tables.row_seq.data_ptr(),
                                 tables.seq_slot.data_ptr(), tables.seq_row0.data_ptr(), tables.seq_len.data_ptr(),
-                                seqs, heads, k_heads, q_heads, dim, vdim, extra, coef.shape[2], float(q_scale))
+                                seqs, heads, k_heads, q_heads, dim, vdim, extra,
+                                coef.shape[2] if coef is not None else 0, float(q_scale),
+                                decay.data_ptr() if decay is not None else 0)
     _check(library().kidi_scalar_recurrence(ctypes.byref(args), dtype_code(v.dtype), ops._stream()), "scalar_recurrence")
     return out
 

@@ -138,7 +138,7 @@ class SandwichNormBlock(Part):
     """A norm before and a norm behind each sublayer:
         x <- x + mixer_out_norm(mixer(input_norm(x)));  x <- x + feed_forward_out_norm(feed_forward(post_norm(x)))
     The feed-forward (with its two norms) is optional. The norms behind the sublayers have a weight and no bias
-    (`delta_weight()`); a sublayer's result goes to the stream together with its norm, and the norm that reads the
+    (`apply_delta()`); a sublayer's result goes to the stream together with its norm, and the norm that reads the
     stream next normalises the result, forms the 32-bit sum and normalises the sum in one kernel."""
 
     ROLES = {"input_norm": "norm", "mixer": "mixer", "mixer_out_norm": "norm"}
@@ -155,7 +155,7 @@ class SandwichNormBlock(Part):
         if len({self.post_norm is None, self.feed_forward is None, self.feed_forward_out_norm is None}) != 1:
             raise invalid_argument("a sandwich block has a feed-forward with the norms before and behind it, or none")
         for norm in (self.mixer_out_norm, self.feed_forward_out_norm):
-            if norm is not None and not hasattr(norm, "delta_weight"):
+            if norm is not None and not hasattr(norm, "apply_delta"):
                 raise invalid_argument("the norm behind a sublayer must be one that a residual delta can pass")
 
     def children(self):
@@ -174,6 +174,42 @@ class SandwichNormBlock(Part):
         if self.feed_forward is not None:
             result = self.feed_forward.forward(plain_rows(self.post_norm.forward(stream)), ctx)
             stream.add(result, normed_by=self.feed_forward_out_norm)
+
+
+@register_part("arrangement", "output_norm")
+class OutputNormBlock(Part):
+    """A norm behind each sublayer and none before it: the sublayers read the residual stream itself,
+        x <- x + mixer_out_norm(mixer(x));  x <- x + feed_forward_out_norm(feed_forward(x))
+    The feed-forward (with its norm) is optional. A sublayer's result goes to the stream together with its norm; the next
+    sublayer's read of the stream normalises the result, forms the 32-bit sum and casts it in one kernel."""
+
+    ROLES = {"mixer": "mixer", "mixer_out_norm": "norm"}
+    OPTIONAL_ROLES = {"feed_forward": "feed_forward", "feed_forward_out_norm": "norm"}
+
+    def __init__(self, spec, env, parts: Dict[str, Part]):
+        super().__init__(spec, env)
+        self.mixer = parts["mixer"]
+        self.mixer_out_norm = parts["mixer_out_norm"]
+        self.feed_forward = parts.get("feed_forward")
+        self.feed_forward_out_norm = parts.get("feed_forward_out_norm")
+        if (self.feed_forward is None) != (self.feed_forward_out_norm is None):
+            raise invalid_argument("a block has a feed-forward and the norm behind it, or neither")
+        for norm in (self.mixer_out_norm, self.feed_forward_out_norm):
+            if norm is not None and not hasattr(norm, "apply_delta"):
+                raise invalid_argument("the norm behind a sublayer must be one that a residual delta can pass")
+
+    def children(self):
+        return tuple(part for part in (self.mixer, self.mixer_out_norm, self.feed_forward, self.feed_forward_out_norm)
+                     if part is not None)
+
+    def cache_requests(self) -> list:
+        return self.mixer.cache_requests()
+
+    def forward(self, stream: ResidualStream, ctx, views, owns_cache: bool) -> None:
+        dtype = self.env.dtype
+        stream.add(self.mixer.forward(stream.read(dtype), ctx, views, owns_cache), normed_by=self.mixer_out_norm)
+        if self.feed_forward is not None:
+            stream.add(self.feed_forward.forward(stream.read(dtype), ctx), normed_by=self.feed_forward_out_norm)
 
 
 @register_part("arrangement", "hyper_connections")

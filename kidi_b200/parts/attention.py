@@ -36,6 +36,16 @@ windowed layer keeps every page and the window is a mask, so that prompts may co
 another layer may read the cache); qk_norm_weight (default true; false: the per-head norm of q and k divides by
 the root mean square and has no weight); query_scale (name of a position part with a `table` of one factor per
 position: q is multiplied by its position's factor after norm and rotation).
+
+And: chunk (positions, or None): a query sees only keys of its own run of `chunk` positions, counted from the
+sequence's position 0 (with `ring` the cache keeps that many tokens); qk_norm_scope ("head", the default, or "rows": one
+RMS norm over all query entries of a token before they are split into heads and one over all key entries, with weights
+of those sizes, float32 arithmetic, tensors q_norm_name and k_norm_name); weights ("softmax", the default, or "sigmoid":
+the weight of a key is sigmoid(score + b), b a number per head from the tensor `weight_bias_name`, and the weights are
+not normalised over the keys); out_scale (a factor on the concatenated heads, default 1).
+
+The part can also run on projections that another part holds (`joint_input`, `mix`, `joint_output`; see
+`parallel_mixers`).
 """
 from __future__ import annotations
 
@@ -47,7 +57,7 @@ import torch
 from ..cache.sequence_cache import KVRequest
 from ..errors import invalid_argument, unsupported
 from ..kernels import ops
-from ..kernels.attention import AttentionLauncher
+from ..kernels.attention import AttentionLauncher, reach_of
 from .base import Part
 from .linear import Linear
 from .registry import register_part
@@ -82,7 +92,16 @@ class Attention(Part):
         self.names = {key: spec.param(key + "_name", default) for key, default in (
             ("q", "q_proj.weight"), ("k", "k_proj.weight"), ("v", "v_proj.weight"), ("o", "o_proj.weight"),
             ("sink", "sinks"), ("gate", "gate_proj.weight"), ("q_bias", "q_proj.bias"), ("k_bias", "k_proj.bias"),
-            ("v_bias", "v_proj.bias"))}
+            ("v_bias", "v_proj.bias"), ("q_norm", "q_norm.weight"), ("k_norm", "k_norm.weight"),
+            ("weight_bias", "weight_bias"))}
+        self.chunk = spec.param("chunk", None)
+        self.wide_norm = self.qk_norm and spec.param("qk_norm_scope", "head") == "rows"
+        if spec.param("qk_norm_scope", "head") not in ("head", "rows"):
+            raise invalid_argument("the norm of queries and keys runs over a head or over whole rows")
+        if spec.param("weights", "softmax") not in ("softmax", "sigmoid"):
+            raise invalid_argument("attention weights are a 'softmax' or a 'sigmoid' of the scores")
+        self.sigmoid = spec.param("weights", "softmax") == "sigmoid"
+        self.weight_bias: Optional[torch.Tensor] = None
         scale = spec.param("scale", None)
         self.scale = float(scale) if scale is not None else 1.0 / math.sqrt(float(self.head_dim))
         if self.hidden <= 0 or self.heads <= 0 or self.kv_heads <= 0 or self.heads % self.kv_heads or self.head_dim <= 0:
@@ -91,6 +110,12 @@ class Attention(Part):
             raise unsupported(f"head widths {self.head_dim} and {self.value_dim}: the kernels take 1 to 256")
         if self.window is not None and int(self.window) <= 0:
             raise invalid_argument("an attention window must be positive")
+        if self.chunk is not None and int(self.chunk) <= 0:
+            raise invalid_argument("an attention chunk must be positive")
+        if self.sigmoid and (self.has_sink or self.has_gate):
+            raise unsupported("sigmoid weights with a sink or a gate per head are not built")
+        if self.wide_norm and not (self.own_kv and self.norm_weight):
+            raise unsupported("a norm over whole rows of queries and keys needs both projections and both weights")
         name = spec.param("position", None)
         self.position = env.positions[name] if name is not None else None
         if self.position is not None and self.position.head_dim != self.head_dim:
@@ -122,7 +147,8 @@ class Attention(Part):
             if slopes is not None else None
         self.launcher = AttentionLauncher(heads=self.heads, kv_heads=self.kv_heads, head_dim=self.head_dim,
                                           scale=self.scale, window=self.window, softcap=self.softcap,
-                                          slopes=self.slopes)
+                                          slopes=self.slopes, chunk=self.chunk,
+                                          out_scale=float(spec.param("out_scale", 1.0)))
 
     def parameter_specs(self) -> List[ParamSpec]:
         n = self.names
@@ -142,8 +168,11 @@ class Attention(Part):
         if self.out_bias:
             specs.append(ParamSpec("o_proj.bias", (self.hidden,)))
         if self.qk_norm and self.norm_weight:
-            specs.append(ParamSpec("q_norm.weight", (self.head_dim,), init=("one_plus_normal", 0.1)))
-            specs.append(ParamSpec("k_norm.weight", (self.head_dim,), init=("one_plus_normal", 0.1)))
+            sizes = (self.q_width, self.kv_width) if self.wide_norm else (self.head_dim, self.head_dim)
+            specs.append(ParamSpec(n["q_norm"], (sizes[0],), init=("one_plus_normal", 0.1)))
+            specs.append(ParamSpec(n["k_norm"], (sizes[1],), init=("one_plus_normal", 0.1)))
+        if self.sigmoid:
+            specs.append(ParamSpec(n["weight_bias"], (self.heads,), init=("normal", 1.0)))
         if self.has_sink:
             specs.append(ParamSpec(n["sink"], (self.heads,), init=("normal", 1.0)))
         return specs
@@ -162,14 +191,16 @@ class Attention(Part):
         if self.qk_norm and not self.norm_weight:
             self.q_norm = self.k_norm = torch.ones(self.head_dim, dtype=torch.float32, device=fused.device)
         elif self.qk_norm:
-            self.q_norm, self.k_norm = tensors["q_norm.weight"], tensors["k_norm.weight"]
-            if self.q_norm.dtype != self.k_norm.dtype:
+            self.q_norm, self.k_norm = tensors[self.names["q_norm"]], tensors[self.names["k_norm"]]
+            if self.wide_norm or self.q_norm.dtype != self.k_norm.dtype:
                 self.q_norm, self.k_norm = self.q_norm.float(), self.k_norm.float()
         if self.has_sink:
             self.sinks = tensors[self.names["sink"]].float().contiguous()
+        if self.sigmoid:
+            self.weight_bias = tensors[self.names["weight_bias"]].float().contiguous()
 
     def cache_requests(self) -> list:
-        window = int(self.window) if self.window is not None and self.ring else None
+        window = reach_of(self.window, self.chunk) if self.ring else None
         return [KVRequest(self.kv_heads, self.head_dim, window,
                           value_dim=self.value_dim if self.value_dim != self.head_dim else None)]
 
@@ -178,13 +209,33 @@ class Attention(Part):
         freezes for this part (the form of its decode kernel)."""
         return self.launcher.launch_signature(self.env.dtype, rows, longest, self.env.device)
 
+    # --- projections that another part holds
+    activated_columns = None      # columns of the input projection that pass SiLU before `mix`: none
+
+    def joint_input(self) -> torch.Tensor:
+        """The fused input projection [rows, hidden], rows a multiple of 8."""
+        if self.qkv.bias is not None or self.out.bias is not None:
+            raise unsupported("projections with biases are not shared")
+        return self.qkv.weight
+
+    def joint_output(self) -> torch.Tensor:
+        """The output projection [hidden, out_width]."""
+        return self.out.weight
+
+    def release_projections(self) -> None:
+        self.qkv = self.out = None
+
     def forward(self, x, ctx, views, owns_cache: bool, sink=None) -> Optional[torch.Tensor]:
+        return self.out.forward(self.mix(self.qkv.forward(x), ctx, views, owns_cache), sink=sink)
+
+    def mix(self, qkv: torch.Tensor, ctx, views, owns_cache: bool, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """The concatenated heads' result [rows, out_width] (into `out`, if given) from the projected rows (a view of
+        which may be changed in place)."""
         view = views[0]
         plan = ctx.plan
         if owns_cache and not self.own_kv:
             raise invalid_argument("an attention layer without key and value projections reads another layer's cache "
                                    "(the schedule entry's `cache_from`)")
-        qkv = self.qkv.forward(x)
         position = self.position
         rotate = dict(cos=position.cos, sin=position.sin, rotary_dim=position.rotary_dim) if position is not None \
             else dict(cos=None, sin=None, rotary_dim=0)
@@ -200,6 +251,8 @@ class Attention(Part):
             extras["gate"] = qkv[:, self.gate_begin:self.gate_begin + self.heads]
         if self.value_dim != self.head_dim:
             extras["value_dim"] = self.value_dim
+        if self.sigmoid:
+            extras["weight_bias"] = self.weight_bias
         # A ring that is written before attention would lose keys that the step's
         # earlier rows still need; it is written afterwards unless the step is one
         # token per sequence. A full-history cache is written first.
@@ -209,11 +262,21 @@ class Attention(Part):
         # One token per sequence on the tensor-core path: the attention kernel takes the rows as
         # the projection left them and does norm, rotation and the cache write itself.
         fused = owns_cache and store_first and self.value_dim == self.head_dim and self.query_scale is None \
+            and not self.wide_norm \
             and self.launcher.fuses_rotation(plan, qkv, kv_view=view, q_norm=self.q_norm, k_norm=self.k_norm, **rotate)
-        if not fused:
+        if self.wide_norm:
+            plain = position is None and self.query_scale is None
+            ops.wide_norm_store(qkv, q_norm=self.q_norm, k_norm=self.k_norm, eps=self.eps, tables=ctx.tables, kv_view=view,
+                                store=store_first and plain, heads=self.heads, kv_heads=self.kv_heads,
+                                head_dim=self.head_dim, value_dim=self.value_dim)
+            if not plain:
+                ops.rope_store(qkv, q_norm=None, k_norm=None, eps=self.eps, tables=ctx.tables, kv_view=view,
+                               store=store_first, **rotate, **common)
+        elif not fused:
             ops.rope_store(qkv, q_norm=self.q_norm, k_norm=self.k_norm, eps=self.eps, tables=ctx.tables, kv_view=view,
                            store=store_first, **rotate, **common)
-        attended = torch.empty((qkv.shape[0], self.out_width), dtype=qkv.dtype, device=qkv.device)
+        attended = out if out is not None else torch.empty((qkv.shape[0], self.out_width), dtype=qkv.dtype,
+                                                           device=qkv.device)
         keys_in_step = owns_cache and not plan.is_decode
         rotation = dict(q_norm=self.q_norm, k_norm=self.k_norm, eps=self.eps, store=True, **rotate) if fused else None
         self.launcher.run(ctx, qkv, attended, kv_view=view, keys_in_step=keys_in_step, rotation=rotation,
@@ -223,4 +286,4 @@ class Attention(Part):
                            transform=False, cos=None, sin=None, rotary_dim=0, **common)
         if self.output_gate:
             ops.sigmoid_gate(attended, qkv[:, self.gate_begin:self.gate_begin + self.out_width])
-        return self.out.forward(attended, sink=sink)
+        return attended

@@ -12,6 +12,7 @@ Interfaces by role (each is registered with `register_part(role, kind)`):
                  (both optionally: class attribute `accepts_row_scaled = True`: x may be a `RowScaled`;
                  `takes_sink = True`: `forward(..., sink=ResidualSink)` may return None after adding y
                  to the residual stream itself)
+                 (both of which another part may run on projections it holds itself: see `parallel_mixers`)
 * arrangement:   `__init__(spec, env, parts)`; `forward(stream, ctx, views, owns_cache)`
 * token_input:   `forward(stream, ctx, mix=None)`: adds something computed from the rows' token ids to the stream
                  (after taking the pending delta); `mix`, a stream_mix part, may be applied in the same kernel
@@ -73,6 +74,9 @@ class Part:
         for name, tensor in tensors.items():
             setattr(self, "_" + name.replace(".", "_"), tensor)
 
+    def bound(self) -> None:
+        """Called once the part and all its children have received their tensors."""
+
     # --- cache
     def cache_requests(self) -> list:
         return []
@@ -100,6 +104,7 @@ def bind_all(part: Part, bound: Dict[str, torch.Tensor]) -> None:
         part.bind(own)
     for child in part.children():
         bind_all(child, bound)
+    part.bound()
 
 
 class RowScaled:
@@ -157,7 +162,7 @@ class ResidualStream:
     def __init__(self, hidden: torch.Tensor):
         self.hidden = hidden
         self.pending: Optional[torch.Tensor] = None
-        self.pending_norm = None      # a norm (with `delta_weight()`) that the pending delta passes before it is added
+        self.pending_norm = None      # a norm (with `apply_delta()`) that the pending delta passes before it is added
         self.prepared = None
         # Copies of the stream that a part keeps for later layers (role "stream_mix"): [n, rows, hidden]
         # float32, and how many of them are filled. `hidden` is then a view of one of them.
@@ -173,8 +178,8 @@ class ResidualStream:
 
     def add(self, delta: Optional[torch.Tensor], normed_by=None) -> None:
         """`delta` None: the part that made it has added it through a sink already. `normed_by`: a norm part
-        with `delta_weight()` (a layer norm without bias) that the delta passes before it is added; the norm
-        that reads the stream next does both in its kernel when it can (`take_pending_normed`)."""
+        with `apply_delta()` (a layer norm without bias, an RMS norm) that the delta passes before it is added; what
+        reads the stream next does both in its kernel when it can (`take_pending_normed`)."""
         if delta is None:
             return
         if self.pending is not None:
@@ -205,10 +210,25 @@ class ResidualStream:
         delta, norm = self.take_pending_normed()
         if norm is None:
             return delta
-        from ..kernels import ops
-        weight, eps = norm.delta_weight()
-        ops.add_layernorm(self.hidden, delta, None, None, 0.0, None, delta_weight=weight, delta_eps=eps)
+        norm.apply_delta(self.hidden, delta)
         return None
+
+    def read(self, dtype: torch.dtype) -> torch.Tensor:
+        """The stream itself, with its pending delta added, in `dtype` (for sublayers that read no norm of it)."""
+        from ..kernels import ops
+        self.prepared = None
+        delta, norm = self.take_pending_normed()
+        copy = dtype if dtype != torch.float32 else None
+        if delta is not None and norm is not None:
+            if hasattr(norm, "delta_parts"):
+                weight, groups, eps = norm.delta_parts()
+                made = ops.add_parts_norm(self.hidden, delta, copy, delta_weight=weight, delta_groups=groups, delta_eps=eps)
+            else:
+                norm.apply_delta(self.hidden, delta)
+                made = ops.add_parts_norm(self.hidden, None, copy) if copy is not None else None
+        else:
+            made = ops.add_parts_norm(self.hidden, delta, copy) if delta is not None or copy is not None else None
+        return self.hidden if copy is None else made
 
     def take_pending_normed(self):
         """(delta, norm): the pending delta and the norm it has to pass first (None: none)."""

@@ -42,12 +42,15 @@ class Linear:
         self.bias = bias.float().contiguous() if bias is not None else None
 
     def forward(self, x, out_dtype: Optional[torch.dtype] = None, out: Optional[torch.Tensor] = None,
-                sink=None) -> Optional[torch.Tensor]:
-        """`x`: a matrix or a `RowScaled` (rows that lack their norm's factor: the weight-streaming
+                sink=None, silu_columns=None) -> Optional[torch.Tensor]:
+        """`silu_columns`: (begin, end) of result columns that pass SiLU. `x`: a matrix or a `RowScaled` (rows that lack their norm's factor: the weight-streaming
         kernel applies it to its result, any other kernel gets plain rows). `sink`: a
         `ResidualSink`; if the weight-streaming kernel runs and the sink's norm takes prepared
         rows, the result goes into the residual stream and None is returned."""
         from ..kernels import skinny
+        if silu_columns is not None:
+            from ..kernels import linear_attention
+            return linear_attention.silu_columns(self.forward(x, out_dtype, out), *silu_columns)
         weight, bias = self.weight, self.bias
         factors = None
         if isinstance(x, RowScaled):

@@ -12,7 +12,8 @@ weight_on ("input"), router_name ("router"), expert_name ("e{index}."), gate_nam
 holds each expert's three matrices under `<prefix><expert_name><gate|up|down>`; they are bound as two stacked
 tensors, [experts, 2 * expert_size, hidden] (gate rows, then up rows) and [experts, hidden, expert_size].
 
-Variants, all parameters: score "softmax" (s = softmax(z) over all experts); renormalise_eps (added to the sum
+Variants, all parameters: router_bias_name (a tensor [experts] added to the logits; a softmax score that is
+renormalised with renormalise_eps 0 is then the softmax over the chosen logits alone, bias included); score "softmax" (s = softmax(z) over all experts); renormalise_eps (added to the sum
 that the chosen scores are divided by); groups and keep_groups: the experts form `groups` equal runs of
 neighbours, a group's score is its largest, and only experts of the `keep_groups` best groups can be chosen;
 expert_form "plain": an expert has no gate, expert(x) = W_down gelu(W_up x) with the exact (erf) gelu, and the
@@ -80,6 +81,8 @@ class RoutedExperts(Part):
         if self.shared_size is not None and self.shared_size <= 0:
             raise invalid_argument("a shared expert has a positive width")
         self.router_name = spec.param("router_name", "router")
+        self.router_bias_name = spec.param("router_bias_name", None)
+        self.router_bias: Optional[torch.Tensor] = None
         self.expert_name = spec.param("expert_name", "e{index}.")
         self.gate_name, self.up_name, self.down_name = (spec.param(key + "_name", key) for key in ("gate", "up", "down"))
         self.router: Optional[torch.Tensor] = None
@@ -96,6 +99,8 @@ class RoutedExperts(Part):
             down.append((name + self.down_name, (self.hidden, self.inter)))
         per = (2 if self.gated else 1) * self.inter
         specs = [ParamSpec(self.router_name, (self.experts, self.hidden)),
+                 *([ParamSpec(self.router_bias_name, (self.experts,), init=("normal", 0.1))]
+                   if self.router_bias_name is not None else []),
                  ParamSpec("experts.gate_up", (self.experts * per, self.hidden), sources=tuple(first)),
                  ParamSpec("experts.down", (self.experts * self.hidden, self.inter), sources=tuple(down))]
         if self.shared_size is not None:
@@ -112,6 +117,8 @@ class RoutedExperts(Part):
     def bind(self, tensors) -> None:
         per = (2 if self.gated else 1) * self.inter
         self.router = tensors[self.router_name]
+        if self.router_bias_name is not None:
+            self.router_bias = tensors[self.router_bias_name].float().contiguous()
         self.gate_up = tensors["experts.gate_up"].view(self.experts, per, self.hidden)
         self.down = tensors["experts.down"].view(self.experts, self.hidden, self.inter)
         self._gate_up = [Linear(self.gate_up[index]) for index in range(self.experts)]
@@ -142,7 +149,7 @@ class RoutedExperts(Part):
     def _forward_routed(self, x, ctx, addend=None) -> torch.Tensor:
         rows = x.shape[0]
         chosen, weight = routed.route(x, self.router, self.top, self.renormalise, self.score, self.groups,
-                                      self.keep_groups, self.renormalise_eps)
+                                      self.keep_groups, self.renormalise_eps, self.router_bias)
         slots = rows * self.top
         if x.dtype == torch.float32 or self.gate_up.dtype == torch.float32 or ctx.plan.is_decode \
                 or slots <= SLOT_PATH_MAX:

@@ -94,3 +94,4 @@ def _load_builtin() -> None:
         from .models import gakenex  # noqa: F401
         from .models import gazezen  # noqa: F401
         from .models import biropel  # noqa: F401
+        from .models import dibesun  # noqa: F401
