@@ -2,7 +2,7 @@
 """Decode and prefill throughput of the library on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch B] [--model 8b|14b|32b] [--impl ours|reference]
-    python bench.py --design sanozen|gakenex|gazezen|biropel [--widths 2048,4096] [--layers 4]     (another record; see `design_comparison`)
+    python bench.py --design sanozen|gakenex|gazezen|biropel|dibesun [--widths 2048,4096] [--layers 4]     (another record; see `design_comparison`)
 
 A step is one decode step of the batch. The default run is the Qwen3-8B shape (every
 layer size, all 36 layers) with random bfloat16 weights drawn on the device from a
@@ -384,7 +384,28 @@ def biropel_shape(width: int, layers: int = 4) -> dict:
             "streams": 2, "layers": stack}
 
 
-DESIGN_SHAPES = {"sanozen": sanozen_shape, "gakenex": gakenex_shape, "gazezen": gazezen_shape, "biropel": biropel_shape}
+def dibesun_shape(width: int, layers: int = 4) -> dict:
+    """A Dibesun stack at the layer sizes of a model of `width`: in every layer attention with sigmoid weights (half the
+    heads, of 128, a key/value head for four heads, runs of 1,536 positions, bounded scores) beside linear attention (as
+    many heads of 128 x 128); dense SiLU-gated feed-forwards of the Qwen3 layers' size in turn with sixteen routed
+    experts of a quarter of it, two a token, plus a shared one of half of it (a token uses as many feed-forward
+    weights); norms in eight parts."""
+    heads = max(1, width // 256)
+    inter = (8 * width // 3 + 127) // 128 * 128
+    left = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+            "softcap": 50.0, "mask": {"size": 1536}}
+    right = {"heads": heads, "dim": 128, "vdim": 128,
+             "decay": [1.0 - 2.0 ** (-1.0 - 9.0 * index / max(1, heads - 1)) for index in range(heads)]}
+    mixer = {"left": left, "right": right, "left_scale": 0.8, "right_scale": 0.6}
+    dense = {"kind": "dense", "ff": inter}
+    routed = {"kind": "moe", "expert": {"ff": inter // 4}, "router": {"experts": 16, "top": 2}, "shared": {"ff": inter // 2}}
+    stack = [{"type": "parallel", "mixer": mixer, "mlp": dense if index % 2 == 0 else routed} for index in range(layers)]
+    return {"architecture": "Dibesun", "vocab": 32768, "width": width, "max_positions": 8192,
+            "norm": {"eps": 1e-5, "groups": 8}, "embedding": {"scale": 2.0}, "layers": stack}
+
+
+DESIGN_SHAPES = {"sanozen": sanozen_shape, "gakenex": gakenex_shape, "gazezen": gazezen_shape, "biropel": biropel_shape,
+                 "dibesun": dibesun_shape}
 
 
 def qwen3_shape(width: int, layers: int = 4) -> dict:
@@ -400,9 +421,9 @@ KERNEL_CLASSES = (
     ("products", ("gemm_", "library_mm", "library_bmm", "gemm_heads")),
     ("prompt attention", ("attention_prefill",)),
     ("decode attention", ("attention_decode", "latent_attention")),
-    ("recurrence", ("gated_recurrence", "scalar_recurrence")),
-    ("stream norm", ("add_rmsnorm", "add_layernorm", "lanes_")),
-    ("activation", ("silu_gate", "poly_norm", "bounded_gate", "gelu", "relu_squared")),
+    ("recurrence", ("gated_recurrence", "scalar_recurrence", "linear_attention")),
+    ("stream norm", ("add_rmsnorm", "add_layernorm", "lanes_", "add_parts_norm")),
+    ("activation", ("silu_gate", "poly_norm", "bounded_gate", "gelu", "relu_squared", "silu_columns")),
     ("experts through the choice", ("expert_slots",)),
 )
 
@@ -537,7 +558,40 @@ def class_work(design: str, config: dict, rows: int, context: int, decode: bool)
         work["decode attention"] = ("bytes", cache)
         work["recurrence"] = ("bytes", scan)
         norms = 2                                                     # the embedding's norm and the final one
-        stream += 0.0
+    elif design == "dibesun":
+        width, layers = config["width"], config["layers"]
+        weights, norms, act_width, attention, cache, chosen, scan = config["vocab"] * width, 1, 0, 0.0, 0.0, 0.0, 0.0
+        for layer in layers:
+            left, right, mlp = layer["mixer"]["left"], layer["mixer"]["right"], layer["mlp"]
+            heads, groups, dim, vdim, chunk = left["heads"], left["kv_heads"], left["dim"], left["vdim"], left["mask"]["size"]
+            keys, values = right["heads"] * right["dim"], right["heads"] * right["vdim"]
+            norms += 2
+            weights += width * (heads * dim + groups * (dim + vdim) + 2 * keys + 2 * values) + (heads * vdim + values) * width
+            act_width += 0 if decode else 2 * (2 * keys + values)        # decoding: in the product's epilogue
+            whole, rest = divmod(rows, chunk)
+            pairs = whole * chunk * (chunk + 1) / 2 + rest * (rest + 1) / 2
+            attention += 2.0 * heads * (dim + vdim) * pairs
+            cache += rows * ((context - 1) % chunk + 1) * groups * (dim + vdim) * 2.0
+            scan += rows * (2 * keys + values) * 2.0 + rows * values * 4.0 \
+                + (rows if decode else 1) * 2.0 * right["heads"] * right["dim"] * right["vdim"] * 4
+            if mlp["kind"] == "dense":
+                weights += 3 * width * mlp["ff"]
+                act_width += 0 if decode else 3 * mlp["ff"]
+                continue
+            router, ff, shared = mlp["router"], mlp["expert"]["ff"], mlp["shared"]["ff"]
+            weights += router["experts"] * width + 3 * width * shared
+            used = 3 * width * ff * router["top"]                                    # per token
+            act_width += 3 * shared
+            if decode:         # each (row, choice) streams its expert's weights
+                chosen += rows * used * 2.0
+            else:
+                weights += used
+                act_width += 3 * ff * router["top"]
+        work["prompt attention"] = ("flops", attention)
+        work["decode attention"] = ("bytes", cache)
+        work["recurrence"] = ("bytes", scan)
+        if decode:
+            work["experts through the choice"] = ("bytes", chosen)
     else:
         width, layers = config["width"], config["layers"]
         weights, norms, act_width, attention, cache, scan_flops, scan_bytes, state = config["vocab"] * width, 1, 0, 0.0, 0.0, 0.0, 0.0, 0.0
@@ -571,7 +625,7 @@ def class_work(design: str, config: dict, rows: int, context: int, decode: bool)
 
 
 def design_comparison(args) -> int:
-    """`--design sanozen` / `--design gakenex` / `--design gazezen` / `--design biropel`: prompts and decoding of a stack of that design beside Qwen3 layers
+    """`--design <one of DESIGN_SHAPES>`: prompts and decoding of a stack of that design beside Qwen3 layers
     of equal size, with every class of kernel against its roofline."""
     import torch
     from kidi_b200 import Engine
@@ -633,8 +687,8 @@ def design_comparison(args) -> int:
 
 def main() -> int:
     parser = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
-    parser.add_argument("--design", default="", choices=["", "sanozen", "gakenex", "gazezen", "biropel"],
-                        help="a Sanozen, Gakenex or Gazezen stack beside Qwen3 layers of equal size, kernel class by kernel class "
+    parser.add_argument("--design", default="", choices=["", *sorted(DESIGN_SHAPES)],
+                        help="a stack of one of these designs beside Qwen3 layers of equal size, kernel class by kernel class "
                              "(the default workload is left as it is)")
     parser.add_argument("--widths", default="2048,4096", help="model widths of --design runs")
     parser.add_argument("--gpus", type=int, default=1)

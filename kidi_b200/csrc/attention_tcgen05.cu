@@ -214,6 +214,32 @@ struct Control {
     int gave_up;
 };
 
+// tanh(x) = x T(x^2) near zero: see `sigmoid_share`.
+constexpr float NEAR_REACH = 0.3f, TANH_REACH = 0.75f;
+constexpr double NEAR0 = 0.999999989568623, NEAR1 = -0.33332962017166656, NEAR2 = 0.13312577657806252,
+                 NEAR3 = -0.05022099099332847;
+// (Made on the host: a kernel parameter is read where it is used and holds no register in between.)
+struct SigmoidShape {
+    float inner, outer;                 // tanh's argument is raw * inner; exponent = outer * tanh(..) + bias (FORM 0: raw * outer + bias)
+    float near[4];                      // FORM 1: exponent = raw * (near0 + near1 raw^2 + ..) + bias
+    float near_raw, reach_raw;          // the largest raw scores that forms 1 and 2 take
+};
+static SigmoidShape sigmoid_shape(float scale, float softcap) {
+    SigmoidShape shape;
+    const bool bounded = softcap > 0.f;
+    shape.inner = bounded ? scale / softcap : 0.f;
+    shape.outer = (bounded ? -softcap : -scale) * LOG2E;
+    const double square = (double)shape.inner * shape.inner, factor = (double)shape.inner * shape.outer;
+    shape.near[0] = (float)(NEAR0 * factor);
+    shape.near[1] = (float)(NEAR1 * factor * square);
+    shape.near[2] = (float)(NEAR2 * factor * square * square);
+    shape.near[3] = (float)(NEAR3 * factor * square * square * square);
+    shape.reach_raw = bounded ? TANH_REACH / shape.inner : 0.f;
+    // (the powers of the scale in the short polynomial's coefficients must not vanish)
+    shape.near_raw = bounded && shape.inner > 1e-4f ? NEAR_REACH / shape.inner : -1.f;
+    return shape;
+}
+
 struct Params {
     bf16* out;              // [rows, ldo]
     long long ldo;
@@ -236,6 +262,8 @@ struct Params {
     const float* weight_bias;   // [heads], sigmoid build only: a key's weight is sigmoid(score + weight_bias[h])
     int chunk;              // > 0: only keys of the query's own run of `chunk` positions are seen
     float out_scale;        // the result is multiplied by it
+    SigmoidShape shape;
+    int block_heads;        // query heads of a block: HEADS, or 1 where blocks of HEADS would leave SMs without one
 };
 
 // Where a block works: its sequence, query rows, heads and key tiles.
@@ -247,10 +275,10 @@ struct Place {
         const int q_index = gridDim.z - 1 - blockIdx.z;
         const int seq = blockIdx.y;
         const int group_size = p.heads / p.kv_heads;
-        const int pairs = (group_size + HEADS - 1) / HEADS;
+        const int pairs = (group_size + p.block_heads - 1) / p.block_heads;
         kv_head = blockIdx.x / pairs;
-        head0 = kv_head * group_size + (blockIdx.x % pairs) * HEADS;     // the block's first query head
-        heads_here = min(HEADS, (kv_head + 1) * group_size - head0);
+        head0 = kv_head * group_size + (blockIdx.x % pairs) * p.block_heads;     // the block's first query head
+        heads_here = min(p.block_heads, (kv_head + 1) * group_size - head0);
         count = p.seq_len[seq];
         q0 = q_index * BM;
         row0 = p.seq_row0[seq];
@@ -303,10 +331,10 @@ __device__ __forceinline__ float probabilities(const float (&s)[SHARE], float sc
     return sum;
 }
 
-// Bounded scores for the sigmoid: tanh(x) = x T(x^2) on |x| <= TANH_REACH, T the polynomial that interpolates
-// tanh(sqrt(y)) / sqrt(y) at the six Chebyshev nodes of [0, TANH_REACH^2] (error below 2e-8): multiply-adds instead
-// of an exponential and a division for every score while a thread's scores all lie within the reach.
-constexpr float TANH_REACH = 0.75f;
+// Bounded scores for the sigmoid: tanh(x) = x T(x^2) on |x| <= reach, T a polynomial that interpolates
+// tanh(sqrt(y)) / sqrt(y) at Chebyshev nodes of [0, reach^2]: multiply-adds instead of an exponential and a division
+// for every score while a thread's scores all lie within the reach. Two polynomials: four coefficients for scores up
+// to 0.3 of the bound (error below 3.1e-9), six for scores up to 0.75 of it (below 2e-8).
 __device__ __forceinline__ float tanh_ratio(float y) {
     float t = fmaf(y, -0.004711522234108173f, 0.019576216423628997f);
     t = fmaf(y, t, -0.053341115327886254f);
@@ -321,27 +349,64 @@ __device__ __forceinline__ float reciprocal_approx(float x) {
     return y;
 }
 
+// Pairs of 32-bit numbers in one register pair: one instruction for two multiply-adds.
+typedef unsigned long long float_pair;
+__device__ __forceinline__ float_pair pair_of(float x, float y) {
+    float_pair p;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(p) : "f"(x), "f"(y));
+    return p;
+}
+__device__ __forceinline__ void parts_of(float_pair p, float& x, float& y) {
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(p));
+}
+__device__ __forceinline__ float_pair pair_mul(float_pair a, float_pair b) {
+    float_pair p;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(p) : "l"(a), "l"(b));
+    return p;
+}
+__device__ __forceinline__ float_pair pair_fma(float_pair a, float_pair b, float_pair c) {
+    float_pair p;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(p) : "l"(a), "l"(b), "l"(c));
+    return p;
+}
+__device__ __forceinline__ float_pair pair_add(float_pair a, float_pair b) {
+    float_pair p;
+    asm("add.rn.f32x2 %0, %1, %2;" : "=l"(p) : "l"(a), "l"(b));
+    return p;
+}
+
 // P = sigmoid(score + bias), rounded to bfloat16 and packed in pairs. Two weights share one reciprocal:
 // 1 / a = b / (a b) with a, b = 1 + exp(-z); z is held above -41.6 (2^-60), so that the product stays finite.
-// FORM 0: scores as they are; 1: bounded, all within the reach of the polynomial; 2: bounded, any.
+// FORM 0: scores as they are; 1: bounded, all within the reach of the short polynomial, whose coefficients come with the
+// score's scale and the factors of the exponent in them; 2: bounded, all within the reach of the long polynomial; 3: any.
 template <bool MASKED, int FORM>
-__device__ __forceinline__ void sigmoid_share(const float (&s)[SHARE], float inner, float outer, float bias_log2, int first,
-                                              int last, unsigned (&packed)[SHARE / 2]) {
+__device__ __forceinline__ void sigmoid_share(const float (&s)[SHARE], const SigmoidShape& shape, float bias_log2, int first, int last,
+                                              unsigned (&packed)[SHARE / 2]) {
+    const float_pair bias = pair_of(bias_log2, bias_log2), one = pair_of(1.f, 1.f);
+    float_pair near[4];
+    if (FORM == 1) {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) near[k] = pair_of(shape.near[k], shape.near[k]);
+    }
+    const float_pair outer = pair_of(shape.outer, shape.outer);
 #pragma unroll
     for (int i = 0; i < SHARE; i += 2) {
-        float z[2];
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-            float x = s[i + e];
-            if (FORM == 1) {
-                x *= inner;
-                x *= tanh_ratio(x * x);
-            } else if (FORM == 2) {
-                x = tanh_near(x * inner);
+        float_pair x = pair_of(s[i], s[i + 1]), z;
+        if (FORM == 1) {
+            const float_pair y = pair_mul(x, x);
+            z = pair_fma(x, pair_fma(y, pair_fma(y, pair_fma(y, near[3], near[2]), near[1]), near[0]), bias);
+        } else {
+            if (FORM == 2) {
+                const float u = s[i] * shape.inner, v = s[i + 1] * shape.inner;
+                x = pair_of(u * tanh_ratio(u * u), v * tanh_ratio(v * v));
+            } else if (FORM == 3) {
+                x = pair_of(tanh_near(s[i] * shape.inner), tanh_near(s[i + 1] * shape.inner));
             }
-            z[e] = fmaf(outer, x, bias_log2);
+            z = pair_fma(x, outer, bias);
         }
-        const float a = 1.f + exp2_approx(fminf(z[0], 60.f)), b = 1.f + exp2_approx(fminf(z[1], 60.f));
+        float z0, z1, a, b;
+        parts_of(z, z0, z1);
+        parts_of(pair_add(pair_of(exp2_approx(fminf(z0, 60.f)), exp2_approx(fminf(z1, 60.f))), one), a, b);
         const float both = reciprocal_approx(a * b);
         float p0 = b * both, p1 = a * both;
         if (MASKED) {
@@ -354,21 +419,19 @@ __device__ __forceinline__ void sigmoid_share(const float (&s)[SHARE], float inn
 }
 
 template <bool MASKED>
-__device__ __forceinline__ void sigmoid_weights(const float (&s)[SHARE], float scale, float softcap, float bias, int first,
-                                                int last, unsigned (&packed)[SHARE / 2]) {
-    const float bias_log2 = -bias * LOG2E;
-    if (softcap <= 0.f) {
-        sigmoid_share<MASKED, 0>(s, 0.f, -scale * LOG2E, bias_log2, first, last, packed);
+__device__ __forceinline__ void sigmoid_weights(const float (&s)[SHARE], const SigmoidShape& shape, float bias_log2, int first, int last,
+                                                unsigned (&packed)[SHARE / 2]) {
+    if (shape.inner == 0.f) {
+        sigmoid_share<MASKED, 0>(s, shape, bias_log2, first, last, packed);
         return;
     }
-    const float inner = scale / softcap, outer = -softcap * LOG2E;
     float most[2] = {0.f, 0.f};
 #pragma unroll
     for (int i = 0; i < SHARE; ++i) most[i & 1] = fmaxf(most[i & 1], fabsf(s[i]));
-    if (fmaxf(most[0], most[1]) * inner <= TANH_REACH)
-        sigmoid_share<MASKED, 1>(s, inner, outer, bias_log2, first, last, packed);
-    else
-        sigmoid_share<MASKED, 2>(s, inner, outer, bias_log2, first, last, packed);
+    const float top = fmaxf(most[0], most[1]);
+    if (top <= shape.near_raw) sigmoid_share<MASKED, 1>(s, shape, bias_log2, first, last, packed);
+    else if (top <= shape.reach_raw) sigmoid_share<MASKED, 2>(s, shape, bias_log2, first, last, packed);
+    else sigmoid_share<MASKED, 3>(s, shape, bias_log2, first, last, packed);
 }
 
 // Writes a thread's packed P into the swizzled K-major tile. `p_row` is the shared-memory
@@ -567,7 +630,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map, const 
             const int first_seen = first_visible(position, p.window, p.chunk);
             const int last_first_seen = first_visible(at.start + q0 + BM - 1, p.window, p.chunk);
             const float scale_log2 = p.scale * LOG2E;
-            const float weight_bias = SIGMOID ? p.weight_bias[head0 + h] : 0.f;
+            const float bias_log2 = SIGMOID ? -p.weight_bias[head0 + h] * LOG2E : 0.f;
             float reference = -INFINITY;                            // what the exponentials are taken against
             float denom = 0.f;                                      // this thread's part of the row sum
             unsigned exchanges = 0;                                 // uses of row_shared so far
@@ -597,8 +660,8 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map, const 
                 mbarrier_arrive(&ctl.s_free[h]);
                 if constexpr (SIGMOID) {
                     unsigned packed[SHARE / 2];
-                    if (masked) sigmoid_weights<true>(s, p.scale, p.softcap, weight_bias, first, last, packed);
-                    else sigmoid_weights<false>(s, p.scale, p.softcap, weight_bias, first, last, packed);
+                    if (masked) sigmoid_weights<true>(s, p.shape, bias_log2, first, last, packed);
+                    else sigmoid_weights<false>(s, p.shape, bias_log2, first, last, packed);
                     if (j > 0) {                     // the product of the tile before has read its P
                         ok = mbarrier_wait(&ctl.pv_done[h], (j - 1) & 1, abort_flag);
                         if (!ok) break;
@@ -855,9 +918,17 @@ KIDI_API int kidi_attention_prefill_tcgen05(const void* qkv, long long ld, int r
         p.chunk = extras->chunk;
         p.out_scale = extras->out_scale;
     }
+    p.shape = sigmoid_shape(p.scale, p.softcap);
     if (p.chunk < 0 || (SIGMOID && (!p.weight_bias || p.sinks || p.gate))) return KIDI_REFUSED_SIZE;
     const int group_size = heads / kv_heads;
-    dim3 grid(kv_heads * ((group_size + HEADS - 1) / HEADS), seqs, (max_new + BM - 1) / BM);
+    const long long row_tiles = (long long)seqs * ((max_new + BM - 1) / BM);
+    static int sms[64] = {};
+    if (!sms[device] && cudaDeviceGetAttribute(&sms[device], cudaDevAttrMultiProcessorCount, device) != cudaSuccess)
+        return KIDI_REFUSED_SIZE;
+    // A block fills an SM. Blocks of one head load K and V once a head instead of once a pair, but there are twice as many:
+    // they win while blocks of two heads are fewer than the SMs.
+    p.block_heads = row_tiles * kv_heads * ((group_size + HEADS - 1) / HEADS) < sms[device] ? 1 : HEADS;
+    dim3 grid(kv_heads * ((group_size + p.block_heads - 1) / p.block_heads), seqs, (max_new + BM - 1) / BM);
     attention_prefill_tcgen05_kernel<<<grid, THREADS, SHARED_BYTES, stream>>>(map, k_map, v_map, p);
     return kidi_launch_status();
 }

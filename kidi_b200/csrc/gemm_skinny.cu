@@ -49,7 +49,8 @@ struct Epilogue {
     float* parts_out;
     int parts_stride;
     int gelu;                     // the plain store writes an activation of y + bias instead of y + bias: 1 the exact
-                                  // (erf) gelu, 2 the squared relu max(y + bias, 0)^2
+                                  // (erf) gelu, 2 the squared relu max(y + bias, 0)^2, 3 SiLU on the output features
+    int silu_begin, silu_end;     // silu_begin .. silu_end - 1
 };
 
 __device__ __forceinline__ uint4 load_streaming(const void* pointer) {
@@ -249,6 +250,7 @@ gemm_skinny_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, TY* _
         } else if (inside) {
             if (!GATED && e.gelu == 1) sum = 0.5f * sum * (1.0f + erff(sum * 0.70710678118654752440f));
             if (!GATED && e.gelu == 2) sum = fmaxf(sum, 0.f) * fmaxf(sum, 0.f);
+            if (!GATED && e.gelu == 3 && n0 + r >= e.silu_begin && n0 + r < e.silu_end) sum = sum / (1.0f + expf(-sum));
             y[m * ldy + n0 + r] = from_float<TY>(sum);
         }
     }
@@ -298,7 +300,8 @@ struct KidiSkinnyExtras {          // every pointer may be null: the plain produ
     float* parts_out;
     int parts_stride;
     int gelu;                      // not gated, not into the residual: the result passes the exact gelu (1) or the
-                                   // squared relu (2)
+                                   // squared relu (2), or its features silu_begin .. silu_end - 1 pass SiLU (3)
+    int silu_begin, silu_end;
 };
 
 // How many parts per row the product into the residual writes for N features.
@@ -327,6 +330,8 @@ KIDI_API int kidi_gemm_skinny(const void* x, const void* w, void* y, int y_dtype
         e.parts_out = extras->parts_out;
         e.parts_stride = extras->parts_stride;
         e.gelu = extras->gelu;
+        e.silu_begin = extras->silu_begin;
+        e.silu_end = extras->silu_end;
         if (e.gelu && (gated || e.residual)) return KIDI_REFUSED_SIZE;
         if (e.factor_parts && (e.factor_count < 1 || e.factor_stride < e.factor_count || e.factor_width < 1))
             return KIDI_REFUSED_SIZE;

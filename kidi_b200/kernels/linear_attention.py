@@ -3,6 +3,8 @@ when a model with such a layer first runs."""
 from __future__ import annotations
 
 import ctypes
+import os
+from typing import Dict
 
 import torch
 
@@ -20,7 +22,46 @@ class LinearStepArgs(ctypes.Structure):
                 ("vdim", c_int)]
 
 
+class LinearChunksArgs(ctypes.Structure):
+    _fields_ = [("q", c_void_p), ("ldq", c_longlong), ("k", c_void_p), ("ldk", c_longlong), ("v", c_void_p),
+                ("ldv", c_longlong), ("decay", c_void_p), ("state", c_void_p), ("out", c_void_p), ("sums", c_void_p),
+                ("before", c_void_p), ("row_seq", c_void_p), ("seq_slot", c_void_p), ("seq_row0", c_void_p),
+                ("seq_len", c_void_p), ("seqs", c_int), ("heads", c_int), ("head0", c_int), ("group", c_int),
+                ("max_chunks", c_int)]
+
+
+# The chunked form on the tensor cores: steps whose longest sequence brings at least this many tokens (0: never).
+MIN_CHUNKED_TOKENS = int(os.environ.get("KIDI_B200_LINEAR_CHUNKS", "32"))
+CHUNK = 64                              # tokens of a chunk (csrc/linear_chunks.cu)
+SCRATCH_FLOATS = 48 * 1024 * 1024       # the heads of a step are taken in groups that need at most this much scratch memory
+
 _library = None
+_chunk_libraries: Dict[tuple, ctypes.CDLL] = {}
+
+
+def chunk_library_request(dim: int, vdim: int):
+    """(name, sources, definitions) of the chunked kernels for one pair of head widths."""
+    return (f"linear_chunks_d{dim}_v{vdim}", ("linear_chunks.cu",), {"KIDI_LINEAR_DIM": dim, "KIDI_LINEAR_VDIM": vdim})
+
+
+def chunk_library(dim: int, vdim: int) -> ctypes.CDLL:
+    lib = _chunk_libraries.get((dim, vdim))
+    if lib is None:
+        lib = load_library(*chunk_library_request(dim, vdim))
+        lib.kidi_linear_chunks.argtypes = [c_void_p, c_void_p]
+        lib.kidi_linear_chunks.restype = c_int
+        lib.kidi_linear_chunks_scratch.argtypes = [c_int, c_int, c_int]
+        lib.kidi_linear_chunks_scratch.restype = c_longlong
+        _chunk_libraries[(dim, vdim)] = lib
+    return lib
+
+
+def chunks_fit(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, dim: int, vdim: int, longest: int) -> bool:
+    """Whether a step takes the chunked kernels: bfloat16 rows on 16-byte boundaries, head widths that are multiples of
+    16, and a sequence of enough tokens."""
+    return (0 < MIN_CHUNKED_TOKENS <= longest and q.dtype == torch.bfloat16 and dim % 16 == 0 and vdim % 16 == 0
+            and dim <= 256 and vdim <= 256
+            and all(x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 for x in (q, k, v)))
 
 
 def library():
@@ -38,12 +79,12 @@ def library():
 
 
 def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, *,
-                     heads: int, dim: int, vdim: int, tables, seqs: int, one_token: bool) -> torch.Tensor:
+                     heads: int, dim: int, vdim: int, tables, seqs: int, one_token: bool, longest: int) -> torch.Tensor:
     """S_t = decay_h S_(t-1) + k_t v_t^T and o_t = S_t^T q_t for every sequence's rows of the step, from and into `state`
     [slots + 1, heads, dim, vdim] (float32). q, k [rows, heads * dim] and v [rows, heads * vdim] are views of the step's
-    element type; decay float32 [heads]. `one_token`: every sequence of the step brings one token (decoding). Returns the
-    read-out, float32 [rows, heads * vdim]."""
-    if not one_token:
+    element type; decay float32 [heads]. `one_token`: every sequence of the step brings one token (decoding); `longest`:
+    the most tokens that a sequence brings. Returns the read-out, float32 [rows, heads * vdim]."""
+    if not one_token and not chunks_fit(q, k, v, dim, vdim, longest):
         return scalar_recurrence.scalar_recurrence(k, q, v, None, state, heads=heads, k_heads=heads, q_heads=heads, dim=dim,
                                                    vdim=vdim, tables=tables, seqs=seqs, decay=decay)
     ops._need_cuda(q, k, v, decay, state)
@@ -56,6 +97,22 @@ def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: t
     if state.dtype != torch.float32 or tuple(state.shape[1:]) != (heads, dim, vdim) or not state.is_contiguous():
         raise invalid_argument("linear attention: the state is float32 [slots, heads, dim, vdim]")
     out = torch.empty((rows, heads * vdim), dtype=torch.float32, device=v.device)
+    if not one_token:
+        lib = chunk_library(dim, vdim)
+        group = heads
+        while group > 1 and lib.kidi_linear_chunks_scratch(rows, seqs, group) > SCRATCH_FLOATS:
+            group = -(-group // 2)
+        scratch = torch.empty(lib.kidi_linear_chunks_scratch(rows, seqs, group), dtype=torch.float32, device=v.device)
+        for head0 in range(0, heads, group):
+            here = min(group, heads - head0)
+            sums = (rows // CHUNK + seqs + 1) * here * dim * vdim        # floats of the sums; the states follow them
+            args = LinearChunksArgs(
+                q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), decay.data_ptr(),
+                state.data_ptr(), out.data_ptr(), scratch.data_ptr(), scratch.data_ptr() + 4 * sums,
+                tables.row_seq.data_ptr(), tables.seq_slot.data_ptr(), tables.seq_row0.data_ptr(),
+                tables.seq_len.data_ptr(), seqs, heads, head0, here, -(-longest // CHUNK))
+            _check(lib.kidi_linear_chunks(ctypes.byref(args), ops._stream()), "linear_attention[chunks]", 3)
+        return out
     args = LinearStepArgs(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), decay.data_ptr(),
                           state.data_ptr(), out.data_ptr(), tables.row_seq.data_ptr(), tables.seq_slot.data_ptr(),
                           tables.seq_row0.data_ptr(), seqs, heads, dim, vdim)

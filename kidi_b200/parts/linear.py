@@ -50,6 +50,8 @@ class Linear:
         from ..kernels import skinny
         if silu_columns is not None:
             from ..kernels import linear_attention
+            if not isinstance(x, RowScaled) and skinny.fits(x, self.weight):      # few rows: SiLU in the epilogue
+                return skinny.gemm(x, self.weight, out_dtype or x.dtype, out=out, bias=self.bias, silu_columns=silu_columns)
             return linear_attention.silu_columns(self.forward(x, out_dtype, out), *silu_columns)
         weight, bias = self.weight, self.bias
         factors = None

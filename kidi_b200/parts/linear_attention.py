@@ -101,7 +101,8 @@ class LightningAttention(Part):
         qk, v = self.qk_width, self.out_width
         read = kernels.linear_attention(projected[:, :qk], projected[:, qk:2 * qk], projected[:, 2 * qk:2 * qk + v],
                                         self.decay, views[0], heads=self.heads, dim=self.dim, vdim=self.vdim,
-                                        tables=ctx.tables, seqs=ctx.plan.n_seqs, one_token=ctx.plan.is_decode)
+                                        tables=ctx.tables, seqs=ctx.plan.n_seqs, one_token=ctx.plan.is_decode,
+                                        longest=ctx.plan.max_new)
         if out is None:
             out = torch.empty((projected.shape[0], v), dtype=projected.dtype, device=projected.device)
         return kernels.normed_gate(read, self.norm, projected[:, 2 * qk + v:2 * qk + 2 * v], self.eps, self.out_scale, out)
