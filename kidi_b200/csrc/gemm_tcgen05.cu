@@ -149,6 +149,9 @@ struct Params {
     long long tail_first;  // the first tile of the tail
     int share, extra;      // of the tail's k-blocks a block takes `share`, the first `extra` blocks one more
     int staged;            // results leave through shared memory and TMA stores (bfloat16 y, 16-byte aligned rows)
+    const int* group_of_tile;   // [token tiles] or null: the tile's tokens take the weight rows from group * group_rows on
+                                // (a tile whose group is negative holds no tokens and is left out)
+    int group_rows;
 };
 
 // Tiles are numbered so that the blocks at work at one time share few weight tiles and few token
@@ -201,6 +204,15 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
         feature_tile = (int)(within / wide);
     };
 
+    // Weights in groups (the experts of a routed feed-forward): the first weight row of a tile's group, -1: no such tile.
+    auto group_begin = [&](long long tile) -> int {
+        if (!p.group_of_tile) return 0;
+        int token_tile, feature_tile;
+        locate(tile, token_tile, feature_tile);
+        const int group = p.group_of_tile[token_tile];
+        return group < 0 ? -1 : group * p.group_rows;
+    };
+
     if (threadIdx.x == 0) {
         for (int s = 0; s < STAGES; ++s) {
             mbarrier_init(&full_bar[s], 1);
@@ -231,7 +243,9 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
         auto load = [&](long long tile, int kb_first, int kb_count) {
             int token_tile, feature_tile;
             locate(tile, token_tile, feature_tile);
-            const int f0 = feature_tile * SPAN, t0 = token_tile * BN;
+            const int begin = group_begin(tile);
+            if (begin < 0) return;
+            const int f0 = begin + feature_tile * SPAN, t0 = token_tile * BN;
             for (int i = 0; i < kb_count; ++i, ++issued) {
                 const int s = issued % STAGES;
                 if (issued >= STAGES && !mbarrier_wait(&empty_bar[s], ((issued / STAGES) - 1) & 1, abort_flag)) {
@@ -296,7 +310,9 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
             ++done;
         };
         for (int round = 0; round < p.rounds && !*abort_flag; ++round)
-            if (blockIdx.x + (long long)round * gridDim.x < p.tail_first) multiply(p.k_blocks);
+            if (blockIdx.x + (long long)round * gridDim.x < p.tail_first &&
+                group_begin(blockIdx.x + (long long)round * gridDim.x) >= 0)
+                multiply(p.k_blocks);
         for (long long g = piece_begin; g < piece_end && !*abort_flag;) {
             const int kb_first = (int)(g % p.k_blocks);
             const int kb_count = (int)min((long long)(p.k_blocks - kb_first), piece_end - g);
@@ -483,7 +499,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
             }
         };
         for (int round = 0; round < p.rounds; ++round)
-            if (blockIdx.x + (long long)round * gridDim.x < p.tail_first)
+            if (blockIdx.x + (long long)round * gridDim.x < p.tail_first &&
+                group_begin(blockIdx.x + (long long)round * gridDim.x) >= 0)
                 finish(blockIdx.x + (long long)round * gridDim.x, -1, 0, p.k_blocks);
         for (long long g = piece_begin; g < piece_end;) {
             const long long tail_tile = g / p.k_blocks;
@@ -724,6 +741,8 @@ KIDI_API int kidi_gemm_tcgen05(const void* x, const void* w, void* y, int y_dtyp
     p.features = features;
     p.k_blocks = (K + BK - 1) / BK;
     p.token_tiles = (tokens + bn - 1) / bn;
+    p.group_of_tile = nullptr;
+    p.group_rows = 0;
     const long long tiles = (long long)((features + span - 1) / span) * p.token_tiles;
     const int blocks = kidi_gemm_tcgen05_blocks(tokens, features, K, gated, splits);
     if (tiles / blocks > 0x7fffffffLL) return KIDI_REFUSED_SIZE;
@@ -758,4 +777,44 @@ KIDI_API int kidi_gemm_tcgen05(const void* x, const void* w, void* y, int y_dtyp
     if (y_dtype == KIDI_BF16) return by_tokens<false, bf16>(bn, map_w, map_x, map_y, p, blocks, stream);
     if (y_dtype == KIDI_F32) return by_tokens<false, float>(bn, map_w, map_x, map_y, p, blocks, stream);
     return KIDI_REFUSED_DTYPE;
+}
+
+// The same for weights in groups (the experts of a routed feed-forward) and rows that are sorted by group: x [tokens, K] in
+// tiles of 128 rows, tile i's rows taking group group_of_tile[i] of w [groups, features (2 * features when gated), K]
+// (negative: the tile holds nothing; its rows of y are not written). Whole tiles only; no bias.
+KIDI_API int kidi_gemm_tcgen05_grouped(const void* x, const void* w, void* y, int tokens, int features, int K, long long ldx,
+                                       long long ldy, int gated, int groups, const int* group_of_tile, int* error,
+                                       cudaStream_t stream) {
+    constexpr int BN = 128;
+    if (tokens <= 0 || features <= 0) return 0;
+    const long long rows = (long long)groups * features * (gated ? 2 : 1);
+    if (K <= 0 || (K & 7) || (ldx & 7) || (ldy & 7) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15) || ((uintptr_t)y & 15) ||
+        groups <= 0 || rows > 0x7fffffffLL || tokens % BN || !group_of_tile || !error)
+        return KIDI_REFUSED_SIZE;
+    const int span = gated ? 64 : BM;
+    Params p;
+    memset(&p, 0, sizeof(p));
+    p.y = y;
+    p.error = error;
+    p.ldy = ldy;
+    p.tokens = tokens;
+    p.features = features;
+    p.k_blocks = (K + BK - 1) / BK;
+    p.token_tiles = tokens / BN;
+    p.tiles = (long long)((features + span - 1) / span) * p.token_tiles;
+    p.group_of_tile = group_of_tile;
+    p.group_rows = features * (gated ? 2 : 1);
+    p.staged = 1;
+    const long long sms = sm_count_of_current_device();
+    const int blocks = (int)(p.tiles < sms ? p.tiles : sms);
+    if (p.tiles / blocks > 0x7fffffffLL) return KIDI_REFUSED_SIZE;
+    p.rounds = (int)((p.tiles + blocks - 1) / blocks);
+    p.tail_first = p.tiles;
+    CUtensorMap map_w, map_x, map_y;
+    int status = make_map(&map_w, w, rows, K, K, gated ? 64 : BM);
+    if (!status) status = make_map(&map_x, x, tokens, K, ldx, BN);
+    if (!status) status = make_store_map(&map_y, y, tokens, features, ldy, span);
+    if (status) return status;
+    if (gated) return by_tokens<true, bf16>(BN, map_w, map_x, map_y, p, blocks, stream);
+    return by_tokens<false, bf16>(BN, map_w, map_x, map_y, p, blocks, stream);
 }

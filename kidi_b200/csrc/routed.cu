@@ -17,9 +17,9 @@
 //    (slot, feature) reads the chosen expert's two weight rows once and applies the activation; the
 //    input weight is applied to the two products in 32-bit (W (w h) = w (W h));
 //  * slots, down: a warp per (row, feature) sums its choices' products in the order of the choices;
-//  * gather / combine: for many rows the slots are sorted by expert on the host, their scaled input
-//    rows gathered, each expert's rows run through the ordinary products, and the results summed per
-//    row in the order of the choices.
+//  * group / gather / combine: for many rows the slots are grouped by expert, their scaled input rows
+//    gathered, each expert's rows run through a product over groups (or the ordinary products), and the
+//    results summed per row in the order of the choices.
 // Nothing here depends on which other rows share the step: a row's result is the same alone and in
 // a batch.
 #include "common.cuh"
@@ -292,6 +292,64 @@ KIDI_API int kidi_expert_slots(const void* x, int dtype, const void* gate_up, co
     KIDI_CASE(KIDI_BF16, bf16, KIDI_F32, float)
 #undef KIDI_CASE
     return KIDI_REFUSED_DTYPE;
+}
+
+// ------------------------------------------------------ grouping the slots by expert
+// Every expert's slots stand together, each expert's run beginning on a tile of TILE rows: place[slot] is a slot's row,
+// source[row] the row's slot (-1: padding), expert_of_tile[tile] the tile's expert (-1: the tile is not used). One block
+// counts, lays out and deals; the order of an expert's slots is whatever the atomics make it (a row's result does not
+// depend on its place). `rows` is what any choice fits in: slots + experts * (TILE - 1), rounded up to whole tiles.
+constexpr int GROUP_TILE = 128, GROUP_THREADS = 1024;
+__global__ void __launch_bounds__(GROUP_THREADS) group_slots_kernel(const int* __restrict__ chosen, int* __restrict__ source,
+                                                                    int* __restrict__ place, int* __restrict__ expert_of_tile,
+                                                                    int slots, int experts, int rows) {
+    __shared__ int count[1024], begin[1025], warp_total[32];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    count[threadIdx.x] = 0;
+    __syncthreads();
+    for (int i = threadIdx.x; i < slots; i += GROUP_THREADS) atomicAdd(&count[chosen[i]], 1);
+    __syncthreads();
+    // where the experts begin: an exclusive sum of their counts in whole tiles, an expert a thread
+    const int mine = threadIdx.x < experts ? (count[threadIdx.x] + GROUP_TILE - 1) / GROUP_TILE : 0;
+    int sum = mine;
+#pragma unroll
+    for (int step = 1; step < 32; step <<= 1) {
+        const int other = __shfl_up_sync(0xffffffffu, sum, step);
+        if (lane >= step) sum += other;
+    }
+    if (lane == 31) warp_total[warp] = sum;
+    __syncthreads();
+    int before = 0;
+    for (int w = 0; w < warp; ++w) before += warp_total[w];
+    begin[threadIdx.x] = before + sum - mine;
+    if (threadIdx.x == GROUP_THREADS - 1) begin[GROUP_THREADS] = before + sum;
+    __syncthreads();
+    for (int row = threadIdx.x; row < rows; row += GROUP_THREADS) source[row] = -1;
+    for (int tile = threadIdx.x + begin[GROUP_THREADS]; tile < rows / GROUP_TILE; tile += GROUP_THREADS) expert_of_tile[tile] = -1;
+    for (int e = warp; e < experts; e += 32)
+        for (int tile = begin[e] + lane; tile < begin[e + 1]; tile += 32) expert_of_tile[tile] = e;
+    count[threadIdx.x] = begin[threadIdx.x] * GROUP_TILE;          // the next free row of an expert
+    __syncthreads();
+    for (int i = threadIdx.x; i < slots; i += GROUP_THREADS) {
+        const int row = atomicAdd(&count[chosen[i]], 1);
+        place[i] = row;
+        source[row] = i;
+    }
+}
+
+// Rows that `slots` choices among `experts` experts may take.
+KIDI_API int kidi_group_slots_rows(int slots, int experts) {
+    const long long rows = ((long long)slots + (long long)experts * (GROUP_TILE - 1) + GROUP_TILE - 1) / GROUP_TILE * GROUP_TILE;
+    return rows > 0x7fffffffLL ? -1 : (int)rows;
+}
+
+KIDI_API int kidi_group_slots(const int* chosen, int* source, int* place, int* expert_of_tile, int slots, int experts,
+                              cudaStream_t stream) {
+    const int rows = kidi_group_slots_rows(slots, experts);
+    if (slots <= 0) return 0;
+    if (experts <= 0 || experts > 1024 || rows < 0) return KIDI_REFUSED_SIZE;
+    return kidi_launch(group_slots_kernel, 1, GROUP_THREADS, 0, stream, chosen, source, place, expert_of_tile, slots, experts,
+                       rows);
 }
 
 // ------------------------------------------------------ gather / combine

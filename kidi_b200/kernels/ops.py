@@ -106,10 +106,24 @@ class time_launches:
         global _timed
         _timed = self._outer
 
+    def restart(self) -> None:
+        """A new head start, after the host has waited for the device in the middle of what is timed."""
+        torch.cuda._sleep(int(self.head_start_ms * 1.5e6))
+        self.mark(self.WAITED)
+
+    WAITED = "(the host waited)"
+
     def spans(self) -> list:
         torch.cuda.synchronize()
         return [(name, 1e3 * before.elapsed_time(after))
-                for name, before, after in zip(self.names[1:], self.events[:-1], self.events[1:])]
+                for name, before, after in zip(self.names[1:], self.events[:-1], self.events[1:]) if name != self.WAITED]
+
+
+def host_waited() -> None:
+    """Called where the host has read something back in the middle of a step: the device stands idle then, which is no
+    time of the launches that follow (`time_launches`)."""
+    if _timed is not None and _timed.head_start_ms > 0:
+        _timed.restart()
 
 
 def _check(status: int, what: str, launches: int = 1) -> None:

@@ -26,7 +26,9 @@ def library():
                                           c_void_p]
         lib.kidi_combine_slots.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                            c_void_p, c_void_p]
-        for name in ("kidi_route", "kidi_expert_slots", "kidi_gather_slots", "kidi_combine_slots"):
+        lib.kidi_group_slots.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p]
+        lib.kidi_group_slots_rows.argtypes = [c_int, c_int]
+        for name in ("kidi_group_slots", "kidi_group_slots_rows", "kidi_route", "kidi_expert_slots", "kidi_gather_slots", "kidi_combine_slots"):
             getattr(lib, name).restype = c_int
         _library = lib
     return _library
@@ -85,6 +87,31 @@ def expert_slots(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, cho
                                        1 if gated else 0, addend.data_ptr() if addend is not None else 0,
                                        ops._stream()), "expert_slots", 2)
     return out
+
+
+def group_rows(slots: int, experts: int) -> int:
+    """Rows that any choice of `slots` (row, choice) pairs among `experts` experts fits in when every expert's run begins
+    on a tile of 128 rows (-1: too many)."""
+    return library().kidi_group_slots_rows(int(slots), int(experts))
+
+
+def group_slots(chosen: torch.Tensor, experts: int):
+    """Groups the (row, choice) pairs of `chosen` (int32, slot = row * top + choice) by expert on the device: (source,
+    place, expert_of_tile), int32: the slot of every grouped row (-1: padding), the row of every slot, the expert of every
+    tile of 128 rows (-1: not used). The order within an expert is not fixed."""
+    ops._need_cuda(chosen)
+    if chosen.dtype != torch.int32 or not chosen.is_contiguous():
+        raise invalid_argument("group_slots takes the router's choices")
+    slots = chosen.numel()
+    rows = group_rows(slots, experts)
+    if rows < 0:
+        raise invalid_argument("group_slots: too many slots")
+    source = torch.empty(rows, dtype=torch.int32, device=chosen.device)
+    place = torch.empty(slots, dtype=torch.int32, device=chosen.device)
+    tiles = torch.empty(rows // 128, dtype=torch.int32, device=chosen.device)
+    _check(library().kidi_group_slots(chosen.data_ptr(), source.data_ptr(), place.data_ptr(), tiles.data_ptr(), slots,
+                                      int(experts), ops._stream()), "group_slots")
+    return source, place, tiles
 
 
 def gather_slots(x: torch.Tensor, order: torch.Tensor, weight: torch.Tensor, top: int, weight_on_input: bool) -> torch.Tensor:

@@ -53,6 +53,9 @@ def _library():
                                           c_longlong, c_longlong, c_int, c_int, c_void_p, c_void_p, c_void_p,
                                           c_void_p, c_void_p]
         lib.kidi_gemm_tcgen05.restype = c_int
+        lib.kidi_gemm_tcgen05_grouped.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong,
+                                                  c_int, c_int, c_void_p, c_void_p, c_void_p]
+        lib.kidi_gemm_tcgen05_grouped.restype = c_int
         lib.kidi_gemm_tcgen05_token_tile.argtypes = [c_int]
         lib.kidi_gemm_tcgen05_token_tile.restype = c_int
         lib.kidi_gemm_tcgen05_workspace.argtypes = [c_int, c_int, c_int, c_int, c_int]
@@ -138,4 +141,28 @@ def gemm_silu_gate(x: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Te
     if out is None:
         out = torch.empty((x.shape[0], inter), dtype=torch.bfloat16, device=x.device)
     _run(x, weight, out, inter, True, splits)
+    return out
+
+
+GROUP_TILE = 128                        # rows of a tile of a grouped product
+
+
+def gemm_grouped(x: torch.Tensor, weight: torch.Tensor, group_of_tile: torch.Tensor, gated: bool) -> torch.Tensor:
+    """A product with weights in groups: rows 128 i .. 128 i + 127 of x [rows, K] take weight[group_of_tile[i]] of
+    weight [groups, features, K] (`gated`: [groups, 2 * features, K], gate rows first, and the result is silu(gate) * up);
+    bfloat16. Rows of tiles whose group (int32) is negative are not written."""
+    _need_cuda(x, weight, group_of_tile)
+    groups, height, K = weight.shape
+    rows = x.shape[0]
+    if (x.dtype != torch.bfloat16 or weight.dtype != torch.bfloat16 or x.dim() != 2 or x.shape[1] != K or x.stride(1) != 1
+            or not weight.is_contiguous() or rows % GROUP_TILE or (gated and height % 2)
+            or group_of_tile.dtype != torch.int32 or group_of_tile.shape != (rows // GROUP_TILE,)):
+        raise invalid_argument("gemm_grouped: the operands do not fit this kernel")
+    features = height // 2 if gated else height
+    out = torch.empty((rows, features), dtype=torch.bfloat16, device=x.device)
+    _, _, error = _device_state(x.device)
+    _check(_library().kidi_gemm_tcgen05_grouped(
+        _ptr(x), _ptr(weight), _ptr(out), rows, features, K, x.stride(0), out.stride(0), 1 if gated else 0, groups,
+        _ptr(group_of_tile), _ptr(error), _stream()),
+        "gemm_silu_gate[tcgen05, groups]" if gated else "gemm_tcgen05[groups]")
     return out

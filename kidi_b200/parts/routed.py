@@ -22,21 +22,24 @@ of the same form and that width, under `<prefix><shared_name><gate|up|down>`, th
 result is added with weight 1.
 
 Steps of few rows, steps inside a captured decode graph, and every step of the 32-bit engine read the
-chosen experts' weights through the choice on the device (no host round trip). Prompts of the bfloat16
-engine sort the (row, choice) pairs by expert on the host and gather the rows; every expert's rows, up to twice
-the mean count, are then padded to one count and run through two batched products of the vendor library, and
-what an expert has beyond that (or everything, where the widths are no multiples of 8) through the ordinary
-products, with one activation kernel for all of them.
+chosen experts' weights through the choice on the device. Prompts of the bfloat16 engine group the (row,
+choice) pairs by expert on the device, gather the rows and run them through two products over groups of this
+package's tcgen05 kernel (a gated expert's SiLU gate in the first one's epilogue): no host round trip either.
+Where the widths are no multiples of 8, or the experts so many that the groups' padding would more than
+triple the rows, the pairs are sorted by expert on the host instead; every expert's rows, up to twice the mean count,
+are then padded to one count and run through two batched products of the vendor library, and what an expert has
+beyond that (or everything, for odd widths) through the ordinary products, with one activation kernel for all of them.
 """
 from __future__ import annotations
 
+import os
 from typing import List, Optional
 
 import numpy as np
 import torch
 
 from ..errors import invalid_argument, unsupported
-from ..kernels import ops, routed, skinny
+from ..kernels import ops, routed, skinny, tcgen05
 from .base import Part, plain_rows
 from .linear import Linear
 from .registry import register_part
@@ -45,6 +48,8 @@ from .spec import ParamSpec
 # Up to this many (row, choice) pairs a step reads the experts through the choice; above, a bfloat16 prompt
 # sorts them by expert.
 SLOT_PATH_MAX = 128
+# Prompts group the pairs on the device and take the products over groups (0: sorted on the host, batched products).
+GROUPED = os.environ.get("KIDI_B200_GROUPED_EXPERTS", "1") == "1"
 
 
 @register_part("feed_forward", "routed_experts")
@@ -154,9 +159,19 @@ class RoutedExperts(Part):
         if x.dtype == torch.float32 or self.gate_up.dtype == torch.float32 or ctx.plan.is_decode \
                 or slots <= SLOT_PATH_MAX:
             return routed.expert_slots(x, self.gate_up, self.down, chosen, weight, self.weight_on_input, self.gated, addend)
+        if GROUPED and self.hidden % 8 == 0 and self.inter % 8 == 0 \
+                and 0 < routed.group_rows(slots, self.experts) <= 4 * slots:
+            source, place, tiles = routed.group_slots(chosen, self.experts)
+            gathered = routed.gather_slots(x, source, weight, self.top, self.weight_on_input)
+            mid = tcgen05.gemm_grouped(gathered, self.gate_up, tiles, self.gated)
+            if not self.gated:
+                mid = self._activate(mid)
+            result = tcgen05.gemm_grouped(mid, self.down, tiles, False)
+            return routed.combine_slots(result, place, weight, rows, self.top, self.weight_on_input, addend)
         # Many rows: (row, choice) pairs in the order of their experts (a stable sort, so a row's place among
         # its expert's rows follows its place in the step), one host round trip for the counts.
         picked = chosen.reshape(-1).cpu().numpy()
+        ops.host_waited()
         order = np.argsort(picked, kind="stable").astype(np.int32)
         counts = np.bincount(picked, minlength=self.experts)
         # Every expert's first `cap` rows stand in one padded batch [experts, cap] (two batched products of the

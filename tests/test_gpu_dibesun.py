@@ -795,3 +795,59 @@ def test_the_trace_runner_replays_a_model_folder(tmp_path, dtype, record_propert
           torch.cat([torch.stack([want["a"][0], want["b"][0], want["b"][69], want["c"][5], want["c"][128]]),
                      torch.stack([want["b"][71], want["c"][130]]), want["b"][74:75], want["d"][[0, 45, 89]]]),
           dtype, record_property, "prompts together, decoded together, the last one alone, on reused pages", slack=2.0)
+
+
+# ------------------------------------------------------------------ routed experts on prompts
+@pytest.mark.parametrize("gated", [True, False])
+@pytest.mark.parametrize("rows,experts,top,hidden,inter", [(200, 6, 2, 64, 24), (700, 16, 3, 136, 72), (300, 5, 5, 256, 200),
+                                                           (129, 40, 1, 48, 136)])
+def test_products_over_groups_of_experts(rows, experts, top, hidden, inter, gated, monkeypatch):
+    """Slots grouped on the device (an expert that nobody chooses, one that most choose), the product over groups with and
+    without the gate, and the routed feed-forward as a whole against its form with the slots sorted on the host."""
+    from kidi_b200.kernels import ops, routed, tcgen05
+    generator = torch.Generator().manual_seed(rows)
+    bias = torch.randn(experts, generator=generator)
+    bias[experts // 2] += 6.0
+    bias[0] -= 60.0 if top < experts else 0.0
+    chosen = torch.topk(torch.randn(rows, experts, generator=generator) + bias, top).indices.int()
+    source, place, tiles = (t.cpu() for t in routed.group_slots(chosen.cuda(), experts))
+    flat = chosen.reshape(-1)
+    assert torch.equal(source[place.long()], torch.arange(rows * top, dtype=torch.int32))      # every slot has its row
+    assert int((source >= 0).sum()) == rows * top and source.numel() % 128 == 0
+    assert torch.equal(tiles[place.long() // 128], flat)                                      # in a tile of its expert
+    used = (torch.bincount(flat, minlength=experts) + 127) // 128
+    assert torch.equal(torch.bincount(tiles[tiles >= 0], minlength=experts), used) and int((tiles < 0).sum()) == tiles.numel() - int(used.sum())
+    x = torch.randn(source.numel(), hidden, generator=generator).bfloat16()
+    weight = (torch.randn(experts, (2 if gated else 1) * inter, hidden, generator=generator) / hidden ** 0.5).bfloat16()
+    got = tcgen05.gemm_grouped(x.cuda(), weight.cuda(), tiles.cuda(), gated).double().cpu()
+    for tile, expert in enumerate(tiles.tolist()):
+        if expert < 0:
+            continue
+        y = x[128 * tile:128 * tile + 128].double() @ weight[expert].double().t()
+        want = plain_dibesun.silu(y[:, :inter]) * y[:, inter:] if gated else y
+        assert torch.allclose(got[128 * tile:128 * tile + 128], want, atol=2e-2, rtol=2e-2)
+
+
+def test_routed_prompts_grouped_on_the_device_and_sorted_on_the_host(monkeypatch, record_property):
+    """The same prompt through both forms of the routed feed-forward: each names its kernels, the logits agree within
+    bfloat16 rounding, and a request in a batch is what it is alone."""
+    from kidi_b200 import StepBatch
+    from kidi_b200.kernels import ops
+    from kidi_b200.parts import routed as part
+    config = configs.single(configs.layer(configs.attention(2, 1, 16, 16, 0.3, softcap=20.0), configs.linear(4, 16, 16),
+                                          configs.routed(6, 2, 40, shared=24)), width=64, groups=2)
+    engine, tensors = make(config, "bfloat16", seed=3)
+    a, b = prompt(config, 300, 1), prompt(config, 120, 2)
+    found = {}
+    for grouped in (True, False):
+        monkeypatch.setattr(part, "GROUPED", grouped)
+        with ops.record_launches() as names:
+            found[grouped] = in_steps(engine, a, [300])
+        assert ("group_slots" in names and "gemm_silu_gate[tcgen05, groups]" in names) == grouped
+        assert ("library_bmm" in names) == (not grouped)
+        close(found[grouped], follow(engine, 0, "bfloat16", config, tensors, a, None), "bfloat16", record_property, str(grouped))
+    monkeypatch.setattr(part, "GROUPED", True)
+    slots = [engine.acquire(), engine.acquire()]
+    both = engine.step(StepBatch(slots, [b, a], [[], list(range(300))])).double().cpu()
+    assert float((both - found[True]).abs().max()) < 0.05 * float(both.abs().max())
+    engine.check_device_errors()

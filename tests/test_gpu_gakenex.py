@@ -87,11 +87,13 @@ def test_the_small_kernels(dtype):
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("experts,top,rows,inter", [(6, 2, 5, 24), (3, 3, 300, 24), (16, 1, 200, 24), (9, 4, 64, 24),
                                                      (4, 2, 150, 20)])
-def test_routed_experts_alone(dtype, experts, top, rows, inter):
+def test_routed_experts_alone(dtype, experts, top, rows, inter, monkeypatch):
     """The router's choice (sigmoid scores, the largest first, the weight on the expert's input) and the experts,
-    through the choice on the device and, for many rows in bfloat16, sorted by expert (padded to one count and
-    batched, or expert by expert where the widths are no multiples of 8): against the plain function."""
+    through the choice on the device and, for many rows in bfloat16, grouped by expert on the device (products over
+    groups) or sorted on the host (padded to one count and batched, or expert by expert where the widths are no multiples of 8): against the plain function."""
     from types import SimpleNamespace
+    from kidi_b200.kernels import routed
+    from kidi_b200.parts import routed as routed_part
     from kidi_b200.parts.base import BuildEnv
     from kidi_b200.parts.routed import RoutedExperts
     from kidi_b200.parts.spec import PartSpec
@@ -115,13 +117,18 @@ def test_routed_experts_alone(dtype, experts, top, rows, inter):
     tolerance = 2e-5 if dtype == torch.float32 else 0.08
     scale = float(want.abs().max())
     from kidi_b200.kernels import ops
-    for decode in (False, True):                          # the sorted path (many bfloat16 rows), and through the choice
+    # many bfloat16 rows grouped on the device or sorted on the host, and through the choice
+    for decode, grouped in ((False, True), (False, False), (True, True)):
+        monkeypatch.setattr(routed_part, "GROUPED", grouped)
         ctx = SimpleNamespace(plan=SimpleNamespace(is_decode=decode))
         with ops.record_launches() as names:
             found = part.forward(h.cuda(), ctx).double().cpu()
         if dtype == torch.bfloat16 and not decode and rows * top > 128:
+            over_groups = sum(name in ("gemm_silu_gate[tcgen05, groups]", "gemm_tcgen05[groups]") for name in names)
+            device = grouped and inter % 8 == 0 and routed.group_rows(rows * top, experts) <= 4 * rows * top
+            assert over_groups == (2 if device else 0)
             batched = names.count("library_bmm")          # unless one expert has far more rows than the others
-            assert batched == 0 if inter % 8 else batched == 2 if top == experts else batched in (0, 2)
+            assert batched == 0 if inter % 8 or device else batched == 2 if top == experts else batched in (0, 2)
             assert "expert_slots" not in names
         else:
             assert "expert_slots" in names
