@@ -324,23 +324,13 @@ __global__ void __launch_bounds__(WIDE_THREADS) wide_norm_store_kernel(WideNormA
     constexpr int WARPS = WIDE_THREADS / 32;
     constexpr int HELD = V == 8 ? 2 : 1;          // pieces of q that stay in registers between the two passes
     const int row = blockIdx.x;
-    const int seq = a.row_seq[row];
-    if (seq < 0) return;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     T* q = (T*)a.qkv + row * a.ld;
     const int q_width = a.heads * a.head_dim, k_width = a.kv_heads * a.head_dim, v_width = a.kv_heads * a.value_dim;
     T* k = q + q_width;
     const T* v = k + k_width;
-    const int position = a.row_pos[row];
-    bool keep = a.k_cache != nullptr;
-    if (keep && a.cache.ring_pages)   // a ring keeps the last ring_tokens tokens of the step only
-        keep = position >= a.seq_start[seq] + a.seq_len[seq] - (a.cache.ring_pages << a.cache.page_shift);
-    const long long offset = keep ? cache_row_offset(a.cache, a.seq_slot[seq], position, 0) : 0;
-    const long long key_stride = (long long)a.head_dim << a.cache.page_shift;      // from one head's row to the next head's
-    const long long value_stride = (long long)a.value_dim << a.cache.page_shift;
-    T* k_cached = (T*)a.k_cache + offset;
-    T* v_cached = (T*)a.v_cache + offset / a.head_dim * a.value_dim;
-
+    // (The row's entries are asked for together with its sequence and position; a padding row's are there to be read.)
+    const int seq = a.row_seq[row], position = a.row_pos[row];
     float held[HELD][V], held_k[V], piece[V];
     float q_square = 0.f, k_square = 0.f;
     int index = 0;
@@ -364,6 +354,15 @@ __global__ void __launch_bounds__(WIDE_THREADS) wide_norm_store_kernel(WideNormA
 #pragma unroll
         for (int i = 0; i < V; ++i) k_square = fmaf(piece[i], piece[i], k_square);
     }
+    if (seq < 0) return;                              // the same for the whole block
+    bool keep = a.k_cache != nullptr;
+    if (keep && a.cache.ring_pages)   // a ring keeps the last ring_tokens tokens of the step only
+        keep = position >= a.seq_start[seq] + a.seq_len[seq] - (a.cache.ring_pages << a.cache.page_shift);
+    const long long offset = keep ? cache_row_offset(a.cache, a.seq_slot[seq], position, 0) : 0;
+    const long long key_stride = (long long)a.head_dim << a.cache.page_shift;      // from one head's row to the next head's
+    const long long value_stride = (long long)a.value_dim << a.cache.page_shift;
+    T* k_cached = (T*)a.k_cache + offset;
+    T* v_cached = (T*)a.v_cache + offset / a.head_dim * a.value_dim;
     if (keep)
         for (int c = threadIdx.x * V; c < v_width; c += WIDE_THREADS * V) {
             const int head = c / a.value_dim;

@@ -88,8 +88,8 @@ __device__ __forceinline__ void tma_store_2d(const CUtensorMap* map, const void*
                  :
                  : "l"((unsigned long long)map), "r"(smem_u32(smem)), "r"(x), "r"(y)
                  : "memory");
-    asm volatile("cp.async.bulk.commit_group;" ::: "memory");
 }
+__device__ __forceinline__ void tma_store_commit() { asm volatile("cp.async.bulk.commit_group;" ::: "memory"); }
 
 // Shared memory descriptor of a K-major tile with the 128-byte swizzle: rows are 128
 // bytes apart, groups of eight rows 1024 bytes apart (the stride byte offset), version 1.
@@ -134,6 +134,31 @@ __device__ __forceinline__ void tmem_load_16(unsigned address, float (&v)[16]) {
     for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(r[i]);
 }
 
+// 16 or 32 columns at once: every load is issued before the wait.
+template <int N>
+__device__ __forceinline__ void tmem_load(unsigned address, float (&v)[N]) {
+    if constexpr (N == 16) {
+        tmem_load_16(address, v);
+    } else {
+        static_assert(N == 32, "16 or 32 columns");
+        asm volatile(
+            "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
+            "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,"
+            "%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];\n\t"
+            "tcgen05.wait::ld.sync.aligned;"
+            : "=f"(v[0]), "=f"(v[1]), "=f"(v[2]), "=f"(v[3]), "=f"(v[4]), "=f"(v[5]), "=f"(v[6]), "=f"(v[7]), "=f"(v[8]),
+              "=f"(v[9]), "=f"(v[10]), "=f"(v[11]), "=f"(v[12]), "=f"(v[13]), "=f"(v[14]), "=f"(v[15]), "=f"(v[16]),
+              "=f"(v[17]), "=f"(v[18]), "=f"(v[19]), "=f"(v[20]), "=f"(v[21]), "=f"(v[22]), "=f"(v[23]), "=f"(v[24]),
+              "=f"(v[25]), "=f"(v[26]), "=f"(v[27]), "=f"(v[28]), "=f"(v[29]), "=f"(v[30]), "=f"(v[31])
+            : "r"(address)
+            : "memory");
+    }
+}
+
+// Token columns that the epilogue takes at a time: its barriers and copies are paid for once a piece. (Small tiles have
+// two blocks an SM and no shared memory to spare.)
+template <int BN> constexpr int epilogue_columns() { return BN >= 128 ? 32 : 16; }
+
 struct Params {
     void* y;               // [tokens, ldy]
     float* workspace;      // [2 * blocks][BM][BN] partial tiles
@@ -175,12 +200,13 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
     constexpr int SPAN = GATED ? 64 : BM;                  // output features per tile
     extern __shared__ unsigned char raw[];
     unsigned char* tiles = (unsigned char*)(((uintptr_t)raw + 1023) & ~(uintptr_t)1023);
-    // The gated epilogue passes the up rows of a 16-column chunk between warps (64 x 17 floats).
+    // The gated epilogue passes the up rows of a chunk of columns between warps (64 x (columns + 1) floats).
     float* exchange = reinterpret_cast<float*>(tiles + (size_t)STAGES * STAGE_BYTES);
-    // Results on their way out (p.staged): two buffers of 16 tokens x SPAN features, which TMA stores
-    // write to y in whole lines (a thread holds one feature of 16 tokens: stored directly, every
+    // Results on their way out (p.staged): two buffers of CW tokens x SPAN features, which TMA stores
+    // write to y in whole lines (a thread holds one feature of CW tokens: stored directly, every
     // token's 32 features of a warp would be a 64-byte piece of its own).
-    bf16* staging = reinterpret_cast<bf16*>(tiles + (size_t)STAGES * STAGE_BYTES + 64 * 17 * sizeof(float));
+    constexpr int CW = epilogue_columns<BN>();
+    bf16* staging = reinterpret_cast<bf16*>(tiles + (size_t)STAGES * STAGE_BYTES + 64 * (CW + 1) * sizeof(float));
     __shared__ unsigned long long full_bar[STAGES], empty_bar[STAGES], ready_bar[2], drained_bar[2];
     __shared__ unsigned tmem_base_slot;
     __shared__ int gave_up, is_last;
@@ -374,44 +400,48 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
             {
                 TY* y = (TY*)p.y;
 #pragma unroll 1
-                for (int c = 0; c < BN; c += 16) {
-                    float v[16];
-                    if (ok) tmem_load_16(accumulator + c, v);
+                for (int c = 0; c < BN; c += CW) {
+                    float v[CW];
+                    if (ok) tmem_load<CW>(accumulator + c, v);
                     else
 #pragma unroll
-                        for (int i = 0; i < 16; ++i) v[i] = 0.f;
+                        for (int i = 0; i < CW; ++i) v[i] = 0.f;
                     bool mine = f0 + row < p.features;    // this thread has results of this chunk
                     if (GATED) {
                         // Rows 64..127 hold the up projection of the features in rows 0..63.
                         if (row >= 64)
 #pragma unroll
-                            for (int i = 0; i < 16; ++i) exchange[(row - 64) * 17 + i] = v[i];
+                            for (int i = 0; i < CW; ++i) exchange[(row - 64) * (CW + 1) + i] = v[i];
                         asm volatile("bar.sync 1, 128;" ::: "memory");
                         mine = mine && row < 64;
                         if (row < 64)
 #pragma unroll
-                            for (int i = 0; i < 16; ++i) v[i] = v[i] / (1.0f + expf(-v[i])) * exchange[row * 17 + i];
+                            for (int i = 0; i < CW; ++i) v[i] = v[i] / (1.0f + expf(-v[i])) * exchange[row * (CW + 1) + i];
                         asm volatile("bar.sync 1, 128;" ::: "memory");
                     } else if (p.bias && mine) {
                         const float shift = p.bias[f0 + row];
 #pragma unroll
-                        for (int i = 0; i < 16; ++i) v[i] += shift;
+                        for (int i = 0; i < CW; ++i) v[i] += shift;
                     }
                     if (sizeof(TY) == 2 && p.staged) {
-                        bf16* out = staging + (staged_chunks & 1) * (16 * SPAN);
+                        bf16* out = staging + (staged_chunks & 1) * (CW * SPAN);
                         // The copy that read this buffer two chunks ago must be through with it.
                         if (threadIdx.x == 64 && staged_chunks >= 2) asm volatile("cp.async.bulk.wait_group.read 1;" ::: "memory");
                         asm volatile("bar.sync 1, 128;" ::: "memory");
                         if (row < SPAN)
 #pragma unroll
-                            for (int i = 0; i < 16; ++i) out[i * SPAN + row] = __float2bfloat16_rn(v[i]);
+                            for (int i = 0; i < CW; ++i) out[i * SPAN + row] = __float2bfloat16_rn(v[i]);
                         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");   // the copy reads what these threads wrote
                         asm volatile("bar.sync 1, 128;" ::: "memory");
-                        if (threadIdx.x == 64) tma_store_2d(&map_y, out, f0, t0 + c);
+                        if (threadIdx.x == 64) {
+                            tma_store_2d(&map_y, out, f0, t0 + c);
+                            if (CW > 16) tma_store_2d(&map_y, out + 16 * SPAN, f0, t0 + c + 16);
+                            tma_store_commit();
+                        }
                         ++staged_chunks;
                     } else if (mine) {
 #pragma unroll
-                        for (int i = 0; i < 16; ++i) {
+                        for (int i = 0; i < CW; ++i) {
                             const int token = t0 + c + i;
                             if (token < p.tokens) y[token * p.ldy + f0 + row] = from_float<TY>(v[i]);
                         }
@@ -580,7 +610,9 @@ int make_store_map(CUtensorMap* map, void* base, long long tokens, long long fea
 // buffer and two buffers of results on their way out.
 template <int BN, int STAGES>
 constexpr size_t shared_bytes() {
-    return (size_t)STAGES * (BM * BK * 2 + BN * BK * 2) + 1024 + 64 * 17 * sizeof(float) + 2 * 16 * BM * sizeof(bf16);
+    constexpr int columns = epilogue_columns<BN>();
+    return (size_t)STAGES * (BM * BK * 2 + BN * BK * 2) + 1024 + 64 * (columns + 1) * sizeof(float) +
+           2 * columns * BM * sizeof(bf16);
 }
 
 // Sets the kernel up (once) and returns how many of its blocks the device promises to hold on an SM

@@ -270,18 +270,18 @@ __global__ void __launch_bounds__(128) expert_down_kernel(const T* __restrict__ 
 
 KIDI_API int kidi_expert_slots(const void* x, int dtype, const void* gate_up, const void* down, int weight_dtype,
                                const int* chosen, const float* weight, void* mid, void* out, int rows, int top,
-                               int hidden, int inter, int weight_on_input, int gated, const void* addend,
-                               cudaStream_t stream) {
+                               int hidden, int inter, int weight_on_input, int gated, const void* addend, int parts,
+                               cudaStream_t stream) {       // parts: 1 the gate and up products, 2 the down product, 3 both
     if (rows <= 0) return 0;
     const long long slots = (long long)rows * top;
     const long long first = slots * inter, second = (long long)rows * hidden;
     if (first >= (1LL << 33) || second >= (1LL << 33)) return KIDI_REFUSED_SIZE;
 #define KIDI_CASE(D, T, W, TW)                                                                                     \
     if (dtype == D && weight_dtype == W) {                                                                         \
-        int status = kidi_launch(expert_gate_up_kernel<T, TW>, (unsigned)((first + 3) / 4), 128, 0, stream,       \
-                                 (const T*)x, (const TW*)gate_up, chosen, weight, (T*)mid, slots, top, hidden,     \
-                                 inter, weight_on_input, gated);                                                   \
-        if (status) return status;                                                                                 \
+        int status = parts & 1 ? kidi_launch(expert_gate_up_kernel<T, TW>, (unsigned)((first + 3) / 4), 128, 0,    \
+                                             stream, (const T*)x, (const TW*)gate_up, chosen, weight, (T*)mid,     \
+                                             slots, top, hidden, inter, weight_on_input, gated) : 0;               \
+        if (status || !(parts & 2)) return status;                                                                 \
         return kidi_launch(expert_down_kernel<T, TW>, (unsigned)((second + 3) / 4), 128, 0, stream, (const T*)mid, \
                            (const TW*)down, chosen, weight, (T*)out, (long long)rows, top, hidden, inter,          \
                            weight_on_input, (const T*)addend);                                                     \

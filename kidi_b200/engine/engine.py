@@ -45,6 +45,7 @@ class StepContext:
                  device: torch.device, workspaces: Optional[Dict[str, torch.Tensor]] = None):
         self.plan, self.tables, self.cache, self.dtype, self.device = plan, tables, cache, dtype, device
         self._workspaces = workspaces if workspaces is not None else {}
+        self._side_stream = None
 
     def workspace(self, name: str, count: int, zero: bool = False) -> torch.Tensor:
         """Scratch memory of at least `count` 32-bit elements that kernels of one step may
@@ -56,6 +57,29 @@ class StepContext:
             held = make(max(count, 1), dtype=torch.float32, device=self.device)
             self._workspaces[name] = held
         return held
+
+    def beside(self, work):
+        """Queues `work()` beside whatever the caller queues before it calls the returned function, which waits for the
+        work (on the device) and returns its result. In a captured step the two become branches of the graph that may run
+        at the same time; elsewhere `work()` is queued at once, in the caller's order. The work must not use scratch
+        memory (`workspace`) that the caller's own launches use meanwhile, and what it writes for the caller is allocated
+        before the call or returned."""
+        if self.device.type != "cuda" or not torch.cuda.is_current_stream_capturing():
+            result = work()
+            return lambda: result
+        main = torch.cuda.current_stream(self.device)
+        if self._side_stream is None:
+            self._side_stream = torch.cuda.Stream(device=self.device)
+        side = self._side_stream
+        side.wait_stream(main)
+        with torch.cuda.stream(side):
+            result = work()
+
+        def join():
+            main.wait_stream(side)
+            return result
+
+        return join
 
 
 class Engine:

@@ -21,7 +21,7 @@ def library():
         lib.kidi_route.argtypes = [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                                    c_int, c_int, c_int, c_float, c_void_p, c_void_p]
         lib.kidi_expert_slots.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
-                                          c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p]
+                                          c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p]
         lib.kidi_gather_slots.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                           c_void_p]
         lib.kidi_combine_slots.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
@@ -66,11 +66,12 @@ def route(x: torch.Tensor, router: torch.Tensor, top: int, renormalise: bool, sc
 
 def expert_slots(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, chosen: torch.Tensor,
                  weight: torch.Tensor, weight_on_input: bool, gated: bool = True,
-                 addend: Optional[torch.Tensor] = None) -> torch.Tensor:
+                 addend=None) -> torch.Tensor:
     """Every row through its chosen experts, the experts' weights read through the choice: x [rows, hidden],
     gate_up [experts, 2 * inter, hidden] (without a gate: the up rows only, [experts, inter, hidden], and the
     exact gelu as activation), down [experts, hidden, inter] -> [rows, hidden]. `addend` [rows, hidden], if given, is
-    added to the result (in 32-bit, before it is rounded)."""
+    added to the result (in 32-bit, before it is rounded); it may be a function that returns it (or None), which is
+    called between the two kernels."""
     ops._need_cuda(x, gate_up, down, chosen, weight)
     rows, hidden = x.shape
     experts, first_rows, _ = gate_up.shape
@@ -78,14 +79,27 @@ def expert_slots(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, cho
     if (not x.is_contiguous() or gate_up.shape != (experts, (2 if gated else 1) * inter, hidden) or down.shape != (experts, hidden, inter)
             or not gate_up.is_contiguous() or not down.is_contiguous() or gate_up.dtype != down.dtype):
         raise invalid_argument("expert_slots: the experts' weights do not fit the rows")
-    _check_addend(addend, x, rows, hidden)
+    later = addend if callable(addend) else None
+    if later is None:
+        _check_addend(addend, x, rows, hidden)
     mid = torch.empty((rows * top, inter), dtype=x.dtype, device=x.device)
     out = torch.empty((rows, hidden), dtype=x.dtype, device=x.device)
-    _check(library().kidi_expert_slots(x.data_ptr(), dtype_code(x.dtype), gate_up.data_ptr(), down.data_ptr(),
-                                       dtype_code(gate_up.dtype), chosen.data_ptr(), weight.data_ptr(), mid.data_ptr(),
-                                       out.data_ptr(), rows, top, hidden, inter, 1 if weight_on_input else 0,
-                                       1 if gated else 0, addend.data_ptr() if addend is not None else 0,
-                                       ops._stream()), "expert_slots", 2)
+
+    def launch(parts: int, what: str, launches: int) -> None:
+        _check(library().kidi_expert_slots(
+            x.data_ptr(), dtype_code(x.dtype), gate_up.data_ptr(), down.data_ptr(), dtype_code(gate_up.dtype),
+            chosen.data_ptr(), weight.data_ptr(), mid.data_ptr(), out.data_ptr(), rows, top, hidden, inter,
+            1 if weight_on_input else 0, 1 if gated else 0, addend.data_ptr() if addend is not None else 0, parts,
+            ops._stream()), what, launches)
+
+    if later is None:
+        launch(3, "expert_slots", 2)
+        return out
+    addend = None
+    launch(1, "expert_slots[gate and up]", 1)
+    addend = later()
+    _check_addend(addend, x, rows, hidden)
+    launch(2, "expert_slots", 1)
     return out
 
 

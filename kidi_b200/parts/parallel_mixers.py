@@ -122,6 +122,8 @@ class ParallelMixers(Part):
         make = torch.empty if self.out.in_features == self._out_used else torch.zeros
         mixed = make((x.shape[0], self.out.in_features), dtype=projected.dtype, device=projected.device)
         middle = self.left.out_width
+        joined = ctx.beside(lambda: self.right.mix(projected[:, self._left_columns:], ctx, right_views, owns_cache,
+                                                   out=mixed[:, middle:self._out_used]))
         self.left.mix(projected[:, :self._left_columns], ctx, left_views, owns_cache, out=mixed[:, :middle])
-        self.right.mix(projected[:, self._left_columns:], ctx, right_views, owns_cache, out=mixed[:, middle:self._out_used])
+        joined()
         return self.out.forward(mixed)

@@ -140,25 +140,30 @@ class RoutedExperts(Part):
 
     def forward(self, x, ctx) -> torch.Tensor:
         x = plain_rows(x)
-        shared = None
+        # The shared expert runs beside the routed ones; its result joins their sum in the kernel that forms it (32-bit).
+        beside = getattr(ctx, "beside", None)
+        shared = lambda: None
         if self._shared is not None:
-            # The shared expert's result joins the routed sum in the kernel that forms it (a 32-bit sum).
-            up, down = self._shared
-            if not self.gated and up.bias is None and skinny.fits(x, up.weight):
-                mid = skinny.gemm(x, up.weight, x.dtype, activation="gelu")       # few rows: the gelu in the epilogue
-            else:
-                mid = self._activate(up.forward(x))
-            shared = down.forward(mid)
+            shared = beside(lambda: self._forward_shared(x)) if beside is not None else lambda: self._forward_shared(x)
         return self._forward_routed(x, ctx, shared)
 
-    def _forward_routed(self, x, ctx, addend=None) -> torch.Tensor:
+    def _forward_shared(self, x) -> torch.Tensor:
+        up, down = self._shared
+        if skinny.fits(x, up.weight) and up.bias is None:            # few rows: the activation in the epilogue
+            mid = skinny.gemm_silu_gate(x, up.weight) if self.gated else skinny.gemm(x, up.weight, x.dtype, activation="gelu")
+        else:
+            mid = self._activate(up.forward(x))
+        return down.forward(mid)
+
+    def _forward_routed(self, x, ctx, shared=lambda: None) -> torch.Tensor:
+        """`shared()`: the shared expert's result (or None), asked for where the routed sum is formed."""
         rows = x.shape[0]
         chosen, weight = routed.route(x, self.router, self.top, self.renormalise, self.score, self.groups,
                                       self.keep_groups, self.renormalise_eps, self.router_bias)
         slots = rows * self.top
         if x.dtype == torch.float32 or self.gate_up.dtype == torch.float32 or ctx.plan.is_decode \
                 or slots <= SLOT_PATH_MAX:
-            return routed.expert_slots(x, self.gate_up, self.down, chosen, weight, self.weight_on_input, self.gated, addend)
+            return routed.expert_slots(x, self.gate_up, self.down, chosen, weight, self.weight_on_input, self.gated, shared)
         if GROUPED and self.hidden % 8 == 0 and self.inter % 8 == 0 \
                 and 0 < routed.group_rows(slots, self.experts) <= 4 * slots:
             source, place, tiles = routed.group_slots(chosen, self.experts)
@@ -167,7 +172,7 @@ class RoutedExperts(Part):
             if not self.gated:
                 mid = self._activate(mid)
             result = tcgen05.gemm_grouped(mid, self.down, tiles, False)
-            return routed.combine_slots(result, place, weight, rows, self.top, self.weight_on_input, addend)
+            return routed.combine_slots(result, place, weight, rows, self.top, self.weight_on_input, shared())
         # Many rows: (row, choice) pairs in the order of their experts (a stable sort, so a row's place among
         # its expert's rows follows its place in the step), one host round trip for the counts.
         picked = chosen.reshape(-1).cpu().numpy()
@@ -214,4 +219,4 @@ class RoutedExperts(Part):
             ops.note("library_bmm")
         for index, begin, end in spans:
             self._down[index].forward(mid[begin:end], out=result[begin:end])
-        return routed.combine_slots(result, tables[total:], weight, rows, self.top, self.weight_on_input, addend)
+        return routed.combine_slots(result, tables[total:], weight, rows, self.top, self.weight_on_input, shared())
