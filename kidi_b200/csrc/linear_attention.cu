@@ -131,6 +131,12 @@ normed_gate_kernel(const float* __restrict__ read, const float* __restrict__ wei
         out[row * ldo + c] = from_float<T>(source[c] * inv * weight[c] / (1.0f + expf(-to_float(gate[row * ldg + c]))));
 }
 
+// y sigmoid(z) with the fast exponential and division (a few units in the last place; for results that are rounded to
+// bfloat16; far below zero the exponential is held at 2^115, so that the quotient stays a number).
+__device__ __forceinline__ float sigmoid_times(float y, float z) {
+    return __fdividef(y, 1.0f + __expf(fminf(-z, 80.f)));
+}
+
 // The same for bfloat16 results of widths that are multiples of 4, from 16-byte pieces of the read-out; up to HELD
 // pieces a thread stay in registers between the two passes.
 __global__ void __launch_bounds__(THREADS)
@@ -169,10 +175,10 @@ normed_gate_bf16x4_kernel(const float* __restrict__ read, const float* __restric
         const float2 g0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
         const float2 g1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
         uint2 packed;
-        *reinterpret_cast<__nv_bfloat162*>(&packed.x) = __floats2bfloat162_rn(x.x * inv * w.x / (1.0f + expf(-g0.x)),
-                                                                             x.y * inv * w.y / (1.0f + expf(-g0.y)));
-        *reinterpret_cast<__nv_bfloat162*>(&packed.y) = __floats2bfloat162_rn(x.z * inv * w.z / (1.0f + expf(-g1.x)),
-                                                                             x.w * inv * w.w / (1.0f + expf(-g1.y)));
+        *reinterpret_cast<__nv_bfloat162*>(&packed.x) = __floats2bfloat162_rn(sigmoid_times(x.x * inv * w.x, g0.x),
+                                                                             sigmoid_times(x.y * inv * w.y, g0.y));
+        *reinterpret_cast<__nv_bfloat162*>(&packed.y) = __floats2bfloat162_rn(sigmoid_times(x.z * inv * w.z, g1.x),
+                                                                             sigmoid_times(x.w * inv * w.w, g1.y));
         *reinterpret_cast<uint2*>(out + row * ldo + 4 * c) = packed;
     };
 #pragma unroll
@@ -204,7 +210,7 @@ __global__ void silu_columns_bf16x8_kernel(bf16* __restrict__ x, long long ld, l
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
         const float2 z = __bfloat1622float2(pairs[i]);
-        pairs[i] = __floats2bfloat162_rn(z.x / (1.0f + expf(-z.x)), z.y / (1.0f + expf(-z.y)));
+        pairs[i] = __floats2bfloat162_rn(sigmoid_times(z.x, z.x), sigmoid_times(z.y, z.y));
     }
     *reinterpret_cast<uint4*>(at) = raw;
 }
