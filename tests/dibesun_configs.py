@@ -71,7 +71,7 @@ ODD = model(71, 50, 3e-6, 1, 1.0, [
 # twelve heads (decoding's wider form), linear attention with heads that the chunked form takes and with heads that it
 # does not; chunks whose edge falls inside a tile
 WIDE = model(211, 240, 1e-5, 5, 4.0, [
-    layer(attention(8, 2, 64, 64, 0.15, chunk=150, softcap=25.0), linear(4, 64, 32), dense(256)),
+    layer(attention(8, 2, 64, 64, 0.15, chunk=150, softcap=25.0), linear(4, 32, 64), dense(256)),
     layer(attention(2, 1, 128, 128, 0.1, chunk=200, softcap=30.0), linear(2, 128, 128), routed(8, 2, 64, shared=96)),
     layer(attention(3, 1, 48, 48, 0.15, chunk=100), linear(3, 48, 16), routed(6, 2, 72)),
     layer(attention(12, 1, 32, 32, 0.2, softcap=15.0), linear(2, 24, 40), dense(128)),
