@@ -47,9 +47,23 @@ constexpr float LOG2E = 1.4426950408889634f;
 #define KIDI_SIGMOID_WEIGHTS 0
 #endif
 constexpr bool SIGMOID = KIDI_SIGMOID_WEIGHTS != 0;
+// With -DKIDI_TIED_VALUES=1 a value is its key before the key norm: the cache and the step hold that row once, a tile is
+// loaded once and serves both products, and a key's factor 1 / sqrt(mean square + eps) is formed here from the tile and
+// multiplied into its scores (the norm's weight rides in q).
+#ifndef KIDI_TIED_VALUES
+#define KIDI_TIED_VALUES 0
+#endif
+constexpr bool TIED = KIDI_TIED_VALUES != 0;
+// With -DKIDI_DISTANCE_BIAS=1 a number per head and distance is added to a score.
+#ifndef KIDI_DISTANCE_BIAS
+#define KIDI_DISTANCE_BIAS 0
+#endif
+constexpr bool BIASED = KIDI_DISTANCE_BIAS != 0;
+static_assert(!SIGMOID || (!TIED && !BIASED), "sigmoid weights come with plain keys and values");
+constexpr int KV_TILES = TIED ? 2 : 4;       // two buffers of keys and, unless they are the keys, two of values
 // Shared memory of a decode block: the query rows and two key and two value tiles (or, once
 // they are consumed, the warps' partial results).
-constexpr size_t DECODE_TILES = (size_t)(16 + 4 * TILE) * PITCH * sizeof(bf16);
+constexpr size_t DECODE_TILES = (size_t)(16 + KV_TILES * TILE) * PITCH * sizeof(bf16);
 constexpr size_t DECODE_MERGE =
     (size_t)16 * PITCH * sizeof(bf16) + (size_t)(4 * 16 * D + 4 * 16 * 2 + 2 * 8 * 32 + 8) * sizeof(float);
 constexpr size_t DECODE_SHARED = DECODE_TILES > DECODE_MERGE ? DECODE_TILES : DECODE_MERGE;
@@ -59,14 +73,15 @@ constexpr size_t DECODE_SHARED = DECODE_TILES > DECODE_MERGE ? DECODE_TILES : DE
 // fit an SM.
 constexpr int NARROW_RECV_OUT_FLOATS = 8 * D + 8 * 4;    // [splits][share], share rounded up to four
 constexpr int NARROW_RECV_FLOATS = NARROW_RECV_OUT_FLOATS + 8 * 8 * 2;
-constexpr size_t NARROW_TILES = (size_t)(8 + 4 * TILE) * PITCH * sizeof(bf16);
+constexpr size_t NARROW_TILES = (size_t)(8 + KV_TILES * TILE) * PITCH * sizeof(bf16);
 constexpr size_t NARROW_MERGE =
     (size_t)8 * PITCH * sizeof(bf16) + (size_t)(4 * 8 * (D + 4) + 4 * 8 * 2 + 2 * 8 * 32 + 8) * sizeof(float);
 constexpr size_t NARROW_TILE_BYTES = ((NARROW_TILES > NARROW_MERGE ? NARROW_TILES : NARROW_MERGE) + 15) / 16 * 16;
 constexpr size_t NARROW_SHARED = NARROW_TILE_BYTES + NARROW_RECV_FLOATS * sizeof(float);
-// The swizzled form: four unpadded tiles on a 1024-byte boundary, then the query rows (the
+// The swizzled form: four unpadded tiles (three, where values are keys) on a 1024-byte boundary, then the query rows (the
 // warps' partial results reuse the tiles).
-constexpr size_t SWIZZLED_TILE_BYTES = ((size_t)(4 * TILE * D + 8 * PITCH) * sizeof(bf16) + 15) / 16 * 16;
+constexpr int SWIZZLED_TILES = TIED ? 3 : 4;
+constexpr size_t SWIZZLED_TILE_BYTES = ((size_t)(SWIZZLED_TILES * TILE * D + 8 * PITCH) * sizeof(bf16) + 15) / 16 * 16;
 constexpr size_t SWIZZLED_SHARED = 1024 + SWIZZLED_TILE_BYTES + NARROW_RECV_FLOATS * sizeof(float);
 // The ring form of it: three tiles.
 constexpr size_t RING_TILE_BYTES = ((size_t)(3 * TILE * D + 8 * PITCH) * sizeof(bf16) + 15) / 16 * 16;
@@ -151,6 +166,10 @@ struct Args {
     const float* weight_bias; // [heads], sigmoid build only: a key's weight is sigmoid(score + weight_bias[h])
     int chunk;                // > 0: only keys of the query's own run of `chunk` positions are seen
     float out_scale;          // the result is multiplied by it
+    const float* distance_bias;   // [heads, bias_stride], biased build only: entry min(p - u, bias_last) of head h's row is
+    int bias_stride, bias_last;   // added to a score (in base-2 exponent units)
+    const bf16* element_gate;     // [rows, ld_element_gate] or null: the result is multiplied by sigmoid of it
+    long long ld_element_gate;
 };
 
 // How a raw dot product becomes a score in base-2 exponent units: times scale * log2(e), or, bounded,
@@ -188,6 +207,17 @@ __device__ __forceinline__ float finish_factor(const Args& a, long long row, int
     float factor = total > 0.f ? 1.0f / total : 0.f;
     if (a.gate) factor *= 1.0f / (1.0f + expf(-__bfloat162float(a.gate[row * a.ldg + head])));
     return factor * a.out_scale;
+}
+
+// sigmoid of the gate of element c of a (row, head); 1 without a gate.
+__device__ __forceinline__ float gate_of(const Args& a, long long row, int head, int c) {
+    if (!a.element_gate) return 1.f;
+    return 1.0f / (1.0f + expf(-__bfloat162float(a.element_gate[row * a.ld_element_gate + (long long)head * D + c])));
+}
+
+// What is added to head h's score of a key `back` positions before the query, in base-2 exponent units.
+__device__ __forceinline__ float bias_of(const Args& a, int head, int back) {
+    return __ldg(a.distance_bias + (long long)head * a.bias_stride + max(0, min(back, a.bias_last)));
 }
 
 // sigmoid(score + bias) from both in base-2 exponent units; a score of -infinity (a key that is not seen) gives 0.
@@ -295,9 +325,10 @@ __device__ __forceinline__ void softmax_and_weighted_sum(float (&s)[NT][4], floa
 
 // Scores of one warp: 16 query rows (A from q_tile rows [q_row, q_row+16)) against
 // NT*8 keys starting at `first_key` of k_tile, as scores in base-2 exponent units.
+// `factor` (tied values): the factors of the tile's 64 keys.
 template <int NT>
 __device__ __forceinline__ void scores(float (&s)[NT][4], const bf16* q_tile, int q_row, const bf16* k_tile,
-                                       int first_key, const ScoreShape& shape, int lane) {
+                                       int first_key, const ScoreShape& shape, int lane, const float* factor) {
 #pragma unroll
     for (int j = 0; j < NT; ++j)
 #pragma unroll
@@ -316,9 +347,34 @@ __device__ __forceinline__ void scores(float (&s)[NT][4], const bf16* q_tile, in
         }
     }
 #pragma unroll
-    for (int j = 0; j < NT; ++j)
+    for (int j = 0; j < NT; ++j) {
+        if constexpr (TIED) {
+            const float f0 = factor[first_key + j * 8 + 2 * (lane & 3)], f1 = factor[first_key + j * 8 + 2 * (lane & 3) + 1];
+            s[j][0] *= f0; s[j][1] *= f1; s[j][2] *= f0; s[j][3] *= f1;
+        }
 #pragma unroll
         for (int i = 0; i < 4; ++i) s[j][i] = shaped(s[j][i], shape);
+    }
+}
+
+// The factors of `count` keys of a tile from `first` on, two neighbouring lanes a key (count = half the lanes that take part,
+// `lane` counted among them).
+__device__ __forceinline__ void key_factors(float* factor, const bf16* k_tile, int first, int lane, float eps) {
+    const int key = first + (lane >> 1);
+    float square = 0.f;
+#pragma unroll 4
+    for (int c = (lane & 1) * 8; c < D; c += 16) {
+        const uint4 raw = *reinterpret_cast<const uint4*>(k_tile + key * PITCH + c);
+        const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float2 two = __bfloat1622float2(pairs[i]);
+            square = fmaf(two.x, two.x, square);
+            square = fmaf(two.y, two.y, square);
+        }
+    }
+    square += __shfl_xor_sync(0xffffffffu, square, 1);
+    if (!(lane & 1)) factor[key] = 1.0f / sqrtf(square / (float)D + eps);
 }
 
 // ------------------------------------------------------------------- prefill
@@ -326,7 +382,8 @@ __global__ void __launch_bounds__(THREADS) attention_prefill_kernel(Args a) {
     extern __shared__ __align__(16) unsigned char raw[];
     bf16* q_tile = reinterpret_cast<bf16*>(raw);            // [64][PITCH]
     bf16* k_tiles = q_tile + TILE * PITCH;                  // [2][64][PITCH]
-    bf16* v_tiles = k_tiles + 2 * TILE * PITCH;             // [2][64][PITCH]
+    bf16* v_tiles = TIED ? k_tiles : k_tiles + 2 * TILE * PITCH;     // [2][64][PITCH]
+    __shared__ float key_factor[TIED ? TILE : 1];
     const int seq = blockIdx.y, head = blockIdx.z;
     const int q0 = blockIdx.x * TILE;
     const int count = a.seq_len[seq];
@@ -349,7 +406,7 @@ __global__ void __launch_bounds__(THREADS) attention_prefill_kernel(Args a) {
         copy_async_16(q_tile + r * PITCH + c * 8, source, valid);
     }
     load_tile(k_tiles, a.k_step, a.ldkv, row0, step_from, a.k_cache, a.cache, slot, kv_head, tile_low, last);
-    load_tile(v_tiles, a.v_step, a.ldkv, row0, step_from, a.v_cache, a.cache, slot, kv_head, tile_low, last);
+    if (!TIED) load_tile(v_tiles, a.v_step, a.ldkv, row0, step_from, a.v_cache, a.cache, slot, kv_head, tile_low, last);
     copy_async_commit();
 
     float best[2] = {-INFINITY, -INFINITY}, denom[2] = {0.f, 0.f};
@@ -369,19 +426,24 @@ __global__ void __launch_bounds__(THREADS) attention_prefill_kernel(Args a) {
         if (tile < tile_high) {
             load_tile(k_tiles + (buffer ^ 1) * TILE * PITCH, a.k_step, a.ldkv, row0, step_from, a.k_cache, a.cache,
                       slot, kv_head, tile + 1, last);
-            load_tile(v_tiles + (buffer ^ 1) * TILE * PITCH, a.v_step, a.ldkv, row0, step_from, a.v_cache, a.cache,
-                      slot, kv_head, tile + 1, last);
+            if (!TIED)
+                load_tile(v_tiles + (buffer ^ 1) * TILE * PITCH, a.v_step, a.ldkv, row0, step_from, a.v_cache, a.cache,
+                          slot, kv_head, tile + 1, last);
             copy_async_commit();
             copy_async_wait<1>();
         } else {
             copy_async_wait<0>();
         }
         __syncthreads();
+        if constexpr (TIED) {
+            key_factors(key_factor, k_tiles + buffer * TILE * PITCH, 0, threadIdx.x, a.eps);
+            __syncthreads();
+        }
         // Warps whose 16 query rows do not exist, or lie wholly before this tile, have nothing to do.
         const bool active = warp * 16 < q_rows && start + q0 + warp * 16 + 15 >= tile * TILE;
         if (active) {
             float s[8][4];
-            scores<8>(s, q_tile, warp * 16, k_tiles + buffer * TILE * PITCH, 0, shape, lane);
+            scores<8>(s, q_tile, warp * 16, k_tiles + buffer * TILE * PITCH, 0, shape, lane, key_factor);
 #pragma unroll
             for (int j = 0; j < 8; ++j)
 #pragma unroll
@@ -389,6 +451,7 @@ __global__ void __launch_bounds__(THREADS) attention_prefill_kernel(Args a) {
                     const int u = tile * TILE + j * 8 + 2 * t + (i & 1);
                     const int p = position0 + (i >> 1) * 8;
                     const bool visible = u <= p && u >= first_seen[i >> 1];
+                    if constexpr (BIASED) s[j][i] += bias_of(a, head, p - u);
                     if (!visible) s[j][i] = -INFINITY;
                 }
             softmax_and_weighted_sum<8>(s, best, denom, o, v_tiles + buffer * TILE * PITCH, 0, lane, bias);
@@ -404,7 +467,9 @@ __global__ void __launch_bounds__(THREADS) attention_prefill_kernel(Args a) {
         bf16* out = a.out + (long long)(row0 + q0 + r) * a.ldo + (long long)head * D;
 #pragma unroll
         for (int n = 0; n < D / 8; ++n) {
-            const unsigned pair = pack_bf16(o[n][half * 2] * inverse, o[n][half * 2 + 1] * inverse);
+            const int c = n * 8 + 2 * t;
+            const unsigned pair = pack_bf16(o[n][half * 2] * inverse * gate_of(a, row0 + q0 + r, head, c),
+                                            o[n][half * 2 + 1] * inverse * gate_of(a, row0 + q0 + r, head, c + 1));
             *reinterpret_cast<unsigned*>(out + n * 8 + 2 * t) = pair;
         }
     }
@@ -417,7 +482,8 @@ __global__ void __launch_bounds__(THREADS) attention_decode_kernel(Args a) {
     extern __shared__ __align__(16) unsigned char raw[];
     bf16* q_tile = reinterpret_cast<bf16*>(raw);            // [16][PITCH]
     bf16* k_tiles = q_tile + 16 * PITCH;                    // [2][64][PITCH]
-    bf16* v_tiles = k_tiles + 2 * TILE * PITCH;             // [2][64][PITCH]
+    bf16* v_tiles = TIED ? k_tiles : k_tiles + 2 * TILE * PITCH;     // [2][64][PITCH]
+    __shared__ float key_factor[TIED ? TILE : 1];
     const int split = blockIdx.x, kv_head = blockIdx.y, row = blockIdx.z;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, t = lane & 3;
@@ -463,7 +529,7 @@ __global__ void __launch_bounds__(THREADS) attention_decode_kernel(Args a) {
             copy_async_16(q_tile + r * PITCH + c * 8, source, valid);
         }
         load_tile(k_tiles, nullptr, 0, 0, 0x7fffffff, a.k_cache, a.cache, slot, kv_head, tile_first, position);
-        load_tile(v_tiles, nullptr, 0, 0, 0x7fffffff, a.v_cache, a.cache, slot, kv_head, tile_first, position);
+        if (!TIED) load_tile(v_tiles, nullptr, 0, 0, 0x7fffffff, a.v_cache, a.cache, slot, kv_head, tile_first, position);
         copy_async_commit();
         const ScoreShape shape = score_shape(a.scale, a.softcap);
         float bias[2] = {0.f, 0.f};
@@ -476,8 +542,9 @@ __global__ void __launch_bounds__(THREADS) attention_decode_kernel(Args a) {
             if (index + 1 < tiles) {
                 load_tile(k_tiles + (buffer ^ 1) * TILE * PITCH, nullptr, 0, 0, 0x7fffffff, a.k_cache, a.cache, slot,
                           kv_head, tile + 1, position);
-                load_tile(v_tiles + (buffer ^ 1) * TILE * PITCH, nullptr, 0, 0, 0x7fffffff, a.v_cache, a.cache, slot,
-                          kv_head, tile + 1, position);
+                if (!TIED)
+                    load_tile(v_tiles + (buffer ^ 1) * TILE * PITCH, nullptr, 0, 0, 0x7fffffff, a.v_cache, a.cache, slot,
+                              kv_head, tile + 1, position);
                 copy_async_commit();
                 copy_async_wait<1>();
             } else {
@@ -487,12 +554,20 @@ __global__ void __launch_bounds__(THREADS) attention_decode_kernel(Args a) {
             const int first_key = warp * 16;
             if (tile * TILE + first_key <= position && tile * TILE + first_key + 15 >= low) {
                 float s[2][4];
-                scores<2>(s, q_tile, 0, k_tiles + buffer * TILE * PITCH, first_key, shape, lane);
+                if constexpr (TIED) {                       // a warp's own sixteen keys
+                    key_factors(key_factor, k_tiles + buffer * TILE * PITCH, first_key, lane, a.eps);
+                    __syncwarp();
+                }
+                scores<2>(s, q_tile, 0, k_tiles + buffer * TILE * PITCH, first_key, shape, lane, key_factor);
 #pragma unroll
                 for (int j = 0; j < 2; ++j)
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
                         const int u = tile * TILE + first_key + j * 8 + 2 * t + (i & 1);
+                        if constexpr (BIASED) {
+                            const int r = g + (i >> 1) * 8;
+                            if (r < group) s[j][i] += bias_of(a, head0 + r, position - u);
+                        }
                         if (u > position || u < low) s[j][i] = -INFINITY;
                     }
                 softmax_and_weighted_sum<2>(s, best, denom, o, v_tiles + buffer * TILE * PITCH, first_key, lane, bias);
@@ -535,7 +610,7 @@ __global__ void __launch_bounds__(THREADS) attention_decode_kernel(Args a) {
         const int head = head0 + r;
         if (a.splits == 1) {
             a.out[(long long)row * a.ldo + (long long)head * D + c] =
-                from_float<bf16>(value * finish_factor(a, row, head, top, total));
+                from_float<bf16>(value * finish_factor(a, row, head, top, total) * gate_of(a, row, head, c));
         } else {
             const long long where = ((long long)row * a.heads + head) * a.splits + split;
             merged_out[where * D + c] = value;
@@ -582,11 +657,11 @@ __device__ __forceinline__ void issue_tile(bf16* k_tile, bf16* v_tile, const bf1
     const int r = threadIdx.x & 63;
     if (threadIdx.x == 0)
         asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(smem_address(bar)),
-                     "r"((unsigned)(rows_valid * D * 2 * 2))
+                     "r"((unsigned)(rows_valid * D * 2 * (TIED ? 1 : 2)))
                      : "memory");
     if (r < rows_valid) {
         if (threadIdx.x < 64) bulk_copy_row(k_tile + r * PITCH, k_cache + page + (long long)r * D, D * 2, bar);
-        else bulk_copy_row(v_tile + r * PITCH, v_cache + page + (long long)r * D, D * 2, bar);
+        else if (!TIED) bulk_copy_row(v_tile + r * PITCH, v_cache + page + (long long)r * D, D * 2, bar);
     }
 }
 
@@ -693,14 +768,16 @@ __global__ void __launch_bounds__(THREADS, 4)     // four blocks an SM where sha
 attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
                                Args a) {
     constexpr bool SWIZZLED = FORM != 0, RING = FORM == 2;
-    constexpr int BUFFERS = RING ? 3 : 4;
+    static_assert(!TIED || !RING, "tiles that serve both products come in one form");
+    constexpr int BUFFERS = RING ? 3 : SWIZZLED ? SWIZZLED_TILES : KV_TILES;
+    constexpr int STAGES = TIED && SWIZZLED ? 3 : 2;       // tiles of keys (and as many of values, unless they are the keys)
     extern __shared__ __align__(16) unsigned char raw_unaligned[];
     // Swizzled tiles want 1024-byte boundaries and come first; the query rows follow them.
     unsigned char* raw = SWIZZLED ? (unsigned char*)(((uintptr_t)raw_unaligned + 1023) & ~(uintptr_t)1023) : raw_unaligned;
     constexpr int TP = SWIZZLED ? D : PITCH;               // elements between rows of a key or value tile
     bf16* q_tile = reinterpret_cast<bf16*>(raw) + (SWIZZLED ? BUFFERS * TILE * TP : 0);   // [8][PITCH]
-    bf16* k_tiles = SWIZZLED ? reinterpret_cast<bf16*>(raw) : q_tile + 8 * PITCH;   // [2][64][TP]
-    bf16* v_tiles = k_tiles + 2 * TILE * TP;                                        // [2][64][TP]
+    bf16* k_tiles = SWIZZLED ? reinterpret_cast<bf16*>(raw) : q_tile + 8 * PITCH;   // [STAGES][64][TP]
+    bf16* v_tiles = TIED ? k_tiles : k_tiles + 2 * TILE * TP;                       // [STAGES][64][TP]
     // Where the eight elements from column `col` (a multiple of 8) of row `r` of a tile lie.
     auto tile_at = [](bf16* tile, int r, int col) -> bf16* {
         if (SWIZZLED) return tile + (col >> 6) * (TILE * 64) + r * 64 + ((((col & 63) >> 3) ^ (r & 7)) << 3);
@@ -774,13 +851,14 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
                     const int page_row = page_row_of(tile - tile_first);
                     asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(
                                      smem_address(&tile_bar[buffer])),
-                                 "r"((unsigned)(2 * TILE * D * 2))
+                                 "r"((unsigned)((TIED ? 1 : 2) * TILE * D * 2))
                                  : "memory");
                     for (int span = 0; span < D / 64; ++span) {
                         tensor_copy_2d(k_tiles + buffer * TILE * TP + span * TILE * 64, &k_map, &tile_bar[buffer],
                                        span * 64, page_row);
-                        tensor_copy_2d(v_tiles + buffer * TILE * TP + span * TILE * 64, &v_map, &tile_bar[buffer],
-                                       span * 64, page_row);
+                        if (!TIED)
+                            tensor_copy_2d(v_tiles + buffer * TILE * TP + span * TILE * 64, &v_map, &tile_bar[buffer],
+                                           span * 64, page_row);
                     }
                 }
             } else {
@@ -812,9 +890,10 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
         } else {
             issue(tile_first, 0);
             if (tiles > 1) issue(tile_first + 1, 1);
+            if (STAGES > 2 && tiles > 2) issue(tile_first + 2, 2);
         }
         uint4 new_raw = make_uint4(0u, 0u, 0u, 0u);          // warp 0: the new key row's chunk, warp 1: the value's
-        if (has_new && warp < 2 && lane < CHUNKS)
+        if (has_new && warp < (TIED ? 1 : 2) && lane < CHUNKS)
             new_raw = *reinterpret_cast<const uint4*>((warp == 0 ? a.k_step : a.v_step) + (long long)row * a.ldkv +
                                                       (long long)kv_head * D + lane * 8);
         // Value rows that no copy writes must be finite (their weights are exact zeros; a
@@ -845,14 +924,21 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
                 if (2 * t + i < group) bias[i] = a.weight_bias[head0 + 2 * t + i] * LOG2E;
         }
         for (int index = 0; index < tiles; ++index) {
-            const int tile = tile_first + index, buffer = index & 1;
+            const int tile = tile_first + index, buffer = index % STAGES;
             const int k_load = 2 * index, v_load = 2 * index + 1;                 // the ring's loads of this tile
             const bool newest = has_new && tile == new_tile;
+            float distance[4] = {0.f, 0.f, 0.f, 0.f};      // what is added to the scores (asked for before the tile is waited for)
+            if constexpr (BIASED) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+                    distance[i] = bias_of(a, head0 + min(2 * t + (i & 1), group - 1),
+                                          position - (tile * TILE + warp * 16 + g + (i >> 1) * 8));
+            }
             if (RING) {
                 wait_tile(&tile_bar[k_load % 3], (k_load / 3) & 1);
                 if (newest) wait_tile(&tile_bar[v_load % 3], (v_load / 3) & 1);   // the step's value goes into the value tile
             } else {
-                wait_tile(&tile_bar[buffer], (index >> 1) & 1);
+                wait_tile(&tile_bar[buffer], (index / STAGES) & 1);
             }
             if (index == 0) {
                 copy_async_wait<0>();
@@ -895,9 +981,9 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
             bf16* v_tile = RING ? k_tiles + (v_load % 3) * TILE * TP : v_tiles + buffer * TILE * TP;
             if (newest) {                                   // the step's own key (warp 0) and value (warp 1)
                 const int r_new = position - tile * TILE;
-                if (warp < 2) {
+                if (warp < (TIED ? 1 : 2)) {
                     uint4 fresh = new_raw;
-                    if (warp == 0 && (a.fuse & 1)) {
+                    if (!TIED && warp == 0 && (a.fuse & 1)) {
                         const int half_lanes = a.rotary_dim / 16;
                         const int partner_lane = (lane * 8 < a.rotary_dim / 2 ? lane + half_lanes : lane - half_lanes) & 31;
                         const float square = head_square_sum(new_raw);
@@ -924,18 +1010,39 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
             unsigned p0 = 0u, p1 = 0u;
             if (active) {
                 float s[4] = {0.f, 0.f, 0.f, 0.f};          // keys g (0,1) and g+8 (2,3) x heads 2t, 2t+1
+                // Tied values: the keys' sums of squares are the diagonal of K K^T, for which a key fragment is both
+                // operands: keys 0..7 of the warp against themselves, and keys 8..15.
+                float low_square[4] = {0.f, 0.f, 0.f, 0.f}, high_square[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
                 for (int kk = 0; kk < D / 16; ++kk) {
                     unsigned k_frag[4];
                     ldmatrix_x4(k_frag, tile_at(k_tile, first_key + within + (matrix & 1) * 8, kk * 16 + (matrix >> 1) * 8));
                     mma_bf16(s, k_frag, q_frag[kk][0], q_frag[kk][1]);
+                    if constexpr (TIED) {
+                        mma_bf16(low_square, k_frag, k_frag[0], k_frag[2]);
+                        mma_bf16(high_square, k_frag, k_frag[1], k_frag[3]);
+                    }
                 }
                 const int u0 = tile * TILE + first_key + g, u1 = u0 + 8;
                 const bool see0 = u0 <= position && u0 >= low, see1 = u1 <= position && u1 >= low;
-                s[0] = see0 ? shaped(s[0], shape) : -INFINITY;
-                s[1] = see0 ? shaped(s[1], shape) : -INFINITY;
-                s[2] = see1 ? shaped(s[2], shape) : -INFINITY;
-                s[3] = see1 ? shaped(s[3], shape) : -INFINITY;
+                if constexpr (TIED) {
+                    // row g of the products is key g (entries 0, 1) or g + 8 (2, 3); lane (g, g / 2) holds its diagonal entry
+                    const int holder = (lane & ~3) | (g >> 1);
+                    const float square0 = __shfl_sync(0xffffffffu, (g & 1) ? low_square[1] : low_square[0], holder);
+                    const float square1 = __shfl_sync(0xffffffffu, (g & 1) ? high_square[3] : high_square[2], holder);
+                    const float factor0 = 1.0f / sqrtf(square0 / (float)D + a.eps), factor1 = 1.0f / sqrtf(square1 / (float)D + a.eps);
+                    s[0] *= factor0; s[1] *= factor0; s[2] *= factor1; s[3] *= factor1;
+                }
+#pragma unroll
+                for (int i = 0; i < 4; ++i) s[i] = shaped(s[i], shape);
+                if constexpr (BIASED) {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) s[i] += distance[i];
+                }
+                s[0] = see0 ? s[0] : -INFINITY;
+                s[1] = see0 ? s[1] : -INFINITY;
+                s[2] = see1 ? s[2] : -INFINITY;
+                s[3] = see1 ? s[3] : -INFINITY;
                 if constexpr (SIGMOID) {
 #pragma unroll
                     for (int i = 0; i < 4; ++i) s[i] = sigmoid_log2(s[i], bias[i & 1]);
@@ -986,8 +1093,8 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
             __syncthreads();
             if (RING) {
                 if (k_load + 4 < 2 * tiles) issue_load(k_load + 4);   // the values are read: the keys of the tile after next
-            } else if (index + 2 < tiles) {
-                issue(tile + 2, buffer);                     // the buffer that was just read takes the tile after next
+            } else if (index + STAGES < tiles) {
+                issue(tile + STAGES, buffer);                // the buffer that was just read takes the tile after next
             }
         }
     }
@@ -1077,8 +1184,8 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
         if (a.splits == 1) {
             const float scale = finish_factor(a, row, head, merge_weight[32 + r * 2], merge_weight[32 + r * 2 + 1]);
             bf16* out = a.out + (long long)row * a.ldo + (long long)head * D + c;
-            *reinterpret_cast<__nv_bfloat162*>(out) = __floats2bfloat162_rn(value.x * scale, value.y * scale);
-            *reinterpret_cast<__nv_bfloat162*>(out + 2) = __floats2bfloat162_rn(value.z * scale, value.w * scale);
+            *reinterpret_cast<__nv_bfloat162*>(out) = __floats2bfloat162_rn(value.x * scale * gate_of(a, row, head, c), value.y * scale * gate_of(a, row, head, c + 1));
+            *reinterpret_cast<__nv_bfloat162*>(out + 2) = __floats2bfloat162_rn(value.z * scale * gate_of(a, row, head, c + 2), value.w * scale * gate_of(a, row, head, c + 3));
         } else if (CLUSTER) {
             const int target = item / share;
             *reinterpret_cast<float4*>(cluster.map_shared_rank(recv_out, target) + split * share + item - target * share) = value;
@@ -1113,9 +1220,10 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
                 value.x += part.x * factor; value.y += part.y * factor; value.z += part.z * factor; value.w += part.w * factor;
             }
             const float scale = finish_factor(a, row, head0 + r, top, total);
-            bf16* out = a.out + (long long)row * a.ldo + (long long)(head0 + r) * D + c;
-            *reinterpret_cast<__nv_bfloat162*>(out) = __floats2bfloat162_rn(value.x * scale, value.y * scale);
-            *reinterpret_cast<__nv_bfloat162*>(out + 2) = __floats2bfloat162_rn(value.z * scale, value.w * scale);
+            const int head = head0 + r;
+            bf16* out = a.out + (long long)row * a.ldo + (long long)head * D + c;
+            *reinterpret_cast<__nv_bfloat162*>(out) = __floats2bfloat162_rn(value.x * scale * gate_of(a, row, head, c), value.y * scale * gate_of(a, row, head, c + 1));
+            *reinterpret_cast<__nv_bfloat162*>(out + 2) = __floats2bfloat162_rn(value.z * scale * gate_of(a, row, head, c + 2), value.w * scale * gate_of(a, row, head, c + 3));
         }
         return;
     }
@@ -1170,7 +1278,8 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
                 value += v3 * stat_factor[r * 32 + sp + 3];
             }
             for (; sp < splits; ++sp) value += __ldcg(part + (long long)sp * D) * stat_factor[r * 32 + sp];
-            a.out[(long long)row * a.ldo + (long long)head * D + c] = from_float<bf16>(value * stat_factor[8 * 32 + r]);
+            a.out[(long long)row * a.ldo + (long long)head * D + c] =
+                from_float<bf16>(value * stat_factor[8 * 32 + r] * gate_of(a, row, head, c));
         }
         if (threadIdx.x == 0) a.counters[(long long)row * a.kv_heads + kv_head] = 0;
     }
@@ -1191,11 +1300,12 @@ __global__ void attention_combine_kernel(Args a) {
             value += a.partial_out[(where + s) * D + c] * factor;
         }
         a.out[(long long)row * a.ldo + (long long)head * D + c] =
-            from_float<bf16>(value * finish_factor(a, row, head, top, total));
+            from_float<bf16>(value * finish_factor(a, row, head, top, total) * gate_of(a, row, head, c));
     }
 }
 
-constexpr size_t PREFILL_SHARED = (size_t)(TILE + 4 * TILE) * PITCH * sizeof(bf16);
+constexpr size_t PREFILL_SHARED = (size_t)(TILE + KV_TILES * TILE) * PITCH * sizeof(bf16);
+constexpr int RING_FORM = TIED ? 1 : 2;      // (tied values have no ring form)
 int kidi_decode_ring = 1;
 
 typedef CUresult (*EncodeTiled)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,
@@ -1226,9 +1336,15 @@ int page_map(CUtensorMap* map, const void* base, long long rows) {
 }
 
 bool aligned(const Args& a) {
-    return !((uintptr_t)a.q & 15) && !((uintptr_t)a.k_step & 15) && !((uintptr_t)a.v_step & 15) &&
+    return !((uintptr_t)a.element_gate & 1) && !((uintptr_t)a.q & 15) && !((uintptr_t)a.k_step & 15) && !((uintptr_t)a.v_step & 15) &&
            !((uintptr_t)a.k_cache & 15) && !((uintptr_t)a.v_cache & 15) && !((uintptr_t)a.out & 3) && !(a.ldq & 7) &&
            !(a.ldkv & 7) && !(a.ldo & 1);
+}
+// Whether the arguments are what this build takes.
+bool variant_fits(const Args& a) {
+    return (!SIGMOID || (a.weight_bias && !a.sinks && !a.gate && !a.element_gate)) &&
+           BIASED == (a.distance_bias != nullptr) && (!BIASED || (a.bias_last >= 0 && a.bias_stride > a.bias_last)) &&
+           (!TIED || (a.k_cache == a.v_cache && a.k_step == a.v_step));
 }
 }  // namespace
 
@@ -1244,7 +1360,7 @@ KIDI_API void kidi_attention_decode_ring(int enabled) { kidi_decode_ring = enabl
 // by shared memory (`swizzled`: the cache is one contiguous array and pages are copied whole).
 KIDI_API int kidi_attention_decode_blocks_per_sm(int swizzled) {
     const size_t block = (swizzled && D % 64 == 0)
-                             ? (kidi_decode_ring ? RING_SHARED : SWIZZLED_SHARED) : NARROW_SHARED;
+                             ? (kidi_decode_ring && !TIED ? RING_SHARED : SWIZZLED_SHARED) : NARROW_SHARED;
     const int fitting = (int)((228 * 1024) / (block + 1024));       // a kilobyte a block is the system's
     return fitting < 1 ? 1 : fitting > 4 ? 4 : fitting;             // four by registers
 }
@@ -1261,7 +1377,7 @@ KIDI_API int kidi_attention_prefill(const Args* args, int max_new, cudaStream_t 
     const Args& a = *args;
     if (a.rows <= 0 || a.seqs <= 0 || max_new <= 0) return 0;
     if (a.cache.head_dim != D || a.heads % a.kv_heads || a.heads > 65535 || a.seqs > 65535 || !aligned(a) ||
-        (a.cache.table && a.cache.page_shift != 6) || a.chunk < 0 || (SIGMOID && (!a.weight_bias || a.sinks || a.gate)))
+        (a.cache.table && a.cache.page_shift != 6) || a.chunk < 0 || !variant_fits(a))
         return KIDI_REFUSED_SIZE;
     static std::atomic<bool> configured{false};      // setting the attribute twice is harmless
     if (!configured.load(std::memory_order_acquire)) {
@@ -1281,7 +1397,7 @@ KIDI_API int kidi_attention_decode(const Args* args, cudaStream_t stream) {
     if (a.rows <= 0) return 0;
     const int group = a.kv_heads > 0 ? a.heads / a.kv_heads : 0;
     if (a.cache.head_dim != D || a.heads % a.kv_heads || group > 16 || a.kv_heads > 65535 || a.rows > 65535 ||
-        !aligned(a) || a.chunk < 0 || (SIGMOID && (!a.weight_bias || a.sinks || a.gate)) ||
+        !aligned(a) || a.chunk < 0 || !variant_fits(a) ||
         a.cache.page_shift != 6 || a.splits < 1 || a.splits > 65535 || (a.counters && a.splits > 32))
         return KIDI_REFUSED_SIZE;
     if (a.fuse) {   // the rotation inside the kernel: the narrow kernel, vectors of eight elements
@@ -1312,21 +1428,21 @@ KIDI_API int kidi_attention_decode(const Args* args, cudaStream_t stream) {
                                  (const void*)attention_decode_narrow_kernel<true, 0>,
                                  (const void*)attention_decode_narrow_kernel<false, 1>,
                                  (const void*)attention_decode_narrow_kernel<true, 1>,
-                                 (const void*)attention_decode_narrow_kernel<false, 2>,
-                                 (const void*)attention_decode_narrow_kernel<true, 2>};
-        const size_t sizes[3] = {NARROW_SHARED, SWIZZLED_SHARED, RING_SHARED};
+                                 (const void*)attention_decode_narrow_kernel<false, RING_FORM>,
+                                 (const void*)attention_decode_narrow_kernel<true, RING_FORM>};
+        const size_t sizes[3] = {NARROW_SHARED, SWIZZLED_SHARED, TIED ? SWIZZLED_SHARED : RING_SHARED};
         for (int i = 0; i < 6 && status == cudaSuccess; ++i)
             status = cudaFuncSetAttribute(narrow[i], cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizes[i >> 1]);
         if (status != cudaSuccess) return (int)status;
         configured.store(true, std::memory_order_release);
     }
     dim3 grid(a.splits, a.kv_heads, a.rows);
-    const int form = !swizzled ? 0 : kidi_decode_ring ? 2 : 1;
+    const int form = !swizzled ? 0 : kidi_decode_ring && !TIED ? 2 : 1;
     const size_t narrow_shared = form == 2 ? RING_SHARED : form == 1 ? SWIZZLED_SHARED : NARROW_SHARED;
     if (clustered) {
         const unsigned cluster = (unsigned)a.splits;
         if (form == 2)
-            return kidi_launch_clusters(attention_decode_narrow_kernel<true, 2>, grid, THREADS, narrow_shared, stream,
+            return kidi_launch_clusters(attention_decode_narrow_kernel<true, RING_FORM>, grid, THREADS, narrow_shared, stream,
                                         cluster, k_map, v_map, a);
         if (form == 1)
             return kidi_launch_clusters(attention_decode_narrow_kernel<true, 1>, grid, THREADS, narrow_shared, stream,
@@ -1337,7 +1453,7 @@ KIDI_API int kidi_attention_decode(const Args* args, cudaStream_t stream) {
     int status;
     if (group > 8) status = kidi_launch(attention_decode_kernel, grid, THREADS, DECODE_SHARED, stream, a);
     else if (form == 2)
-        status = kidi_launch(attention_decode_narrow_kernel<false, 2>, grid, THREADS, narrow_shared, stream, k_map, v_map, a);
+        status = kidi_launch(attention_decode_narrow_kernel<false, RING_FORM>, grid, THREADS, narrow_shared, stream, k_map, v_map, a);
     else if (form == 1)
         status = kidi_launch(attention_decode_narrow_kernel<false, 1>, grid, THREADS, narrow_shared, stream, k_map, v_map, a);
     else
@@ -1372,7 +1488,7 @@ KIDI_API long long kidi_attention_decode_static_need(int rows, int heads, int sp
 KIDI_API int kidi_attention_decode_static(const KidiAttentionArgs* args, cudaStream_t stream) {
     constexpr int MAX_DEVICES = 64;
     static std::atomic<float*> scratch_of_device[MAX_DEVICES];      // zero-initialised
-    if (SIGMOID) return KIDI_REFUSED_SIZE;      // the published block has no weight bias
+    if (SIGMOID || TIED || BIASED) return KIDI_REFUSED_SIZE;      // the published block has none of what these builds need
     Args a = {};           // (the public block ends before the weight bias: it stays null, and there are no chunks)
     memcpy(&a, args, sizeof(KidiAttentionArgs));
     a.out_scale = 1.f;

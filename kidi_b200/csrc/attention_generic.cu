@@ -15,6 +15,9 @@
 //    position p when u <= p (src/kidi/model/gemma4.cpp:736-740); with a window W,
 //    when also u > p - W; with chunks of C positions, when also floor(u / C) = floor(p / C).
 //  * instead of the softmax a key's weight can be sigmoid(s + b_h), b_h a number per head, normalised over nothing.
+//  * a number from a table [heads, distance] can be added to a score (p - u is the distance), and a value can be the key as
+//    it was before its norm: then only that is kept, s = r_u (q . k_u) scale with r_u = 1 / sqrt(sum(k_u^2)/d + eps), and the
+//    norm's weight rides in q.
 // Norm sums, rotation, scores, softmax and the weighted sum are 32-bit.
 #include "common.cuh"
 
@@ -39,14 +42,18 @@ struct RopeStoreArgs {
     int value_dim;             // width of a v head (0: head_dim); the v heads follow the k heads in a row
     const float* q_scale;      // [positions] or null: a q head at position p is multiplied by q_scale[p] (after the
                                // norm and the rotation)
+    int tied;                  // values are the keys before their norm: a row holds q heads and k heads, the k heads stay as
+                               // they are and are what the cache keeps (k_cache)
+    void* k_normed;            // [rows, ld_k_normed] or null (tied): takes the k heads divided by their root mean squares
+    long long ld_k_normed;
 };
 
-// One warp per (row, head) over heads + 2*kv_heads heads.
+// One warp per (row, head) over heads + 2*kv_heads heads (heads + kv_heads where values are keys).
 template <typename T, typename TW>
 __global__ void __launch_bounds__(128) rope_store_kernel(RopeStoreArgs a) {
     __shared__ float normed[4][256];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int total_heads = a.heads + 2 * a.kv_heads;
+    const int total_heads = a.heads + (a.tied ? 1 : 2) * a.kv_heads;
     const long long item = (long long)blockIdx.x * 4 + warp;
     if (item >= (long long)a.rows * total_heads) return;
     const int row = (int)(item / total_heads);
@@ -76,10 +83,18 @@ __global__ void __launch_bounds__(128) rope_store_kernel(RopeStoreArgs a) {
         }
     }
 
-    if (is_value || !a.transform) {  // a value head, or copy only
+    const bool raw_key = a.tied && head >= a.heads;
+    if (is_value || !a.transform || raw_key) {  // a value head, or copy only
         const int width = is_value ? vd : d;
         if (cached)
             for (int c = lane; c < width; c += 32) cached[c] = vector[c];
+        if (raw_key && a.transform && a.k_normed) {
+            float square = 0.f;
+            for (int c = lane; c < d; c += 32) square = fmaf(to_float(vector[c]), to_float(vector[c]), square);
+            const float inv = 1.0f / sqrtf(warp_sum(square) / (float)d + a.eps);
+            T* normed_key = (T*)a.k_normed + row * a.ld_k_normed + (long long)(head - a.heads) * d;
+            for (int c = lane; c < d; c += 32) normed_key[c] = from_float<T>(to_float(vector[c]) * inv);
+        }
         return;
     }
 
@@ -148,7 +163,7 @@ __device__ __forceinline__ void load8(const bf16* p, float (&w)[8]) {
 template <typename TW>
 __global__ void __launch_bounds__(128) rope_store_bf16_kernel(RopeStoreArgs a, int group_lanes) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int total_heads = a.heads + 2 * a.kv_heads;
+    const int total_heads = a.heads + (a.tied ? 1 : 2) * a.kv_heads;
     const int per_warp = 32 / group_lanes;
     const int group = lane / group_lanes, l = lane - group * group_lanes;
     const int item = (blockIdx.x * 4 + warp) * per_warp + group;   // the launcher keeps the count below 2^31
@@ -183,7 +198,8 @@ __global__ void __launch_bounds__(128) rope_store_bf16_kernel(RopeStoreArgs a, i
         }
     }
     if (!mine) raw = make_uint4(0u, 0u, 0u, 0u);
-    const bool plain = head >= a.heads + a.kv_heads || !a.transform;  // a value head, or copy only
+    const bool raw_key = a.tied && head >= a.heads;
+    const bool plain = head >= a.heads + a.kv_heads || !a.transform || raw_key;  // a value head, or copy only
     if (plain && cached && mine) *reinterpret_cast<uint4*>(cached + c0) = raw;
     const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&raw);
     float v[8];
@@ -206,6 +222,14 @@ __global__ void __launch_bounds__(128) rope_store_bf16_kernel(RopeStoreArgs a, i
             load8(weight + c0, w);
 #pragma unroll
             for (int i = 0; i < 8; ++i) v[i] = v[i] * inv * w[i];
+        }
+        if (raw_key && a.k_normed && a.transform && mine) {
+            const float inv = 1.0f / sqrtf(square / (float)d + a.eps);
+            uint4 packed;
+            __nv_bfloat162* out = reinterpret_cast<__nv_bfloat162*>(&packed);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) out[i] = __floats2bfloat162_rn(v[2 * i] * inv, v[2 * i + 1] * inv);
+            *reinterpret_cast<uint4*>((bf16*)a.k_normed + row * a.ld_k_normed + (head - a.heads) * d + c0) = packed;
         }
     }
     if (a.cos_table) {
@@ -246,11 +270,14 @@ KIDI_API int kidi_rope_store(const RopeStoreArgs* args, int dtype, int norm_dtyp
     if (a.rows <= 0) return 0;
     if (a.head_dim > 256 || a.head_dim <= 0 || a.rotary_dim > a.head_dim || (a.rotary_dim & 1) || a.value_dim < 0)
         return KIDI_REFUSED_SIZE;
-    const long long items = (long long)a.rows * (a.heads + 2 * a.kv_heads);
+    if (a.tied && (a.cos_table || a.v_cache || !a.q_norm || (a.value_dim && a.value_dim != a.head_dim)) && a.transform)
+        return KIDI_REFUSED_SIZE;
+    const long long items = (long long)a.rows * (a.heads + (a.tied ? 1 : 2) * a.kv_heads);
     const unsigned blocks = (unsigned)((items + 3) / 4);
     const bool vectors = dtype == KIDI_BF16 && items < (1LL << 30) && (!a.value_dim || a.value_dim == a.head_dim) && !((uintptr_t)a.q_norm & 15) &&
                          !((uintptr_t)a.k_norm & 15) && !(a.head_dim & 7) && !(a.ld & 7) && !((uintptr_t)a.qkv & 15) &&
-                         !((uintptr_t)a.k_cache & 15) && !((uintptr_t)a.v_cache & 15) &&
+                         !((uintptr_t)a.k_cache & 15) && !((uintptr_t)a.v_cache & 15) && !((uintptr_t)a.k_normed & 15) &&
+                         !(a.ld_k_normed & 7) &&
                          (!a.cos_table || (!(a.rotary_dim & 15) && !((uintptr_t)a.cos_table & 15) &&
                                            !((uintptr_t)a.sin_table & 15)));
     if (vectors) {
@@ -446,6 +473,13 @@ struct AttentionArgs {
                                // share of a softmax (nothing is normalised over the keys)
     int chunk;                 // > 0: only keys of the query's own run of `chunk` positions are seen
     float out_scale;           // the result is multiplied by it
+    int tied;                  // k_step / k_cache hold keys before their norm, which are the values too (v_step, v_cache name
+                               // the same rows); a score takes the factor 1 / sqrt(mean square of the key + key_eps)
+    float key_eps;
+    const float* distance_bias;   // [heads, bias_stride] or null: entry min(p - u, bias_last) of head h's row is added to a score
+    int bias_stride, bias_last;
+    const void* element_gate;     // [rows, ld_element_gate] or null: the result is multiplied by sigmoid of it, element by element
+    long long ld_element_gate;
 };
 
 // One block of 4 warps per (row, head). Warp w takes keys lo+w, lo+w+4, ... in
@@ -492,15 +526,21 @@ __global__ void __launch_bounds__(128) attention_generic_kernel(AttentionArgs a)
             key = (const T*)a.k_cache + offset;
             value = (const T*)a.v_cache + offset / d * vd;
         }
-        float dot = 0.f;
+        float dot = 0.f, square = 0.f;
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
             const int c = lane + 32 * i;
-            if (c < d) dot = fmaf(query[c], to_float(key[c]), dot);
+            if (c < d) {
+                const float entry = to_float(key[c]);
+                dot = fmaf(query[c], entry, dot);
+                square = fmaf(entry, entry, square);
+            }
         }
         float score = warp_sum(dot) * a.scale;
+        if (a.tied) score *= 1.0f / sqrtf(warp_sum(square) / (float)d + a.key_eps);
         if (a.softcap > 0.f) score = a.softcap * tanhf(score / a.softcap);
         if (a.slopes) score += a.slopes[head] * (float)(u - position);
+        if (a.distance_bias) score += a.distance_bias[(long long)head * a.bias_stride + min(position - u, a.bias_last)];
         if (a.weight_bias) {             // a weight of its own for every key: nothing to rescale
             const float weight = 1.0f / (1.0f + expf(-(score + a.weight_bias[head])));
 #pragma unroll
@@ -552,6 +592,8 @@ __global__ void __launch_bounds__(128) attention_generic_kernel(AttentionArgs a)
         for (int w = 0; w < 4; ++w) value += part_acc[w][c] * factor[w];
         value /= total;
         if (a.gate) value *= gate;
+        if (a.element_gate)
+            value *= 1.0f / (1.0f + expf(-to_float(((const T*)a.element_gate)[row * a.ld_element_gate + (long long)head * vd + c])));
         out[c] = from_float<T>(value * a.out_scale);
     }
 }
@@ -560,7 +602,8 @@ KIDI_API int kidi_attention_generic(const AttentionArgs* args, int dtype, cudaSt
     const AttentionArgs& a = *args;
     if (a.rows <= 0) return 0;
     if (a.head_dim > 256 || a.head_dim <= 0 || a.heads % a.kv_heads || a.heads > 65535 || a.value_dim < 0 ||
-        a.value_dim > 256 || a.chunk < 0 || (a.weight_bias && a.sinks))
+        a.value_dim > 256 || a.chunk < 0 || (a.weight_bias && a.sinks) || (a.tied && a.value_dim && a.value_dim != a.head_dim) ||
+        (a.distance_bias && (a.bias_last < 0 || a.bias_stride <= a.bias_last)))
         return KIDI_REFUSED_SIZE;
     dim3 grid(a.rows, a.heads);
     if (dtype == KIDI_F32) return kidi_launch(attention_generic_kernel<float>, grid, 128, 0, stream, a);

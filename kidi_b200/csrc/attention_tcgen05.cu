@@ -70,6 +70,13 @@ constexpr float RAISE_AFTER = 8.0f;               // the reference maximum follo
 #define KIDI_SIGMOID_WEIGHTS 0
 #endif
 constexpr bool SIGMOID = KIDI_SIGMOID_WEIGHTS != 0;
+// With -DKIDI_DISTANCE_BIAS=1 a number per head and distance is added to a score: one entry of a table a score near the
+// diagonal, one number a tile where every distance of the tile lies beyond the table's last entry.
+#ifndef KIDI_DISTANCE_BIAS
+#define KIDI_DISTANCE_BIAS 0
+#endif
+constexpr bool BIASED = KIDI_DISTANCE_BIAS != 0;
+static_assert(!SIGMOID || !BIASED, "sigmoid weights come without a distance bias");
 constexpr int TMEM_COLUMNS = 512;                 // S of head h: columns 128 h ..; O of head h: 256 + 128 h ..
 
 __device__ int kidi_attention_timeout = 0;
@@ -263,6 +270,11 @@ struct Params {
     int chunk;              // > 0: only keys of the query's own run of `chunk` positions are seen
     float out_scale;        // the result is multiplied by it
     SigmoidShape shape;
+    const float* distance_bias;   // biased build only: [heads, bias_stride] in base-2 exponent units, readable from entry -128
+    int bias_stride, bias_last;   // to bias_last + 384 of a row; distances beyond bias_last take that entry
+    const bf16* element_gate;     // [rows, ld_element_gate] or null: the result is multiplied by sigmoid of it
+    long long ld_element_gate;
+    int keys_apart;         // the keys are a matrix of their own (k_map); the rows hold query heads, then value heads
     int block_heads;        // query heads of a block: HEADS, or 1 where blocks of HEADS would leave SMs without one
 };
 
@@ -563,9 +575,10 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map, const 
                 // -------------------------------------------------------------- copies
                 const Place at(p);
                 const int tiles = at.tiles, tile_low = at.tile_low, row0 = at.row0, q0 = at.q0, head0 = at.head0;
-                const int k_col = (p.heads + at.kv_head) * D, v_col = (p.heads + p.kv_heads + at.kv_head) * D;
-                auto load_tile = [&](unsigned char* tile, unsigned long long* bar, int column, int row) {
-                    for (int s = 0; s < SPANS; ++s) tma_load_2d(tile + s * SPAN_BYTES, &map, bar, column + 64 * s, row);
+                const int k_col = (p.keys_apart ? at.kv_head : p.heads + at.kv_head) * D;
+                const int v_col = (p.heads + (p.keys_apart ? 0 : p.kv_heads) + at.kv_head) * D;
+                auto load_tile = [&](unsigned char* tile, unsigned long long* bar, int column, int row, const CUtensorMap* rows) {
+                    for (int s = 0; s < SPANS; ++s) tma_load_2d(tile + s * SPAN_BYTES, rows, bar, column + 64 * s, row);
                 };
                 // From the cache a tile is two pages (64 rows each) of the sequence's row of the block
                 // table; a page past the sequence's last one is replaced by the last one (masked).
@@ -582,16 +595,16 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map, const 
                 auto load_k = [&](int j) {
                     mbarrier_expect_tx(&ctl.k_full, QKV_TILE);
                     if (p.from_cache) load_pages(k_tile, &ctl.k_full, &k_map, j);
-                    else load_tile(k_tile, &ctl.k_full, k_col, row0 + (tile_low + j) * BN);
+                    else load_tile(k_tile, &ctl.k_full, k_col, row0 + (tile_low + j) * BN, p.keys_apart ? &k_map : &map);
                 };
                 auto load_v = [&](int j) {
                     mbarrier_expect_tx(&ctl.v_full[j & 1], QKV_TILE);
                     if (p.from_cache) load_pages(v_tiles + (j & 1) * QKV_TILE, &ctl.v_full[j & 1], &v_map, j);
-                    else load_tile(v_tiles + (j & 1) * QKV_TILE, &ctl.v_full[j & 1], v_col, row0 + (tile_low + j) * BN);
+                    else load_tile(v_tiles + (j & 1) * QKV_TILE, &ctl.v_full[j & 1], v_col, row0 + (tile_low + j) * BN, &map);
                 };
                 mbarrier_expect_tx(&ctl.q_full, heads_here * QKV_TILE);
                 for (int h = 0; h < heads_here; ++h)
-                    load_tile(q_tiles + h * QKV_TILE, &ctl.q_full, (head0 + h) * D, row0 + q0);
+                    load_tile(q_tiles + h * QKV_TILE, &ctl.q_full, (head0 + h) * D, row0 + q0, &map);
                 load_k(0);
                 load_v(0);
                 if (tiles > 1) load_v(1);
@@ -631,6 +644,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map, const 
             const int last_first_seen = first_visible(at.start + q0 + BM - 1, p.window, p.chunk);
             const float scale_log2 = p.scale * LOG2E;
             const float bias_log2 = SIGMOID ? -p.weight_bias[head0 + h] * LOG2E : 0.f;
+            const float* bias_row = BIASED ? p.distance_bias + (long long)(head0 + h) * p.bias_stride : nullptr;
             float reference = -INFINITY;                            // what the exponentials are taken against
             float denom = 0.f;                                      // this thread's part of the row sum
             unsigned exchanges = 0;                                 // uses of row_shared so far
@@ -677,8 +691,19 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map, const 
 #pragma unroll
                     for (int i = 0; i < SHARE; ++i) s[i] = outer * tanh_near(s[i] * inner);
                 }
-                const float mine = masked ? share_maximum<true>(s, scale_log2, first, last)
-                                          : share_maximum<false>(s, scale_log2, first, last);
+                float unit = scale_log2, shift = 0.f;       // a score in base-2 exponent units: s * unit + shift
+                if constexpr (BIASED) {
+                    if (at.start + q0 - (key0 + BN - 1) >= p.bias_last) {
+                        shift = __ldg(bias_row + p.bias_last);
+                    } else {                                // (distance of the thread's i-th key: last - i)
+                        const float* entry = bias_row + last;
+#pragma unroll
+                        for (int i = 0; i < SHARE; ++i) s[i] = fmaf(s[i], scale_log2, __ldg(entry - i));
+                        unit = 1.f;
+                    }
+                }
+                const float mine = (masked ? share_maximum<true>(s, unit, first, last)
+                                           : share_maximum<false>(s, unit, first, last)) + shift;
                 Exchange(&parts)[GROUPS] = ctl.row_part[h][exchanges & 1][r];
                 parts[group] = (Exchange)mine;
                 row_exchange();
@@ -715,10 +740,10 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map, const 
                 }
                 // The exponentials stay in registers until the product of the tile before has read
                 // its P from the tile in shared memory: they are computed while that product runs.
-                const float against = reference == -INFINITY ? 0.f : reference;
+                const float against = (reference == -INFINITY ? 0.f : reference) - shift;
                 unsigned packed[SHARE / 2];
-                denom += masked ? probabilities<true>(s, scale_log2, against, first, last, packed)
-                                : probabilities<false>(s, scale_log2, against, first, last, packed);
+                denom += masked ? probabilities<true>(s, unit, against, first, last, packed)
+                                : probabilities<false>(s, unit, against, first, last, packed);
                 if (!rested) {
                     ok = mbarrier_wait(&ctl.pv_done[h], (j - 1) & 1, abort_flag);
                     if (!ok) break;
@@ -747,6 +772,8 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map, const 
                     inverse *= 1.0f / (1.0f + expf(-__bfloat162float(p.gate[(long long)(row0 + q0 + r) * p.ldg + head0 + h])));
                 }
                 bf16* out = p.out + (long long)(row0 + q0 + r) * p.ldo + (long long)(head0 + h) * D;
+                const bf16* gate = !SIGMOID && p.element_gate ? p.element_gate + (long long)(row0 + q0 + r) * p.ld_element_gate +
+                                                        (long long)(head0 + h) * D : nullptr;
 #pragma unroll 1
                 for (int c = 32 * group; c < D && ok; c += 32 * GROUPS) {
                     float o[32];
@@ -754,6 +781,16 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map, const 
                     if (r < q_rows) {
 #pragma unroll
                         for (int i = 0; i < 32; i += 8) {
+                            if (gate) {
+                                const uint4 raw = *reinterpret_cast<const uint4*>(gate + c + i);
+                                const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+                                for (int t = 0; t < 4; ++t) {
+                                    const float2 z = __bfloat1622float2(pairs[t]);
+                                    o[i + 2 * t] = __fdividef(o[i + 2 * t], 1.0f + __expf(fminf(-z.x, 80.f)));
+                                    o[i + 2 * t + 1] = __fdividef(o[i + 2 * t + 1], 1.0f + __expf(fminf(-z.y, 80.f)));
+                                }
+                            }
                             uint4 packed;
                             __nv_bfloat162* pairs = reinterpret_cast<__nv_bfloat162*>(&packed);
 #pragma unroll
@@ -838,6 +875,12 @@ struct KidiHeadExtras {      // what a head's result passes beside the plain sof
     const float* weight_bias;   // [heads] float32, sigmoid build only (and there needed): a number added to a head's scores
     int chunk;               // > 0: only keys of the query's own run of `chunk` positions are seen
     float out_scale;         // the result is multiplied by it
+    const float* distance_bias;      // biased build only (and there needed): see Params
+    int bias_stride, bias_last;
+    const void* element_gate;        // [rows, ld_element_gate] bfloat16, 16-byte pieces: a gate per element of the result
+    long long ld_element_gate;
+    const void* keys;                // [rows, ld_keys] bfloat16: the step's keys, where qkv holds queries and values only
+    long long ld_keys;
 };
 
 // `cache` null: every sequence starts at position 0 and its keys are rows of qkv. Else every
@@ -855,7 +898,10 @@ KIDI_API int kidi_attention_prefill_tcgen05(const void* qkv, long long ld, int r
     EncodeTiled encode = encode_tiled();
     if (!encode) return KIDI_REFUSED_SIZE;
     CUtensorMap map;
-    const cuuint64_t dims[2] = {(cuuint64_t)(cache && cache->q_only ? heads : heads + 2 * kv_heads) * D, (cuuint64_t)rows};
+    const bool keys_apart = extras && extras->keys;
+    if (keys_apart && (cache || ((uintptr_t)extras->keys & 15) || (extras->ld_keys & 7))) return KIDI_REFUSED_SIZE;
+    const cuuint64_t dims[2] = {(cuuint64_t)(cache && cache->q_only ? heads : heads + (keys_apart ? 1 : 2) * kv_heads) * D,
+                                (cuuint64_t)rows};
     const cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
     const cuuint32_t box[2] = {64, 128};
     const cuuint32_t steps[2] = {1, 1};
@@ -877,6 +923,15 @@ KIDI_API int kidi_attention_prefill_tcgen05(const void* qkv, long long ld, int r
     memset(&v_map, 0, sizeof(v_map));
     Params p;
     memset(&p, 0, sizeof(p));
+    if (keys_apart) {
+        const cuuint64_t key_dims[2] = {(cuuint64_t)kv_heads * D, (cuuint64_t)rows};
+        const cuuint64_t key_strides[1] = {(cuuint64_t)extras->ld_keys * 2};
+        if (encode(&k_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(extras->keys), key_dims, key_strides, box,
+                   steps, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
+            return KIDI_REFUSED_SIZE;
+        p.keys_apart = 1;
+    }
     if (cache) {
         if (!cache->keys || !cache->values || cache->rows <= 0 || !cache->table || !cache->seq_start ||
             !cache->seq_slot || ((uintptr_t)cache->keys & 15) || ((uintptr_t)cache->values & 15))
@@ -917,7 +972,15 @@ KIDI_API int kidi_attention_prefill_tcgen05(const void* qkv, long long ld, int r
         p.weight_bias = extras->weight_bias;
         p.chunk = extras->chunk;
         p.out_scale = extras->out_scale;
+        p.distance_bias = extras->distance_bias;
+        p.bias_stride = extras->bias_stride;
+        p.bias_last = extras->bias_last;
+        p.element_gate = (const bf16*)extras->element_gate;
+        p.ld_element_gate = extras->ld_element_gate;
     }
+    if (BIASED != (p.distance_bias != nullptr) || (BIASED && (p.bias_last < 0 || p.bias_stride <= p.bias_last)) ||
+        ((uintptr_t)p.element_gate & 15) || (p.ld_element_gate & 7) || (SIGMOID && p.element_gate))
+        return KIDI_REFUSED_SIZE;
     p.shape = sigmoid_shape(p.scale, p.softcap);
     if (p.chunk < 0 || (SIGMOID && (!p.weight_bias || p.sinks || p.gate))) return KIDI_REFUSED_SIZE;
     const int group_size = heads / kv_heads;

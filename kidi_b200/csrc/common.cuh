@@ -83,6 +83,20 @@ __host__ __device__ __forceinline__ int first_visible(int position, int window, 
     return max(first, 0);
 }
 
+// What a gated feed-forward makes of a gate g and an up value u: SiLU(g) u, or, bounded, with g <- min(g, limit) and
+// u <- clamp(u, -limit, limit), g sigmoid(alpha g) (u + shift).
+struct GateShape {
+    int bounded;
+    float limit, alpha, shift;
+};
+
+__device__ __forceinline__ float gate_value(const GateShape& shape, float g, float u) {
+    if (!shape.bounded) return g / (1.0f + expf(-g)) * u;
+    g = fminf(g, shape.limit);
+    u = fminf(fmaxf(u, -shape.limit), shape.limit);
+    return g / (1.0f + expf(-shape.alpha * g)) * (u + shape.shift);
+}
+
 static inline int kidi_launch_status() { return (int)cudaGetLastError(); }
 
 __device__ __forceinline__ void prefetch_l2(const void* pointer) {

@@ -12,8 +12,8 @@
 // and their partial sums are added in warp order through shared memory (a fixed order:
 // the result does not depend on timing). Accumulation is 32-bit.
 //
-// Epilogues: plain store (bfloat16 or float32, with an optional bias), or the SiLU gate of
-// a fused [gate | up] projection, out = silu(gate) * up, for which a block reads the 16
+// Epilogues: plain store (bfloat16 or float32, with an optional bias), or the gate of
+// a fused [gate | up] projection, out = silu(gate) * up or its bounded form, for which a block reads the 16
 // gate rows and the 16 matching up rows.
 //
 // Two more epilogues take the RMSNorm between two products out of the step (a norm of its
@@ -51,6 +51,7 @@ struct Epilogue {
     int gelu;                     // the plain store writes an activation of y + bias instead of y + bias: 1 the exact
                                   // (erf) gelu, 2 the squared relu max(y + bias, 0)^2, 3 SiLU on the output features
     int silu_begin, silu_end;     // silu_begin .. silu_end - 1
+    GateShape gate;               // the gated form's activation
 };
 
 __device__ __forceinline__ uint4 load_streaming(const void* pointer) {
@@ -226,7 +227,7 @@ gemm_skinny_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, TY* _
 #pragma unroll
             for (int v = 0; v < W; ++v) up += partial[((long long)v * ROWS + (MT == 1 ? 8 : 16) + r) * COLS + m];
             if (FACTORS && m < M) up *= row_factor[m];
-            sum = sum / (1.0f + expf(-sum)) * up;
+            sum = gate_value(e.gate, sum, up);
         } else if (e.bias && inside) {
             sum += e.bias[n0 + r];
         }
@@ -302,6 +303,7 @@ struct KidiSkinnyExtras {          // every pointer may be null: the plain produ
     int gelu;                      // not gated, not into the residual: the result passes the exact gelu (1) or the
                                    // squared relu (2), or its features silu_begin .. silu_end - 1 pass SiLU (3)
     int silu_begin, silu_end;
+    GateShape gate;                // the gated form's activation (all zero: SiLU)
 };
 
 // How many parts per row the product into the residual writes for N features.
@@ -332,6 +334,7 @@ KIDI_API int kidi_gemm_skinny(const void* x, const void* w, void* y, int y_dtype
         e.gelu = extras->gelu;
         e.silu_begin = extras->silu_begin;
         e.silu_end = extras->silu_end;
+        e.gate = extras->gate;
         if (e.gelu && (gated || e.residual)) return KIDI_REFUSED_SIZE;
         if (e.factor_parts && (e.factor_count < 1 || e.factor_stride < e.factor_count || e.factor_width < 1))
             return KIDI_REFUSED_SIZE;

@@ -177,6 +177,7 @@ struct Params {
     const int* group_of_tile;   // [token tiles] or null: the tile's tokens take the weight rows from group * group_rows on
                                 // (a tile whose group is negative holds no tokens and is left out)
     int group_rows;
+    GateShape gate;             // the gated form's activation (all zero: SiLU)
 };
 
 // Tiles are numbered so that the blocks at work at one time share few weight tiles and few token
@@ -416,7 +417,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                         mine = mine && row < 64;
                         if (row < 64)
 #pragma unroll
-                            for (int i = 0; i < CW; ++i) v[i] = v[i] / (1.0f + expf(-v[i])) * exchange[row * (CW + 1) + i];
+                            for (int i = 0; i < CW; ++i) v[i] = gate_value(p.gate, v[i], exchange[row * (CW + 1) + i]);
                         asm volatile("bar.sync 1, 128;" ::: "memory");
                     } else if (p.bias && mine) {
                         const float shift = p.bias[f0 + row];
@@ -512,7 +513,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                         for (int j = 0; j < 16; ++j)
                             if (j0 + j < count)
                                 y[(long long)(t0 + first + j0 + j) * p.ldy + f0 + row] =
-                                    from_float<TY>(sum[j] / (1.0f + expf(-sum[j])) * exchange[row * 17 + j]);
+                                    from_float<TY>(gate_value(p.gate, sum[j], exchange[row * 17 + j]));
                     asm volatile("bar.sync 1, 128;" ::: "memory");
                 } else if (f0 + row < p.features) {
 #pragma unroll
@@ -775,6 +776,7 @@ KIDI_API int kidi_gemm_tcgen05(const void* x, const void* w, void* y, int y_dtyp
     p.token_tiles = (tokens + bn - 1) / bn;
     p.group_of_tile = nullptr;
     p.group_rows = 0;
+    p.gate = GateShape{};
     const long long tiles = (long long)((features + span - 1) / span) * p.token_tiles;
     const int blocks = kidi_gemm_tcgen05_blocks(tokens, features, K, gated, splits);
     if (tiles / blocks > 0x7fffffffLL) return KIDI_REFUSED_SIZE;
@@ -813,10 +815,11 @@ KIDI_API int kidi_gemm_tcgen05(const void* x, const void* w, void* y, int y_dtyp
 
 // The same for weights in groups (the experts of a routed feed-forward) and rows that are sorted by group: x [tokens, K] in
 // tiles of 128 rows, tile i's rows taking group group_of_tile[i] of w [groups, features (2 * features when gated), K]
-// (negative: the tile holds nothing; its rows of y are not written). Whole tiles only; no bias.
+// (negative: the tile holds nothing; its rows of y are not written). Whole tiles only; no bias. `gate`: the gated form's
+// activation (null: SiLU).
 KIDI_API int kidi_gemm_tcgen05_grouped(const void* x, const void* w, void* y, int tokens, int features, int K, long long ldx,
                                        long long ldy, int gated, int groups, const int* group_of_tile, int* error,
-                                       cudaStream_t stream) {
+                                       const GateShape* gate, cudaStream_t stream) {
     constexpr int BN = 128;
     if (tokens <= 0 || features <= 0) return 0;
     const long long rows = (long long)groups * features * (gated ? 2 : 1);
@@ -837,6 +840,7 @@ KIDI_API int kidi_gemm_tcgen05_grouped(const void* x, const void* w, void* y, in
     p.group_of_tile = group_of_tile;
     p.group_rows = features * (gated ? 2 : 1);
     p.staged = 1;
+    if (gate) p.gate = *gate;
     const long long sms = sm_count_of_current_device();
     const int blocks = (int)(p.tiles < sms ? p.tiles : sms);
     if (p.tiles / blocks > 0x7fffffffLL) return KIDI_REFUSED_SIZE;

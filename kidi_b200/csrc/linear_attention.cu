@@ -3,16 +3,23 @@
 //     S_t = decay_h S_(t-1) + k_t v_t^T            S: [dim, vdim] per head
 //     o_t = S_t^T q_t
 //
-// with q, k and v as their projections' activations left them. What is here beside the scan that other recurrences
+// with q, k and v as their projections' activations left them, or with q and k rotated by position and k times a number
+// ("retention"; both in 32-bit, on the way into the recurrence). What is here beside the scan that other recurrences
 // with one decay per head share (scalar_recurrence.cu):
 //
 //  * one token a sequence (decoding): a block takes 32 columns of a (sequence, head), reads its part of the state
-//    once with every load in flight, writes it back and adds up the read-out;
+//    once with every load in flight, writes it back and adds up the read-out. The blocks of a head can form a cluster
+//    that also finishes the head: divided by its root mean square (the blocks exchange their sums of squares through
+//    distributed shared memory), times the SiLU or sigmoid of a gate, rounded;
+//  * rotated and scaled queries and keys as 32-bit numbers (for the scan);
+//  * the finish head by head as a kernel of its own;
 //  * the finish: a row's concatenated heads divided by their one root mean square, times a weight, times
 //    sigmoid(gate), times a number;
 //  * SiLU on a range of a projection's columns, in place.
 //
 // State, decay, read-out and norm are 32-bit.
+#include <cooperative_groups.h>
+
 #include "common.cuh"
 
 struct LinearStepArgs {
@@ -29,6 +36,20 @@ struct LinearStepArgs {
     const int* seq_slot;   // [seqs]
     const int* seq_row0;   // [seqs]
     int seqs, heads, dim, vdim;
+    // Optional: entries i and i + rotary_dim / 2 of a head's q and k (i < rotary_dim / 2) are turned by position, and k is
+    // multiplied by key_scale.
+    const float* cos_table;   // [positions, rotary_dim / 2] or null
+    const float* sin_table;
+    const int* row_pos;       // [rows]
+    int rotary_dim;
+    float key_scale;
+    // Optional: the head is finished here. `finished` (of the step's element type) takes read / rms(read) * act(gate).
+    const void* gate;         // [rows, ldg] or null: head h at h * vdim
+    long long ldg;
+    void* finished;           // [rows, ldf]
+    long long ldf;
+    float eps;
+    int gate_silu;            // act: 1 SiLU, 0 sigmoid
 };
 
 namespace {
@@ -51,9 +72,27 @@ __device__ __forceinline__ void dot_add(float& s, float keep, float key, const f
     sum = fmaf(s, query, sum);
 }
 
+// Entry d of a head's row x, rotated.
+template <typename T>
+__device__ __forceinline__ float rotated(const T* x, int d, const float* cos_table, const float* sin_table, int rotary_dim,
+                                         int position) {
+    const float own = to_float(x[d]);
+    if (d >= rotary_dim) return own;
+    const int half = rotary_dim / 2, j = d < half ? d : d - half;
+    const float other = to_float(x[d < half ? d + half : d - half]);
+    const float cosine = cos_table[(long long)position * half + j], sine = sin_table[(long long)position * half + j];
+    return own * cosine + (d < half ? -other : other) * sine;
+}
+
+__device__ __forceinline__ float gate_activation(float z, int silu) {
+    const float s = 1.0f / (1.0f + expf(-z));
+    return silu ? z * s : s;
+}
+
 // V columns a thread (4 where the widths allow 16-byte accesses), 32 / V threads beside one another, the others on
 // further state rows; DEPTH rows a thread are in flight together.
-template <typename T, int V>
+// FINISH: the grid's blocks along x (a head's columns) form a cluster and finish the head.
+template <typename T, int V, bool FINISH>
 __global__ void __launch_bounds__(THREADS) linear_step_kernel(LinearStepArgs a) {
     typedef typename Columns<V>::type Vec;
     constexpr int LANES = COLUMNS / V, ROWS = THREADS / LANES, DEPTH = 4;
@@ -61,12 +100,15 @@ __global__ void __launch_bounds__(THREADS) linear_step_kernel(LinearStepArgs a) 
     float* keys = shared;
     float* queries = shared + a.dim;
     float* partial = shared + ((2 * a.dim + 3) & ~3);
-    const int head = blockIdx.y, seq = blockIdx.x;
+    __shared__ float squares[8];                           // of the head's columns, by block of the cluster
+    const int head = blockIdx.y, seq = blockIdx.z;
     const int row = a.seq_row0[seq];
-    if (a.row_seq[row] < 0) return;                        // a padding sequence touches no state
+    if (a.row_seq[row] < 0) return;                        // a padding sequence touches no state (nor does its whole cluster)
     const int dim = a.dim, vdim = a.vdim;
     const int lane = threadIdx.x % LANES, group = threadIdx.x / LANES;
-    const int column = blockIdx.z * COLUMNS + lane * V;
+    // (Every block of a cluster has begun before another one writes to its shared memory.)
+    if constexpr (FINISH) asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");
+    const int column = blockIdx.x * COLUMNS + lane * V;
     const bool live = column < vdim;                       // (vdim is a multiple of V)
     float* state = a.state + ((long long)a.seq_slot[seq] * a.heads + head) * dim * vdim + column;
     Vec s[DEPTH];
@@ -75,9 +117,10 @@ __global__ void __launch_bounds__(THREADS) linear_step_kernel(LinearStepArgs a) 
         const int d = group + j * ROWS;
         if (live && d < dim) s[j] = *reinterpret_cast<const Vec*>(state + (long long)d * vdim);
     }
+    const int rotary_dim = a.cos_table ? a.rotary_dim : 0, position = a.cos_table ? a.row_pos[row] : 0;
     for (int d = threadIdx.x; d < dim; d += THREADS) {
-        keys[d] = to_float(((const T*)a.k)[row * a.ldk + (long long)head * dim + d]);
-        queries[d] = to_float(((const T*)a.q)[row * a.ldq + (long long)head * dim + d]);
+        keys[d] = a.key_scale * rotated((const T*)a.k + row * a.ldk + (long long)head * dim, d, a.cos_table, a.sin_table, rotary_dim, position);
+        queries[d] = rotated((const T*)a.q + row * a.ldq + (long long)head * dim, d, a.cos_table, a.sin_table, rotary_dim, position);
     }
     float value[V], total[V];
 #pragma unroll
@@ -108,11 +151,71 @@ __global__ void __launch_bounds__(THREADS) linear_step_kernel(LinearStepArgs a) 
     }
     *reinterpret_cast<Vec*>(partial + group * COLUMNS + lane * V) = sum;
     __syncthreads();
-    if (threadIdx.x < COLUMNS && blockIdx.z * COLUMNS + threadIdx.x < vdim) {
-        float read = 0.f;
+    float read = 0.f;
+    const int mine = blockIdx.x * COLUMNS + threadIdx.x;     // the column that a thread of the first warp finishes
+    const bool reads = threadIdx.x < COLUMNS && mine < vdim;
+    if (reads) {
 #pragma unroll
         for (int g = 0; g < ROWS; ++g) read += partial[g * COLUMNS + threadIdx.x];
-        a.out[((long long)row * a.heads + head) * vdim + blockIdx.z * COLUMNS + threadIdx.x] = read;
+        if (!FINISH) a.out[((long long)row * a.heads + head) * vdim + mine] = read;
+    }
+    if constexpr (FINISH) {
+        cooperative_groups::cluster_group cluster = cooperative_groups::this_cluster();
+        const int blocks = gridDim.x;                        // == the cluster's size, <= 8
+        float z = 0.f;
+        asm volatile("barrier.cluster.wait.aligned;" ::: "memory");
+        if (reads) z = to_float(((const T*)a.gate)[row * a.ldg + (long long)head * vdim + mine]);
+        if (threadIdx.x < 32) {
+            const float square = warp_sum(read * read);      // (threads without a column hold zero)
+            if (threadIdx.x < blocks) *cluster.map_shared_rank(&squares[blockIdx.x], threadIdx.x) = square;
+        }
+        cluster.sync();                                      // nothing is read from another block after it
+        if (reads) {
+            float total = 0.f;
+            for (int b = 0; b < blocks; ++b) total += squares[b];
+            ((T*)a.finished)[row * a.ldf + (long long)head * vdim + mine] =
+                from_float<T>(read / sqrtf(total / (float)vdim + a.eps) * gate_activation(z, a.gate_silu));
+        }
+    }
+}
+
+// Rotated queries and keys (keys times key_scale) and values, all as 32-bit numbers: out[r] = [q | k | v]. A block a row.
+template <typename T>
+__global__ void __launch_bounds__(THREADS)
+rotate_heads_kernel(const T* __restrict__ q, long long ldq, const T* __restrict__ k, long long ldk, const T* __restrict__ v,
+                    long long ldv, float* __restrict__ out, const float* __restrict__ cos_table,
+                    const float* __restrict__ sin_table, const int* __restrict__ row_pos, int rotary_dim, float key_scale,
+                    int heads, int dim, int vdim) {
+    const long long row = blockIdx.x;
+    const int qk = heads * dim, values = heads * vdim, position = row_pos[row];
+    float* to = out + row * (2 * qk + values);
+    for (int c = threadIdx.x; c < qk; c += THREADS) {
+        const int head = c / dim, d = c - head * dim;
+        to[c] = rotated(q + row * ldq + head * dim, d, cos_table, sin_table, rotary_dim, position);
+        to[qk + c] = key_scale * rotated(k + row * ldk + head * dim, d, cos_table, sin_table, rotary_dim, position);
+    }
+    for (int c = threadIdx.x; c < values; c += THREADS) to[2 * qk + c] = to_float(v[row * ldv + c]);
+}
+
+// y = read / sqrt(mean(read^2) + eps) * weight * act(gate) * factor head by head (weight: [heads * vdim] or null). A warp a
+// (row, head).
+template <typename T>
+__global__ void __launch_bounds__(THREADS)
+head_gate_kernel(const float* __restrict__ read, const float* __restrict__ weight, const T* __restrict__ gate, long long ldg,
+                 T* __restrict__ out, long long ldo, long long items, int heads, int vdim, float eps, float factor, int silu) {
+    const long long item = (long long)blockIdx.x * (THREADS / 32) + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & 31;
+    if (item >= items) return;
+    const long long row = item / heads;
+    const int head = (int)(item - row * heads);
+    const float* source = read + item * vdim;
+    float square = 0.f;
+    for (int c = lane; c < vdim; c += 32) square = fmaf(source[c], source[c], square);
+    const float inv = factor / sqrtf(warp_sum(square) / (float)vdim + eps);
+    for (int c = lane; c < vdim; c += 32) {
+        const int at = head * vdim + c;
+        const float y = source[c] * inv * gate_activation(to_float(gate[row * ldg + at]), silu);
+        out[row * ldo + at] = from_float<T>(weight ? y * weight[at] : y);
     }
 }
 
@@ -222,16 +325,55 @@ KIDI_API int kidi_linear_step(const LinearStepArgs* args, int dtype, cudaStream_
     if (a.seqs <= 0) return 0;
     const int spans = (a.vdim + COLUMNS - 1) / COLUMNS;
     const size_t shared = (size_t)(((2 * a.dim + 3) & ~3) + THREADS * 4) * sizeof(float);    // ROWS * COLUMNS = THREADS * V
-    if (a.heads <= 0 || a.heads > 65535 || a.dim <= 0 || a.vdim <= 0 || spans > 65535 || shared > 48 * 1024)
+    if (a.heads <= 0 || a.heads > 65535 || a.seqs > 65535 || a.dim <= 0 || a.vdim <= 0 || shared > 48 * 1024 ||
+        (a.cos_table && (!a.sin_table || !a.row_pos || (a.rotary_dim & 1) || a.rotary_dim < 0 || a.rotary_dim > a.dim)) ||
+        (a.gate && (spans > 8 || !a.finished)) || (!a.gate && !a.out))
         return KIDI_REFUSED_SIZE;
-    const dim3 grid(a.seqs, a.heads, spans);
+    const dim3 grid(spans, a.heads, a.seqs);
     const bool vectors = !(a.vdim & 3) && !((uintptr_t)a.state & 15);
+#define KIDI_CASE(D, T)                                                                                                     \
+    if (dtype == D) {                                                                                                       \
+        if (a.gate)                                                                                                         \
+            return vectors ? kidi_launch_clusters(linear_step_kernel<T, 4, true>, grid, THREADS, shared, stream, spans, a)  \
+                           : kidi_launch_clusters(linear_step_kernel<T, 1, true>, grid, THREADS, shared, stream, spans, a); \
+        return vectors ? kidi_launch(linear_step_kernel<T, 4, false>, grid, THREADS, shared, stream, a)                     \
+                       : kidi_launch(linear_step_kernel<T, 1, false>, grid, THREADS, shared, stream, a);                    \
+    }
+    KIDI_CASE(KIDI_F32, float)
+    KIDI_CASE(KIDI_BF16, bf16)
+#undef KIDI_CASE
+    return KIDI_REFUSED_DTYPE;
+}
+
+KIDI_API int kidi_rotate_heads(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv, int dtype,
+                               float* out, const float* cos_table, const float* sin_table, const int* row_pos, int rotary_dim,
+                               float key_scale, int rows, int heads, int dim, int vdim, cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (heads <= 0 || dim <= 0 || vdim <= 0 || rotary_dim < 0 || (rotary_dim & 1) || rotary_dim > dim || !row_pos ||
+        (rotary_dim > 0 && (!cos_table || !sin_table)))
+        return KIDI_REFUSED_SIZE;
     if (dtype == KIDI_F32)
-        return vectors ? kidi_launch(linear_step_kernel<float, 4>, grid, THREADS, shared, stream, a)
-                       : kidi_launch(linear_step_kernel<float, 1>, grid, THREADS, shared, stream, a);
+        return kidi_launch(rotate_heads_kernel<float>, rows, THREADS, 0, stream, (const float*)q, ldq, (const float*)k, ldk,
+                           (const float*)v, ldv, out, cos_table, sin_table, row_pos, rotary_dim, key_scale, heads, dim, vdim);
     if (dtype == KIDI_BF16)
-        return vectors ? kidi_launch(linear_step_kernel<bf16, 4>, grid, THREADS, shared, stream, a)
-                       : kidi_launch(linear_step_kernel<bf16, 1>, grid, THREADS, shared, stream, a);
+        return kidi_launch(rotate_heads_kernel<bf16>, rows, THREADS, 0, stream, (const bf16*)q, ldq, (const bf16*)k, ldk,
+                           (const bf16*)v, ldv, out, cos_table, sin_table, row_pos, rotary_dim, key_scale, heads, dim, vdim);
+    return KIDI_REFUSED_DTYPE;
+}
+
+KIDI_API int kidi_head_norm_gate(const float* read, const float* weight, const void* gate, long long ldg, int dtype, void* out,
+                                 long long ldo, int rows, int heads, int vdim, float eps, float factor, int silu,
+                                 cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (heads <= 0 || vdim <= 0) return KIDI_REFUSED_SIZE;
+    const long long items = (long long)rows * heads;
+    const unsigned blocks = (unsigned)((items + THREADS / 32 - 1) / (THREADS / 32));
+    if (dtype == KIDI_F32)
+        return kidi_launch(head_gate_kernel<float>, blocks, THREADS, 0, stream, read, weight, (const float*)gate, ldg, (float*)out,
+                           ldo, items, heads, vdim, eps, factor, silu);
+    if (dtype == KIDI_BF16)
+        return kidi_launch(head_gate_kernel<bf16>, blocks, THREADS, 0, stream, read, weight, (const bf16*)gate, ldg, (bf16*)out, ldo,
+                           items, heads, vdim, eps, factor, silu);
     return KIDI_REFUSED_DTYPE;
 }
 

@@ -14,6 +14,11 @@
 // number to the last bit or nearly (8 + 8 + 8 significant bits), each multiplied into the same 32-bit accumulators. States
 // and their walk are 32-bit throughout.
 //
+// With -DKIDI_LINEAR_WIDE=1 ("retention") q and k are turned by position and k is multiplied by a number, in 32-bit, on the
+// way into the products: they are 32-bit numbers then and enter in three parts too (of a product of two such numbers the six
+// partial products above 2^-24 are kept), and the read-out finishes a head: divided by its root mean square, times the SiLU
+// or sigmoid of a gate, rounded to bfloat16.
+//
 // mma.sync serves these products, not tcgen05: they are 64 x 64 x dim and dim x vdim x 64 with factors that are made in
 // registers (decays, splits), which an mma.sync operand is and a tcgen05 operand is not (it would have to go through
 // shared memory three times over).
@@ -42,6 +47,18 @@ struct LinearChunksArgs {
     int seqs, heads;
     int head0, group;       // the heads of this launch: head0 .. head0 + group - 1
     int max_chunks;         // chunks of the longest sequence
+    // the wide build only
+    const float* cos_table; // [positions, rotary_dim / 2] or null: entries i and i + rotary_dim / 2 of a head's q and k turn
+    const float* sin_table;
+    const int* row_pos;     // [rows]
+    int rotary_dim;
+    float key_scale;
+    const bf16* gate;       // [rows, ldg]: head h at h * vdim
+    long long ldg;
+    bf16* finished;         // [rows, ldf]: takes read / rms(read) * act(gate)
+    long long ldf;
+    float eps;
+    int gate_silu;          // act: 1 SiLU, 0 sigmoid
 };
 
 namespace {
@@ -51,7 +68,22 @@ static_assert(D % 16 == 0 && E % 16 == 0 && D >= 16 && E >= 16 && D <= 256 && E 
 constexpr int CHUNK = 64;
 constexpr int THREADS = 256;
 constexpr int DP = D + 8, EP = E + 8;               // row pitches: ldmatrix without bank conflicts
-constexpr int SLICE = D % 32 == 0 ? 32 : 16;        // rows of the state that are in shared memory at a time
+#ifndef KIDI_LINEAR_WIDE
+#define KIDI_LINEAR_WIDE 0
+#endif
+constexpr bool WIDE = KIDI_LINEAR_WIDE != 0;
+constexpr int SCORE_PITCH = CHUNK + 8;
+// Shared memory of the wide read-out with slices of `slice` rows of the state: q and k in three parts, v, the slices (later
+// the scores in three parts), the decay's powers and the rows' sums of squares.
+__host__ __device__ constexpr size_t wide_read_bytes(int slice) {
+    const size_t slices = (size_t)2 * 3 * slice * EP, scores = (size_t)3 * CHUNK * SCORE_PITCH;
+    return ((size_t)6 * CHUNK * DP + (size_t)CHUNK * EP + (slices > scores ? slices : scores)) * sizeof(bf16) +
+           (size_t)(CHUNK + 4 + 4 * CHUNK) * sizeof(float);
+}
+constexpr size_t MOST_SHARED = 227 * 1024;
+static_assert(!WIDE || wide_read_bytes(16) <= MOST_SHARED, "head widths of the wide build: too large for shared memory");
+constexpr int SLICE = D % 32 == 0 && (!WIDE || wide_read_bytes(32) <= MOST_SHARED) ? 32 : 16;   // rows of the state that are
+                                                                                             // in shared memory at a time
 constexpr int SLICES = D / SLICE;
 
 // A sequence's chunks follow one another; the first one's index (no two sequences overlap: a chunk index grows by at
@@ -120,6 +152,27 @@ struct Chunk {
     }
 };
 
+// The wide build: a chunk's rows of q or k as 32-bit numbers, turned by position and times `scale`, from the bfloat16 tile
+// `raw`; `store(row, column, value)` takes every entry. A thread that takes entry i of a rotated pair takes its partner too.
+template <typename Store>
+__device__ __forceinline__ void widen(const bf16* raw, const LinearChunksArgs& a, int row0, int tokens, float scale, int threads,
+                                      Store store) {
+    const int half = a.cos_table ? a.rotary_dim / 2 : 0, units = D - half;       // pairs, then single entries
+    for (int i = threadIdx.x; i < CHUNK * units; i += threads) {
+        const int r = i / units, c = i - r * units;
+        const bf16* source = raw + r * DP;
+        if (c < half) {
+            const long long at = (long long)a.row_pos[row0 + min(r, tokens - 1)] * half + c;
+            const float cosine = a.cos_table[at], sine = a.sin_table[at];
+            const float u = to_float(source[c]), v = to_float(source[c + half]);
+            store(r, c, scale * (u * cosine - v * sine));
+            store(r, c + half, scale * (v * cosine + u * sine));
+        } else {
+            store(r, c + half, scale * to_float(source[c + half]));
+        }
+    }
+}
+
 // ---------------------------------------------------------------- a chunk's own sum
 // [dim, vdim] = sum over j of a^(n-1-j) k_j v_j^T. A warp takes 16 rows (of dim) by up to 64 columns (of vdim) at a time;
 // the keys come transposed out of shared memory, are decayed and split in registers.
@@ -128,6 +181,7 @@ __global__ void __launch_bounds__(THREADS) chunk_sums_kernel(LinearChunksArgs a)
     bf16* k_tile = reinterpret_cast<bf16*>(raw);            // [64][DP]
     bf16* v_tile = k_tile + CHUNK * DP;                     // [64][EP]
     float* weight = reinterpret_cast<float*>(v_tile + CHUNK * EP);      // [64]
+    float* wide_keys = weight + CHUNK;                      // the wide build: [64][D + 4]
     const Chunk chunk(a, blockIdx.z, blockIdx.x);
     if (!chunk.live) return;
     const int head = a.head0 + blockIdx.y;
@@ -138,6 +192,11 @@ __global__ void __launch_bounds__(THREADS) chunk_sums_kernel(LinearChunksArgs a)
         weight[threadIdx.x] = threadIdx.x < chunk.tokens ? powf(a.decay[head], (float)(chunk.tokens - 1 - threadIdx.x)) : 0.f;
     copy_async_wait<0>();
     __syncthreads();
+    if constexpr (WIDE) {
+        widen(k_tile, a, chunk.row, chunk.tokens, a.key_scale, THREADS,
+              [&](int r, int c, float value) { wide_keys[r * (D + 4) + c] = value; });
+        __syncthreads();
+    }
     constexpr int SPAN = 64, SPANS = (E + SPAN - 1) / SPAN;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     const int matrix = lane >> 3, within = lane & 7;
@@ -154,12 +213,20 @@ __global__ void __launch_bounds__(THREADS) chunk_sums_kernel(LinearChunksArgs a)
             unsigned keys[4], parts[3][4];
             // A operand, rows m0 .. m0 + 15 (of dim) by 16 tokens: matrices (rows, tokens), (rows + 8, tokens),
             // (rows, tokens + 8), (rows + 8, tokens + 8), each transposed on the way.
-            ldmatrix_x4_trans(keys, k_tile + (kk * 16 + within + (matrix >> 1) * 8) * DP + m0 + (matrix & 1) * 8);
+            if constexpr (!WIDE)
+                ldmatrix_x4_trans(keys, k_tile + (kk * 16 + within + (matrix >> 1) * 8) * DP + m0 + (matrix & 1) * 8);
             const float2 w0 = *reinterpret_cast<const float2*>(weight + kk * 16 + 2 * t);
             const float2 w1 = *reinterpret_cast<const float2*>(weight + kk * 16 + 8 + 2 * t);
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
-                const float2 key = unpack(keys[i]), w = i < 2 ? w0 : w1;
+                float2 key;
+                if constexpr (WIDE) {                       // rows m0 + g (+ 8), tokens 2t, 2t + 1 (+ 8)
+                    const float* from = wide_keys + (kk * 16 + 2 * t + (i >> 1) * 8) * (D + 4) + m0 + g + (i & 1) * 8;
+                    key = make_float2(from[0], from[D + 4]);
+                } else {
+                    key = unpack(keys[i]);
+                }
+                const float2 w = i < 2 ? w0 : w1;
                 split_pair(key.x * w.x, key.y * w.y, parts[0][i], parts[1][i], parts[2][i]);
             }
 #pragma unroll
@@ -228,7 +295,9 @@ __global__ void __launch_bounds__(WALK_THREADS) chunk_states_kernel(LinearChunks
 // Four warps by 16 tokens, twice: of the pairs of 8-column tiles one half of the warps takes the even, the other the odd.
 // First q S for the state before the chunk, slice by slice (SLICE rows of S in three parts), its rows times a^(i+1); then
 // the scores q k^T, decayed and split in registers, times v into the same accumulators.
-constexpr int PAIRS = E / 16, MINE = (PAIRS + 1) / 2;
+constexpr int PAIRS = E / 16;
+#if !KIDI_LINEAR_WIDE
+constexpr int MINE = (PAIRS + 1) / 2;
 constexpr size_t READ_SHARED = (size_t)(2 * CHUNK * DP + CHUNK * EP + 2 * 3 * SLICE * EP) * sizeof(bf16) + (CHUNK + 1) * sizeof(float);
 
 __global__ void __launch_bounds__(THREADS) chunk_read_kernel(LinearChunksArgs a) {
@@ -353,7 +422,211 @@ __global__ void __launch_bounds__(THREADS) chunk_read_kernel(LinearChunksArgs a)
     }
 }
 
-constexpr size_t SUMS_SHARED = (size_t)CHUNK * (DP + EP) * sizeof(bf16) + CHUNK * sizeof(float);
+#else   // KIDI_LINEAR_WIDE
+// ---------------------------------------------------------------- the read-out of the wide build
+// Sixteen warps: four times 16 tokens by four sides (a side takes every fourth pair of 8-column tiles). q and k are widened
+// and split in shared memory once; the scores of 16 tokens against 16 keys are one warp's (side = key tile), which leaves
+// them, decayed and split, where the slices of the state were.
+constexpr int WIDE_THREADS = 512, SIDES = 4, WIDE_MINE = (PAIRS + SIDES - 1) / SIDES;
+
+// Three parts of x, the largest first.
+__device__ __forceinline__ void split_store(bf16* at, int plane, float x) {
+    const bf16 first = __float2bfloat16_rn(x);
+    x -= __bfloat162float(first);
+    const bf16 second = __float2bfloat16_rn(x);
+    at[0] = first;
+    at[plane] = second;
+    at[2 * plane] = __float2bfloat16_rn(x - __bfloat162float(second));
+}
+
+__global__ void __launch_bounds__(WIDE_THREADS) chunk_read_wide_kernel(LinearChunksArgs a) {
+    extern __shared__ __align__(16) unsigned char raw[];
+    constexpr int PLANE = CHUNK * DP, SCORE_PLANE = CHUNK * SCORE_PITCH;
+    bf16* q_parts = reinterpret_cast<bf16*>(raw);           // [3][64][DP] (the bfloat16 rows first stand in the first plane)
+    bf16* k_parts = q_parts + 3 * PLANE;                    // [3][64][DP]
+    bf16* v_tile = k_parts + 3 * PLANE;                     // [64][EP]
+    bf16* s_tile = v_tile + CHUNK * EP;                     // [2][3][SLICE][EP], then the scores [3][64][SCORE_PITCH]
+    constexpr int SHARED_TILE = 2 * 3 * SLICE * EP > 3 * SCORE_PLANE ? 2 * 3 * SLICE * EP : 3 * SCORE_PLANE;
+    float* power = reinterpret_cast<float*>(s_tile + SHARED_TILE);      // [65]: a^0 .. a^64
+    float* squares = power + CHUNK + 4;                     // [SIDES][64]
+    const Chunk chunk(a, blockIdx.z, blockIdx.x);
+    if (!chunk.live) return;
+    const int head = a.head0 + blockIdx.y;
+    const bf16* before = a.before + 3 * (((long long)chunk.index * a.group + blockIdx.y) * D * E);
+    auto load_rows_wide = [&](bf16* tile, const bf16* source, long long ld, int width, int pitch) {
+        const int pieces = width / 8;
+        for (int i = threadIdx.x; i < CHUNK * pieces; i += WIDE_THREADS) {
+            const int r = i / pieces, c = i - r * pieces;
+            const bool valid = r < chunk.tokens;
+            copy_async_16(tile + r * pitch + c * 8, source + (long long)(valid ? r : 0) * ld + c * 8, valid);
+        }
+    };
+    auto load_slice = [&](int slice) {
+        constexpr int PIECES = E / 8;
+        bf16* target = s_tile + (slice & 1) * (3 * SLICE * EP);
+        for (int i = threadIdx.x; i < 3 * SLICE * PIECES; i += WIDE_THREADS) {
+            const int r = i / PIECES, c = i - r * PIECES;                  // r: part * SLICE + row
+            const int part = r / SLICE, row = slice * SLICE + r - part * SLICE;
+            copy_async_16(target + r * EP + c * 8, before + ((long long)part * D + row) * E + c * 8, true);
+        }
+        copy_async_commit();
+    };
+    load_rows_wide(q_parts, a.q + chunk.row * a.ldq + (long long)head * D, a.ldq, D, DP);
+    load_rows_wide(k_parts, a.k + chunk.row * a.ldk + (long long)head * D, a.ldk, D, DP);
+    load_rows_wide(v_tile, a.v + chunk.row * a.ldv + (long long)head * E, a.ldv, E, EP);
+    copy_async_commit();
+    load_slice(0);
+    for (int i = threadIdx.x; i <= CHUNK; i += WIDE_THREADS) power[i] = powf(a.decay[head], (float)i);
+    copy_async_wait<1>();
+    __syncthreads();
+    // (In place: a thread reads an entry and its partner before it writes either, and nobody else reads them.)
+    widen(q_parts, a, chunk.row, chunk.tokens, 1.f, WIDE_THREADS,
+          [&](int r, int c, float value) { split_store(q_parts + r * DP + c, PLANE, value); });
+    widen(k_parts, a, chunk.row, chunk.tokens, a.key_scale, WIDE_THREADS,
+          [&](int r, int c, float value) { split_store(k_parts + r * DP + c, PLANE, value); });
+
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    const int matrix = lane >> 3, within = lane & 7;
+    const int row = (warp & 3) * 16, side = warp >> 2;      // the warp's 16 tokens; its pairs: side, side + SIDES, ..
+    float o[2 * WIDE_MINE][4];
+#pragma unroll
+    for (int j = 0; j < 2 * WIDE_MINE; ++j)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) o[j][i] = 0.f;
+    for (int slice = 0; slice < SLICES; ++slice) {
+        if (slice + 1 < SLICES) {
+            load_slice(slice + 1);
+            copy_async_wait<1>();
+        } else {
+            copy_async_wait<0>();
+        }
+        __syncthreads();
+        const bf16* current = s_tile + (slice & 1) * (3 * SLICE * EP);
+#pragma unroll
+        for (int kk = 0; kk < SLICE / 16; ++kk) {
+            unsigned q[3][4];
+#pragma unroll
+            for (int part = 0; part < 3; ++part)
+                ldmatrix_x4(q[part], q_parts + part * PLANE + (row + within + (matrix & 1) * 8) * DP + slice * SLICE + kk * 16 + (matrix >> 1) * 8);
+#pragma unroll
+            for (int p = 0; p < WIDE_MINE; ++p) {
+                const int column = (side + SIDES * p) * 16;
+                if (column >= E) continue;
+                unsigned s[3][4];
+#pragma unroll
+                for (int part = 0; part < 3; ++part)
+                    ldmatrix_x4_trans(s[part], current + (part * SLICE + kk * 16 + within + (matrix & 1) * 8) * EP + column + (matrix >> 1) * 8);
+#pragma unroll
+                for (int order = 2; order >= 0; --order)    // the smallest partial products first
+#pragma unroll
+                    for (int part = order; part >= 0; --part) {
+                        mma_bf16(o[2 * p], q[part], s[order - part][0], s[order - part][1]);
+                        mma_bf16(o[2 * p + 1], q[part], s[order - part][2], s[order - part][3]);
+                    }
+            }
+        }
+        __syncthreads();                                    // the slice is read: its buffer takes the one after next
+    }
+    const float below = power[row + g + 1], above = power[row + g + 9];
+#pragma unroll
+    for (int j = 0; j < 2 * WIDE_MINE; ++j) {
+        o[j][0] *= below; o[j][1] *= below;
+        o[j][2] *= above; o[j][3] *= above;
+    }
+    // Scores: this warp's 16 tokens against key tile `side`, where it holds a key at or before the last of them.
+    bf16* score_parts = s_tile;
+    if (side <= (warp & 3)) {
+        float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+#pragma unroll
+        for (int kk = 0; kk < D / 16; ++kk) {
+            unsigned q[3][4], k[3][4];
+#pragma unroll
+            for (int part = 0; part < 3; ++part) {
+                ldmatrix_x4(q[part], q_parts + part * PLANE + (row + within + (matrix & 1) * 8) * DP + kk * 16 + (matrix >> 1) * 8);
+                ldmatrix_x4(k[part], k_parts + part * PLANE + (side * 16 + within + (matrix >> 1) * 8) * DP + kk * 16 + (matrix & 1) * 8);
+            }
+#pragma unroll
+            for (int order = 2; order >= 0; --order)
+#pragma unroll
+                for (int part = order; part >= 0; --part) {
+                    mma_bf16(s[0], q[part], k[order - part][0], k[order - part][1]);
+                    mma_bf16(s[1], q[part], k[order - part][2], k[order - part][3]);
+                }
+        }
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int i = 0; i < 4; i += 2) {
+                const int r = row + g + (i >> 1) * 8, key = side * 16 + j * 8 + 2 * t, back = r - key;
+                const float x = back >= 0 ? s[j][i] * power[back] : 0.f, y = back >= 1 ? s[j][i + 1] * power[back - 1] : 0.f;
+                unsigned parts[3];
+                split_pair(x, y, parts[0], parts[1], parts[2]);
+#pragma unroll
+                for (int part = 0; part < 3; ++part)
+                    *reinterpret_cast<unsigned*>(score_parts + part * SCORE_PLANE + r * SCORE_PITCH + key) = parts[part];
+            }
+    }
+    __syncthreads();
+    for (int kt = 0; kt <= (warp & 3); ++kt) {
+        unsigned parts[3][4];
+#pragma unroll
+        for (int part = 0; part < 3; ++part)
+            ldmatrix_x4(parts[part], score_parts + part * SCORE_PLANE + (row + within + (matrix & 1) * 8) * SCORE_PITCH + kt * 16 + (matrix >> 1) * 8);
+#pragma unroll
+        for (int p = 0; p < WIDE_MINE; ++p) {
+            const int column = (side + SIDES * p) * 16;
+            if (column >= E) continue;
+            unsigned v[4];
+            ldmatrix_x4_trans(v, v_tile + (kt * 16 + within + (matrix & 1) * 8) * EP + column + (matrix >> 1) * 8);
+#pragma unroll
+            for (int part = 2; part >= 0; --part) {
+                mma_bf16(o[2 * p], parts[part], v[0], v[1]);
+                mma_bf16(o[2 * p + 1], parts[part], v[2], v[3]);
+            }
+        }
+    }
+    // The finish: a row's sum of squares over its columns (a quad's lanes, then the sides in order), norm, gate.
+    float square[2] = {0.f, 0.f};
+#pragma unroll
+    for (int j = 0; j < 2 * WIDE_MINE; ++j)                 // (columns that do not exist hold zeros)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) square[i >> 1] = fmaf(o[j][i], o[j][i], square[i >> 1]);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        square[i] += __shfl_xor_sync(0xffffffffu, square[i], 1);
+        square[i] += __shfl_xor_sync(0xffffffffu, square[i], 2);
+        if (t == 0) squares[side * CHUNK + row + g + i * 8] = square[i];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        const int r = row + g + i * 8;
+        if (r >= chunk.tokens) continue;
+        const float total = squares[r] + squares[CHUNK + r] + squares[2 * CHUNK + r] + squares[3 * CHUNK + r];
+        const float inv = 1.0f / sqrtf(total / (float)E + a.eps);
+        const bf16* gate = a.gate + (long long)(chunk.row + r) * a.ldg + (long long)head * E;
+        bf16* out = a.finished + (long long)(chunk.row + r) * a.ldf + (long long)head * E;
+#pragma unroll
+        for (int p = 0; p < WIDE_MINE; ++p) {
+            const int column = (side + SIDES * p) * 16;
+            if (column >= E) continue;
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+                const int c = column + j * 8 + 2 * t;
+                const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gate + c));
+                // (sigmoid with the fast exponential and division: the result is rounded to bfloat16)
+                const float x = __fdividef(a.gate_silu ? z.x : 1.f, 1.0f + __expf(fminf(-z.x, 80.f)));
+                const float y = __fdividef(a.gate_silu ? z.y : 1.f, 1.0f + __expf(fminf(-z.y, 80.f)));
+                *reinterpret_cast<__nv_bfloat162*>(out + c) =
+                    __floats2bfloat162_rn(o[2 * p + j][2 * i] * inv * x, o[2 * p + j][2 * i + 1] * inv * y);
+            }
+        }
+    }
+}
+
+#endif  // KIDI_LINEAR_WIDE
+
+constexpr size_t SUMS_SHARED = (size_t)CHUNK * (DP + EP) * sizeof(bf16) + (CHUNK + (WIDE ? CHUNK * (D + 4) : 0)) * sizeof(float);
 
 }  // namespace
 
@@ -372,9 +645,22 @@ KIDI_API int kidi_linear_chunks(const LinearChunksArgs* args, cudaStream_t strea
         (a.ldq & 7) || (a.ldk & 7) || (a.ldv & 7) || ((uintptr_t)a.q & 15) || ((uintptr_t)a.k & 15) || ((uintptr_t)a.v & 15) ||
         ((uintptr_t)a.state & 15) || ((uintptr_t)a.out & 15) || ((uintptr_t)a.sums & 15) || ((uintptr_t)a.before & 15))
         return KIDI_REFUSED_SIZE;
+#if KIDI_LINEAR_WIDE
+    if (!a.row_pos || !a.gate || !a.finished || (a.ldg & 1) || (a.ldf & 1) || ((uintptr_t)a.gate & 3) ||
+        ((uintptr_t)a.finished & 3) ||
+        (a.cos_table && (!a.sin_table || a.rotary_dim < 0 || (a.rotary_dim & 1) || a.rotary_dim > D)))
+        return KIDI_REFUSED_SIZE;
+    const auto read_kernel = chunk_read_wide_kernel;
+    const size_t read_shared = wide_read_bytes(SLICE);
+    const int read_threads = WIDE_THREADS;
+#else
+    const auto read_kernel = chunk_read_kernel;
+    const size_t read_shared = READ_SHARED;
+    const int read_threads = THREADS;
+#endif
     cudaError_t status = cudaFuncSetAttribute(chunk_sums_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SUMS_SHARED);
     if (status == cudaSuccess)
-        status = cudaFuncSetAttribute(chunk_read_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)READ_SHARED);
+        status = cudaFuncSetAttribute(read_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)read_shared);
     if (status != cudaSuccess) return (int)status;
     const dim3 grid(a.max_chunks, a.group, a.seqs);
     int launched = kidi_launch(chunk_sums_kernel, grid, THREADS, SUMS_SHARED, stream, a);
@@ -382,5 +668,5 @@ KIDI_API int kidi_linear_chunks(const LinearChunksArgs* args, cudaStream_t strea
     const dim3 walk((D * E / 4 + WALK_THREADS - 1) / WALK_THREADS, a.group, a.seqs);
     launched = kidi_launch(chunk_states_kernel, walk, WALK_THREADS, 0, stream, a);
     if (launched) return launched;
-    return kidi_launch(chunk_read_kernel, grid, THREADS, READ_SHARED, stream, a);
+    return kidi_launch(read_kernel, grid, read_threads, read_shared, stream, a);
 }

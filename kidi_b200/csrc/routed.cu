@@ -4,9 +4,11 @@
 //   experts with the largest scores are taken (ties: the lower index) with weights w = s (optionally divided
 //   by their sum plus a small number). With groups, the experts form equal runs of neighbours, a group's
 //   score is its largest, and only experts of the `keep` best groups (ties: the lower index) can be taken;
+//   Optionally: a correction per expert that the choice sees (scores plus correction, for experts and groups alike) and the
+//   weights do not, groups ranked by the sum of their two largest, weights times a number;
 //   y = sum over the chosen experts of  scale_out * W_down[e] (act(W_gate[e] x) * (W_up[e] x)),
 //   x = scale_in * h, where the weight w is scale_in (a weight on the expert's input) or scale_out
-//   (on its output) and the other is 1. act is SiLU. An expert without a gate is W_down[e] gelu(W_up[e] x)
+//   (on its output) and the other is 1. act(g) u is SiLU(g) u or its bounded form (GateShape). An expert without a gate is W_down[e] gelu(W_up[e] x)
 //   with the exact gelu, 0.5 z (1 + erf(z / sqrt 2)).
 //
 // A (row, choice) pair is a "slot": slot = row * top + choice.
@@ -59,11 +61,17 @@ template <typename T, typename TW>
 __global__ void __launch_bounds__(512) route_kernel(const T* __restrict__ x, const TW* __restrict__ router,
                                                     int* __restrict__ chosen, float* __restrict__ weight, int hidden,
                                                     int experts, int top, int renormalise, int softmax, int groups,
-                                                    int keep, float renormalise_eps, const float* __restrict__ bias) {
+                                                    int keep, float renormalise_eps, const float* __restrict__ bias,
+                                                    const float* __restrict__ correction, int two_largest, float weight_scale,
+                                                    const TW* __restrict__ share_row, float* __restrict__ share) {
     extern __shared__ float score[];       // [experts] scores, then [experts] what may still be chosen
     float* open = score + experts;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long row = blockIdx.x;
+    if (share && warp == 15) {             // the gate of the expert that every row passes
+        const float z = warp_sum(dot1<T, TW>(share_row, x + row * hidden, hidden, lane));
+        if (lane == 0) share[row] = 1.0f / (1.0f + expf(-z));
+    }
     for (int e = warp; e < experts; e += 16) {
         float z = warp_sum(dot1<T, TW>(router + (long long)e * hidden, x + row * hidden, hidden, lane));
         if (bias) z += bias[e];
@@ -81,17 +89,23 @@ __global__ void __launch_bounds__(512) route_kernel(const T* __restrict__ x, con
         for (int e = lane; e < experts; e += 32) score[e] = expf(score[e] - most) / sum;
         __syncwarp();
     }
-    for (int e = lane; e < experts; e += 32) open[e] = score[e];
+    // What the choice goes by.
+    auto choice = [&](int e) { return correction ? score[e] + correction[e] : score[e]; };
+    for (int e = lane; e < experts; e += 32) open[e] = choice(e);
     __syncwarp();
     if (groups > 1 && keep < groups) {
         // The best `keep` groups stay open: one after the other the group with the largest best score is marked,
         // then every expert of an unmarked group is closed. A lane looks after groups lane, lane + 32, ...
         const int per = experts / groups;
         for (int g = lane; g < groups; g += 32) {
-            float best = -INFINITY;
-            for (int e = g * per; e < (g + 1) * per; ++e) best = fmaxf(best, score[e]);
-            // a group's best score is kept in its first expert's `open` entry while the groups are ranked
-            open[g * per] = best;
+            float best = -INFINITY, second = -INFINITY;
+            for (int e = g * per; e < (g + 1) * per; ++e) {
+                const float s = choice(e);
+                second = fmaxf(second, fminf(best, s));
+                best = fmaxf(best, s);
+            }
+            // a group's score is kept in its first expert's `open` entry while the groups are ranked
+            open[g * per] = two_largest && per > 1 ? best + second : best;
         }
         __syncwarp();
         unsigned long long kept_low = 0ull;      // groups kept by this lane, bit j for group lane + 32 j
@@ -115,7 +129,7 @@ __global__ void __launch_bounds__(512) route_kernel(const T* __restrict__ x, con
         __syncwarp();
         for (int g = lane, j = 0; g < groups; g += 32, ++j) {
             const bool kept = kept_low >> j & 1ull;
-            for (int e = g * per; e < (g + 1) * per; ++e) open[e] = kept ? score[e] : -INFINITY;
+            for (int e = g * per; e < (g + 1) * per; ++e) open[e] = kept ? choice(e) : -INFINITY;
         }
         __syncwarp();
     }
@@ -133,7 +147,8 @@ __global__ void __launch_bounds__(512) route_kernel(const T* __restrict__ x, con
             const int other_at = __shfl_xor_sync(0xffffffffu, at, offset);
             if (other > best || (other == best && other_at < at)) { best = other; at = other_at; }
         }
-        if (at == 0x7fffffff) { at = k; best = score[k]; }   // every score left is a NaN or closed
+        if (at == 0x7fffffff) at = k;                    // every score left is a NaN or closed
+        best = score[at];                                // the weight: the score without the correction
         if (lane == 0) {
             chosen[row * top + k] = at;
             weight[row * top + k] = best;
@@ -142,13 +157,18 @@ __global__ void __launch_bounds__(512) route_kernel(const T* __restrict__ x, con
         total += best;
         __syncwarp();
     }
-    if (renormalise && lane < top) weight[row * top + lane] /= total + renormalise_eps;
+    if (lane < top && (renormalise || weight_scale != 1.f)) {
+        const float w = weight[row * top + lane];
+        weight[row * top + lane] = (renormalise ? w / (total + renormalise_eps) : w) * weight_scale;
+    }
 }
 
 KIDI_API int kidi_route(const void* x, int dtype, const void* router, int weight_dtype, int* chosen, float* weight,
                         int rows, int hidden, int experts, int top, int renormalise, int softmax, int groups, int keep,
-                        float renormalise_eps, const float* bias, cudaStream_t stream) {
+                        float renormalise_eps, const float* bias, const float* correction, int two_largest,
+                        float weight_scale, const void* share_row, float* share, cudaStream_t stream) {
     if (rows <= 0) return 0;
+    if (share && !share_row) return KIDI_REFUSED_SIZE;
     if (experts <= 0 || experts > 1024 || top <= 0 || top > experts || top > 32) return KIDI_REFUSED_SIZE;
     if (groups < 1 || experts % groups || keep < 1 || keep > groups || groups > 2048 ||
         (long long)keep * (experts / groups) < top)
@@ -158,7 +178,7 @@ KIDI_API int kidi_route(const void* x, int dtype, const void* router, int weight
     if (dtype == D && weight_dtype == W)                                                                              \
         return kidi_launch(route_kernel<T, TW>, (unsigned)rows, 512, shared, stream, (const T*)x, (const TW*)router,  \
                            chosen, weight, hidden, experts, top, renormalise, softmax, groups, keep, renormalise_eps, \
-                           bias);
+                           bias, correction, two_largest, weight_scale, (const TW*)share_row, share);
     KIDI_CASE(KIDI_F32, float, KIDI_F32, float)
     KIDI_CASE(KIDI_F32, float, KIDI_BF16, bf16)
     KIDI_CASE(KIDI_BF16, bf16, KIDI_BF16, bf16)
@@ -210,7 +230,7 @@ template <typename T, typename TW>
 __global__ void __launch_bounds__(128) expert_gate_up_kernel(const T* __restrict__ x, const TW* __restrict__ gate_up,
                                                              const int* __restrict__ chosen, const float* __restrict__ weight,
                                                              T* __restrict__ mid, long long slots, int top, int hidden,
-                                                             int inter, int weight_on_input, int gated) {
+                                                             int inter, int weight_on_input, int gated, GateShape shape) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long item = (long long)blockIdx.x * 4 + warp;
     if (item >= slots * inter) return;
@@ -235,19 +255,20 @@ __global__ void __launch_bounds__(128) expert_gate_up_kernel(const T* __restrict
         const float w = weight_on_input ? weight[slot] : 1.f;
         g *= w;
         u *= w;
-        mid[slot * inter + n] = from_float<T>(gated ? g / (1.0f + expf(-g)) * u
+        mid[slot * inter + n] = from_float<T>(gated ? gate_value(shape, g, u)
                                                     : 0.5f * g * (1.0f + erff(g * 0.70710678118654752440f)));
     }
 }
 
 // ---------------------------------------------------------- slots: down
 // down [experts, hidden, inter]; out [rows, hidden] = sum over a row's choices, in their order (plus `addend`
-// [rows, hidden], if given: the result of an expert that every row passes).
+// [rows, hidden], if given: the result of an expert that every row passes, times share[row], if given).
 template <typename T, typename TW>
 __global__ void __launch_bounds__(128) expert_down_kernel(const T* __restrict__ mid, const TW* __restrict__ down,
                                                           const int* __restrict__ chosen, const float* __restrict__ weight,
                                                           T* __restrict__ out, long long rows, int top, int hidden, int inter,
-                                                          int weight_on_input, const T* __restrict__ addend) {
+                                                          int weight_on_input, const T* __restrict__ addend,
+                                                          const float* __restrict__ share) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long item = (long long)blockIdx.x * 4 + warp;
     if (item >= rows * hidden) return;
@@ -265,26 +286,30 @@ __global__ void __launch_bounds__(128) expert_down_kernel(const T* __restrict__ 
         a = warp_sum(a);
         total += weight_on_input ? a : a * weight[slot];
     }
-    if (lane == 0) out[row * hidden + n] = from_float<T>(addend ? total + to_float(addend[row * hidden + n]) : total);
+    if (lane == 0) {
+        if (addend) total += to_float(addend[row * hidden + n]) * (share ? share[row] : 1.f);
+        out[row * hidden + n] = from_float<T>(total);
+    }
 }
 
 KIDI_API int kidi_expert_slots(const void* x, int dtype, const void* gate_up, const void* down, int weight_dtype,
                                const int* chosen, const float* weight, void* mid, void* out, int rows, int top,
                                int hidden, int inter, int weight_on_input, int gated, const void* addend, int parts,
-                               cudaStream_t stream) {       // parts: 1 the gate and up products, 2 the down product, 3 both
+                               const GateShape* shape, const float* share, cudaStream_t stream) {       // parts: 1 the gate and up products, 2 the down product, 3 both
     if (rows <= 0) return 0;
     const long long slots = (long long)rows * top;
     const long long first = slots * inter, second = (long long)rows * hidden;
     if (first >= (1LL << 33) || second >= (1LL << 33)) return KIDI_REFUSED_SIZE;
+    const GateShape gate = shape ? *shape : GateShape{};
 #define KIDI_CASE(D, T, W, TW)                                                                                     \
     if (dtype == D && weight_dtype == W) {                                                                         \
         int status = parts & 1 ? kidi_launch(expert_gate_up_kernel<T, TW>, (unsigned)((first + 3) / 4), 128, 0,    \
                                              stream, (const T*)x, (const TW*)gate_up, chosen, weight, (T*)mid,     \
-                                             slots, top, hidden, inter, weight_on_input, gated) : 0;               \
+                                             slots, top, hidden, inter, weight_on_input, gated, gate) : 0;         \
         if (status || !(parts & 2)) return status;                                                                 \
         return kidi_launch(expert_down_kernel<T, TW>, (unsigned)((second + 3) / 4), 128, 0, stream, (const T*)mid, \
                            (const TW*)down, chosen, weight, (T*)out, (long long)rows, top, hidden, inter,          \
-                           weight_on_input, (const T*)addend);                                                     \
+                           weight_on_input, (const T*)addend, share);                                              \
     }
     KIDI_CASE(KIDI_F32, float, KIDI_F32, float)
     KIDI_CASE(KIDI_F32, float, KIDI_BF16, bf16)
@@ -372,7 +397,7 @@ __global__ void gather_slots_kernel(const T* __restrict__ x, const int* __restri
 template <typename T>
 __global__ void combine_slots_kernel(const T* __restrict__ y, const int* __restrict__ place, const float* __restrict__ weight,
                                      T* __restrict__ out, long long total, int top, int hidden, int weight_on_input,
-                                     const T* __restrict__ addend) {
+                                     const T* __restrict__ addend, const float* __restrict__ share) {
     const long long index = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (index >= total) return;
     const long long row = index / hidden;
@@ -383,7 +408,7 @@ __global__ void combine_slots_kernel(const T* __restrict__ y, const int* __restr
         const float value = to_float(y[(long long)place[slot] * hidden + c]);
         sum += weight_on_input ? value : value * weight[slot];
     }
-    if (addend) sum += to_float(addend[index]);
+    if (addend) sum += to_float(addend[index]) * (share ? share[row] : 1.f);
     out[index] = from_float<T>(sum);
 }
 
@@ -413,7 +438,8 @@ __global__ void gather_slots_bf16x8_kernel(const bf16* __restrict__ x, const int
 
 __global__ void combine_slots_bf16x8_kernel(const bf16* __restrict__ y, const int* __restrict__ place,
                                             const float* __restrict__ weight, bf16* __restrict__ out, long long groups,
-                                            int top, int hidden, int weight_on_input, const bf16* __restrict__ addend) {
+                                            int top, int hidden, int weight_on_input, const bf16* __restrict__ addend,
+                                            const float* __restrict__ share) {
     const long long index = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (index >= groups) return;
     const int per_row = hidden >> 3;
@@ -435,11 +461,12 @@ __global__ void combine_slots_bf16x8_kernel(const bf16* __restrict__ y, const in
     if (addend) {
         const uint4 raw = *reinterpret_cast<const uint4*>(addend + row * hidden + c);
         const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&raw);
+        const float part = share ? share[row] : 1.f;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const float2 v = __bfloat1622float2(pairs[j]);
-            sum[2 * j] += v.x;
-            sum[2 * j + 1] += v.y;
+            sum[2 * j] = fmaf(v.x, part, sum[2 * j]);
+            sum[2 * j + 1] = fmaf(v.y, part, sum[2 * j + 1]);
         }
     }
     uint4 result;
@@ -465,17 +492,18 @@ KIDI_API int kidi_gather_slots(const void* x, int dtype, const int* order, const
 }
 
 KIDI_API int kidi_combine_slots(const void* y, int dtype, const int* place, const float* weight, void* out, int rows,
-                                int top, int hidden, int weight_on_input, const void* addend, cudaStream_t stream) {
+                                int top, int hidden, int weight_on_input, const void* addend, const float* share,
+                                cudaStream_t stream) {
     const long long total = (long long)rows * hidden;
     if (total <= 0) return 0;
     const unsigned blocks = (unsigned)((total + 255) / 256);
     if (dtype == KIDI_F32) return kidi_launch(combine_slots_kernel<float>, blocks, 256, 0, stream, (const float*)y, place,
-                                              weight, (float*)out, total, top, hidden, weight_on_input, (const float*)addend);
+                                              weight, (float*)out, total, top, hidden, weight_on_input, (const float*)addend, share);
     if (dtype == KIDI_BF16 && !(hidden & 7) && !((uintptr_t)y & 15) && !((uintptr_t)out & 15) && !((uintptr_t)addend & 15))
         return kidi_launch(combine_slots_bf16x8_kernel, (unsigned)(((total >> 3) + 255) / 256), 256, 0, stream,
                            (const bf16*)y, place, weight, (bf16*)out, total >> 3, top, hidden, weight_on_input,
-                           (const bf16*)addend);
+                           (const bf16*)addend, share);
     if (dtype == KIDI_BF16) return kidi_launch(combine_slots_kernel<bf16>, blocks, 256, 0, stream, (const bf16*)y, place,
-                                               weight, (bf16*)out, total, top, hidden, weight_on_input, (const bf16*)addend);
+                                               weight, (bf16*)out, total, top, hidden, weight_on_input, (const bf16*)addend, share);
     return KIDI_REFUSED_DTYPE;
 }

@@ -235,13 +235,19 @@ class CacheGeometry(ctypes.Structure):
                 ("kv_heads", c_int), ("head_dim", c_int)]
 
 
+class GateShape(ctypes.Structure):
+    """What a gated feed-forward makes of gate and up: SiLU(g) u, or bounded (GateShape of csrc/common.cuh)."""
+    _fields_ = [("bounded", c_int), ("limit", c_float), ("alpha", c_float), ("shift", c_float)]
+
+
 class RopeStoreArgs(ctypes.Structure):
     _fields_ = [("qkv", c_void_p), ("ld", c_longlong), ("q_norm", c_void_p), ("k_norm", c_void_p),
                 ("cos_table", c_void_p), ("sin_table", c_void_p), ("row_seq", c_void_p), ("row_pos", c_void_p),
                 ("seq_slot", c_void_p), ("seq_start", c_void_p), ("seq_len", c_void_p), ("k_cache", c_void_p),
                 ("v_cache", c_void_p), ("cache", CacheGeometry), ("rows", c_int), ("heads", c_int),
                 ("kv_heads", c_int), ("head_dim", c_int), ("rotary_dim", c_int), ("eps", c_float), ("transform", c_int),
-                ("value_dim", c_int), ("q_scale", c_void_p)]
+                ("value_dim", c_int), ("q_scale", c_void_p), ("tied", c_int), ("k_normed", c_void_p),
+                ("ld_k_normed", c_longlong)]
 
 
 class AttentionArgs(ctypes.Structure):
@@ -252,7 +258,8 @@ class AttentionArgs(ctypes.Structure):
                 ("heads", c_int), ("kv_heads", c_int), ("head_dim", c_int), ("window", c_int), ("scale", c_float),
                 ("softcap", c_float), ("slopes", c_void_p), ("value_dim", c_int), ("sinks", c_void_p),
                 ("gate", c_void_p), ("ldg", c_longlong), ("weight_bias", c_void_p), ("chunk", c_int),
-                ("out_scale", c_float)]
+                ("out_scale", c_float), ("tied", c_int), ("key_eps", c_float), ("distance_bias", c_void_p),
+                ("bias_stride", c_int), ("bias_last", c_int), ("element_gate", c_void_p), ("ld_element_gate", c_longlong)]
 
 
 class WideNormArgs(ctypes.Structure):
@@ -260,6 +267,33 @@ class WideNormArgs(ctypes.Structure):
                 ("row_seq", c_void_p), ("row_pos", c_void_p), ("seq_slot", c_void_p), ("seq_start", c_void_p),
                 ("seq_len", c_void_p), ("k_cache", c_void_p), ("v_cache", c_void_p), ("cache", CacheGeometry),
                 ("heads", c_int), ("kv_heads", c_int), ("head_dim", c_int), ("value_dim", c_int), ("eps", c_float)]
+
+
+class DistanceBias:
+    """What is added to the score of a key n positions back, by head: `table` float32 [heads, before + count + behind], entry
+    n of head h at [h, before + n] for n < count; a larger n takes the last entry. The rows are padded on both sides (with
+    zeros before and the last entry behind) so that a kernel may read a tile's worth of entries without looking where they
+    end."""
+
+    BEFORE, BEHIND = 128, 384
+
+    def __init__(self, by_distance: torch.Tensor):
+        """`by_distance` [count, heads], count >= 1."""
+        if by_distance.dim() != 2 or by_distance.shape[0] < 1:
+            raise invalid_argument("a distance bias has a row for every distance")
+        rows = by_distance.float().t()
+        self.heads, self.count = rows.shape
+        self.table = torch.cat([rows.new_zeros(self.heads, self.BEFORE), rows,
+                                rows[:, -1:].expand(self.heads, self.BEHIND)], dim=1).contiguous()
+        self.table_log2 = (self.table.double() * 1.4426950408889634).float().contiguous()
+
+    def fields(self, heads: int, log2: bool = False) -> tuple:
+        """(address of head 0's entry 0, floats from one head to the next, the last entry) for a kernel's arguments; `log2`:
+        of the table in base-2 exponent units."""
+        if heads != self.heads:
+            raise invalid_argument("a distance bias has a row for every query head")
+        _need_cuda(self.table)
+        return (self.table_log2 if log2 else self.table).data_ptr() + 4 * self.BEFORE, self.table.shape[1], self.count - 1
 
 
 def cache_geometry(view, kv_heads: int, head_dim: int) -> CacheGeometry:
@@ -748,23 +782,32 @@ def gemm_simt(x: torch.Tensor, weight: torch.Tensor, out_dtype: torch.dtype,
 def rope_store(qkv: torch.Tensor, *, heads: int, kv_heads: int, head_dim: int, q_norm: Optional[torch.Tensor],
                k_norm: Optional[torch.Tensor], eps: float, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor],
                rotary_dim: int, tables, kv_view, store: bool, transform: bool = True,
-               value_dim: Optional[int] = None, q_scale: Optional[torch.Tensor] = None) -> None:
+               value_dim: Optional[int] = None, q_scale: Optional[torch.Tensor] = None, tied: bool = False,
+               k_normed: Optional[torch.Tensor] = None) -> None:
     """In place on qkv [rows, (heads + kv_heads) * head_dim + kv_heads * value_dim (+ columns that are left
     alone)]: per-head RMSNorm and rotation of the q and k heads; k and v heads are also written to the cache when
     `store` is set. With `transform=False` nothing is normalised or rotated: the k and v
     heads are only copied to the cache. `tables` is the step's `DeviceTables`. `value_dim` (default head_dim) is
     the width of a v head. `q_scale` (float32 [positions]): a q head at position p is multiplied by q_scale[p] after
     its norm and rotation. With `kv_heads` 0 the rows hold q heads only (a layer that reads another layer's keys
-    and values) and nothing is stored."""
-    _need_cuda(qkv)
+    and values) and nothing is stored. `tied`: a value is its key before the norm; the rows hold q heads and k heads, the
+    k heads stay as they are and are all that the cache keeps, `k_normed` ([rows, kv_heads * head_dim], if given) takes them
+    divided by their root mean squares, and q_norm is the product of both norms' weights."""
+    _need_cuda(qkv, k_normed)
     rows = qkv.shape[0]
     value_dim = head_dim if value_dim is None else int(value_dim)
-    if qkv.dim() != 2 or qkv.stride(1) != 1 or qkv.shape[1] < (heads + kv_heads) * head_dim + kv_heads * value_dim:
+    values = 0 if tied else kv_heads * value_dim
+    if tied and (value_dim != head_dim or cos is not None or q_scale is not None or kv_heads <= 0):
+        raise invalid_argument("rope_store: values that are keys come without a rotation and with a key's width")
+    if k_normed is not None and (not tied or k_normed.shape != (rows, kv_heads * head_dim) or k_normed.dtype != qkv.dtype
+                                 or not k_normed.is_contiguous()):
+        raise invalid_argument("rope_store: the normed keys have the wrong shape or type")
+    if qkv.dim() != 2 or qkv.stride(1) != 1 or qkv.shape[1] < (heads + kv_heads) * head_dim + values:
         raise invalid_argument("rope_store: qkv has the wrong shape")
-    if (q_norm is None) != (k_norm is None):
+    if not tied and (q_norm is None) != (k_norm is None):
         raise invalid_argument("rope_store: q_norm and k_norm come together")
     norm_dtype = q_norm.dtype if q_norm is not None else torch.float32
-    if q_norm is not None and (q_norm.shape != (head_dim,) or k_norm.shape != (head_dim,) or k_norm.dtype != norm_dtype):
+    if q_norm is not None and (q_norm.shape != (head_dim,) or (not tied and (k_norm.shape != (head_dim,) or k_norm.dtype != norm_dtype))):
         raise invalid_argument("rope_store: the head norms must have head_dim elements and one type")
     if cos is not None and (cos.dtype != torch.float32 or cos.shape[1] != rotary_dim // 2 or sin.shape != cos.shape):
         raise invalid_argument("rope_store: the rotation tables must be float32 [positions, rotary_dim/2]")
@@ -777,9 +820,10 @@ def rope_store(qkv: torch.Tensor, *, heads: int, kv_heads: int, head_dim: int, q
         qkv.data_ptr(), qkv.stride(0), _ptr(q_norm), _ptr(k_norm), _ptr(cos), _ptr(sin),
         tables.row_seq.data_ptr(), tables.row_pos.data_ptr(), tables.seq_slot.data_ptr(),
         tables.seq_start.data_ptr(), tables.seq_len.data_ptr(),
-        view.keys.data_ptr() if view is not None else 0, view.values.data_ptr() if view is not None else 0,
+        view.keys.data_ptr() if view is not None else 0, view.values.data_ptr() if view is not None and not tied else 0,
         cache_geometry(view, kv_heads, head_dim), rows, heads, kv_heads, head_dim, rotary_dim, float(eps),
-        1 if transform else 0, value_dim, _ptr(q_scale))
+        1 if transform else 0, value_dim, _ptr(q_scale), 1 if tied else 0, _ptr(k_normed),
+        k_normed.stride(0) if k_normed is not None else 0)
     _check(core().kidi_rope_store(ctypes.byref(args), dtype_code(qkv.dtype), dtype_code(norm_dtype), _stream()),
            "rope_store")
 
@@ -811,7 +855,8 @@ def attention_generic(qkv: torch.Tensor, out: torch.Tensor, *, heads: int, kv_he
                       softcap: float = 0.0, slopes: Optional[torch.Tensor] = None, value_dim: Optional[int] = None,
                       sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
                       weight_bias: Optional[torch.Tensor] = None, chunk: Optional[int] = None,
-                      out_scale: float = 1.0) -> None:
+                      out_scale: float = 1.0, tied: bool = False, key_eps: float = 0.0, distance_bias=None,
+                      element_gate: Optional[torch.Tensor] = None) -> None:
     """Causal attention of every row of the step over its sequence's keys. Keys of the
     step's own rows are read from `qkv` when `keys_in_step` is set, earlier ones (or
     all of them) from the cache. `softcap` > 0 bounds a score s to softcap * tanh(s / softcap);
@@ -820,7 +865,10 @@ def attention_generic(qkv: torch.Tensor, out: torch.Tensor, *, heads: int, kv_he
     [heads]): exp(sinks[h]) joins head h's softmax denominator. `gate` ([rows, heads], a view of the step's
     element type): head h of a row is multiplied by sigmoid(gate[row, h]). `weight_bias` (float32 [heads]): a key's
     weight is sigmoid(score + weight_bias[h]), normalised over nothing, instead of its share of a softmax. `chunk`: only
-    keys of the query's own run of `chunk` positions (counted from 0) are seen. `out_scale`: a factor on the result."""
+    keys of the query's own run of `chunk` positions (counted from 0) are seen. `out_scale`: a factor on the result.
+    `tied`: the k heads of qkv and of the cache are keys before their norm and the values too; a score takes the factor
+    1 / sqrt(mean square of the key + `key_eps`). `distance_bias`: a `DistanceBias`. `element_gate` ([rows, heads *
+    value_dim], a view of the step's element type): the result is multiplied by its sigmoid."""
     value_dim = head_dim if value_dim is None else int(value_dim)
     if sinks is not None and (sinks.dtype != torch.float32 or sinks.shape != (heads,) or not sinks.is_contiguous()
                               or sinks.device != qkv.device):
@@ -841,16 +889,21 @@ def attention_generic(qkv: torch.Tensor, out: torch.Tensor, *, heads: int, kv_he
         raise invalid_argument("attention: there is neither a cache nor keys in the step")
     item = qkv.element_size()
     k_step = qkv.data_ptr() + heads * head_dim * item if keys_in_step else 0
-    v_step = qkv.data_ptr() + (heads + kv_heads) * head_dim * item if keys_in_step else 0
+    v_step = (k_step if tied else qkv.data_ptr() + (heads + kv_heads) * head_dim * item) if keys_in_step else 0
+    if element_gate is not None and (element_gate.shape != out.shape or element_gate.dtype != qkv.dtype
+                                     or element_gate.stride(1) != 1):
+        raise invalid_argument("attention: the gate per element has the result's shape and type")
+    values = (kv_view.keys if tied else kv_view.values).data_ptr() if kv_view is not None else 0
     args = AttentionArgs(
         qkv.data_ptr(), qkv.stride(0), k_step, v_step, qkv.stride(0),
-        kv_view.keys.data_ptr() if kv_view is not None else 0, kv_view.values.data_ptr() if kv_view is not None else 0,
+        kv_view.keys.data_ptr() if kv_view is not None else 0, values,
         cache_geometry(kv_view, kv_heads, head_dim), out.data_ptr(), out.stride(0),
         tables.row_seq.data_ptr(), tables.row_pos.data_ptr(), tables.seq_slot.data_ptr(),
         tables.seq_start.data_ptr(), tables.seq_row0.data_ptr(), rows, heads, kv_heads, head_dim,
         int(window or 0), float(scale), float(softcap or 0.0), slopes.data_ptr() if slopes is not None else 0,
         value_dim, _ptr(sinks), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(weight_bias), int(chunk or 0),
-        float(out_scale))
+        float(out_scale), 1 if tied else 0, float(key_eps), *(distance_bias.fields(heads) if distance_bias is not None else (0, 0, 0)),
+        _ptr(element_gate), element_gate.stride(0) if element_gate is not None else 0)
     _check(core().kidi_attention_generic(ctypes.byref(args), dtype_code(qkv.dtype), _stream()), "attention")
 
 

@@ -2,6 +2,7 @@
 feed-forward first runs."""
 from __future__ import annotations
 
+import ctypes
 from typing import Optional
 
 import torch
@@ -19,13 +20,15 @@ def library():
     if _library is None:
         lib = load_library("routed")
         lib.kidi_route.argtypes = [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                   c_int, c_int, c_int, c_float, c_void_p, c_void_p]
+                                   c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p,
+                                   c_void_p]
         lib.kidi_expert_slots.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
-                                          c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p]
+                                          c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p,
+                                          c_void_p, c_void_p]
         lib.kidi_gather_slots.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                           c_void_p]
         lib.kidi_combine_slots.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                                           c_void_p, c_void_p]
+                                           c_void_p, c_void_p, c_void_p]
         lib.kidi_group_slots.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p]
         lib.kidi_group_slots_rows.argtypes = [c_int, c_int]
         for name in ("kidi_group_slots", "kidi_group_slots_rows", "kidi_route", "kidi_expert_slots", "kidi_gather_slots", "kidi_combine_slots"):
@@ -41,15 +44,24 @@ def _check_addend(addend, like: torch.Tensor, rows: int, hidden: int) -> None:
 
 
 def route(x: torch.Tensor, router: torch.Tensor, top: int, renormalise: bool, score: str = "sigmoid", groups: int = 1,
-          keep: int = 1, renormalise_eps: float = 0.0, bias: Optional[torch.Tensor] = None):
+          keep: int = 1, renormalise_eps: float = 0.0, bias: Optional[torch.Tensor] = None,
+          correction: Optional[torch.Tensor] = None, two_largest: bool = False, weight_scale: float = 1.0,
+          share_row: Optional[torch.Tensor] = None, share: Optional[torch.Tensor] = None):
     """(chosen int32 [rows, top], weight float32 [rows, top]) for rows x [rows, hidden] and a router
     [experts, hidden]: logits in 32-bit, scores (a sigmoid of each logit, or with `score` "softmax" a softmax over
     all experts), the `top` largest (ties: the lower index), their scores as weights (with `renormalise` divided by
     their sum plus `renormalise_eps`). With `groups` > 1 the experts form that many equal runs of neighbours and
     only experts of the `keep` groups with the largest best score can be chosen. `bias` (float32 [experts]) is added
-    to the logits."""
-    ops._need_cuda(x, router, bias)
+    to the logits. `correction` (float32 [experts]) is added to the scores that choose experts and groups, not to the
+    weights; `two_largest`: a group's score is the sum of its two largest; the weights are multiplied by `weight_scale`.
+    `share` (float32 [rows], with `share_row` [1, hidden] in the router's type) takes sigmoid(share_row . x)."""
+    ops._need_cuda(x, router, bias, correction, share_row, share)
     ops._float_vector(bias, router.shape[0], "the router's bias")
+    ops._float_vector(correction, router.shape[0], "the router's correction")
+    if share is not None:
+        ops._float_vector(share, x.shape[0], "the shared expert's part")
+        if share_row is None or share_row.numel() != x.shape[1] or share_row.dtype != router.dtype or not share_row.is_contiguous():
+            raise invalid_argument("the shared expert's gate is a row of the router's type")
     if x.dim() != 2 or not x.is_contiguous() or router.dim() != 2 or not router.is_contiguous() \
             or router.shape[1] != x.shape[1]:
         raise invalid_argument("the router takes contiguous rows and a contiguous [experts, hidden] matrix")
@@ -59,19 +71,23 @@ def route(x: torch.Tensor, router: torch.Tensor, top: int, renormalise: bool, sc
     _check(library().kidi_route(x.data_ptr(), dtype_code(x.dtype), router.data_ptr(), dtype_code(router.dtype),
                                 chosen.data_ptr(), weight.data_ptr(), rows, hidden, router.shape[0], top,
                                 1 if renormalise else 0, 1 if score == "softmax" else 0, int(groups), int(keep),
-                                float(renormalise_eps), bias.data_ptr() if bias is not None else 0, ops._stream()),
+                                float(renormalise_eps), bias.data_ptr() if bias is not None else 0,
+                                correction.data_ptr() if correction is not None else 0, 1 if two_largest else 0,
+                                float(weight_scale), share_row.data_ptr() if share is not None else 0,
+                                share.data_ptr() if share is not None else 0, ops._stream()),
            "route")
     return chosen, weight
 
 
 def expert_slots(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, chosen: torch.Tensor,
                  weight: torch.Tensor, weight_on_input: bool, gated: bool = True,
-                 addend=None) -> torch.Tensor:
+                 addend=None, shape: Optional[ops.GateShape] = None, share: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Every row through its chosen experts, the experts' weights read through the choice: x [rows, hidden],
     gate_up [experts, 2 * inter, hidden] (without a gate: the up rows only, [experts, inter, hidden], and the
     exact gelu as activation), down [experts, hidden, inter] -> [rows, hidden]. `addend` [rows, hidden], if given, is
     added to the result (in 32-bit, before it is rounded); it may be a function that returns it (or None), which is
-    called between the two kernels."""
+    called between the two kernels; `share` (float32 [rows]): the addend's rows are multiplied by it. `shape`: another
+    activation of gated experts than SiLU."""
     ops._need_cuda(x, gate_up, down, chosen, weight)
     rows, hidden = x.shape
     experts, first_rows, _ = gate_up.shape
@@ -90,6 +106,7 @@ def expert_slots(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, cho
             x.data_ptr(), dtype_code(x.dtype), gate_up.data_ptr(), down.data_ptr(), dtype_code(gate_up.dtype),
             chosen.data_ptr(), weight.data_ptr(), mid.data_ptr(), out.data_ptr(), rows, top, hidden, inter,
             1 if weight_on_input else 0, 1 if gated else 0, addend.data_ptr() if addend is not None else 0, parts,
+            ctypes.byref(shape) if shape is not None else None, share.data_ptr() if share is not None else 0,
             ops._stream()), what, launches)
 
     if later is None:
@@ -140,14 +157,16 @@ def gather_slots(x: torch.Tensor, order: torch.Tensor, weight: torch.Tensor, top
 
 
 def combine_slots(y: torch.Tensor, place: torch.Tensor, weight: torch.Tensor, rows: int, top: int,
-                  weight_on_input: bool, addend: Optional[torch.Tensor] = None) -> torch.Tensor:
+                  weight_on_input: bool, addend: Optional[torch.Tensor] = None,
+                  share: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[r] = sum over k of y[place[r * top + k]] (times weight[r, k] when the weight is on the output), plus
-    addend[r] if given."""
+    addend[r] if given (times share[r], float32, if given)."""
     hidden = y.shape[1]
     _check_addend(addend, y, rows, hidden)
     out = torch.empty((rows, hidden), dtype=y.dtype, device=y.device)
     _check(library().kidi_combine_slots(y.data_ptr(), dtype_code(y.dtype), place.data_ptr(), weight.data_ptr(),
                                         out.data_ptr(), rows, top, hidden, 1 if weight_on_input else 0,
-                                        addend.data_ptr() if addend is not None else 0, ops._stream()),
+                                        addend.data_ptr() if addend is not None else 0,
+                                        share.data_ptr() if share is not None else 0, ops._stream()),
            "combine_slots")
     return out

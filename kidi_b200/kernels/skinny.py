@@ -24,7 +24,7 @@ class Extras(ctypes.Structure):
                 ("factor_width", c_int), ("factor_eps", c_float), ("residual", c_void_p), ("ld_residual", c_longlong),
                 ("norm_weight", c_void_p), ("norm_weight_is_float", c_int), ("normed", c_void_p),
                 ("ld_normed", c_longlong), ("parts_out", c_void_p), ("parts_stride", c_int), ("gelu", c_int),
-                ("silu_begin", c_int), ("silu_end", c_int)]
+                ("silu_begin", c_int), ("silu_end", c_int), ("gate", ops.GateShape)]
 
 
 _bound = False
@@ -143,8 +143,9 @@ def gemm_into_residual(x: torch.Tensor, weight: torch.Tensor, residual: torch.Te
 
 
 def gemm_silu_gate(x: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Tensor] = None,
-                   row_tiles: int = 0, factors=None) -> torch.Tensor:
-    """silu(x @ Wg.T) * (x @ Wu.T) for weight = [Wg; Wu] of shape [2I, K] (`factors`: as in `gemm`)."""
+                   row_tiles: int = 0, factors=None, shape: Optional[ops.GateShape] = None) -> torch.Tensor:
+    """silu(x @ Wg.T) * (x @ Wu.T) for weight = [Wg; Wu] of shape [2I, K] (`factors`: as in `gemm`; `shape`: another
+    activation than SiLU)."""
     _need_cuda(x, weight)
     if not supports(x, weight) or x.shape[1] != weight.shape[1] or weight.shape[0] % 2:
         raise invalid_argument("gemm_silu_gate: the operands do not fit this kernel")
@@ -154,8 +155,10 @@ def gemm_silu_gate(x: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Te
         out = torch.empty((M, inter), dtype=torch.bfloat16, device=x.device)
     extras = Extras()
     _factor_fields(extras, factors)
+    if shape is not None:
+        extras.gate = shape
     _check(_library().kidi_gemm_skinny(_ptr(x), _ptr(weight), _ptr(out), dtype_code(out.dtype), M, inter, K,
                                        x.stride(0), weight.stride(0), out.stride(0), 1, row_tiles, None,
                                        ctypes.byref(extras), _stream()),
-           "gemm_silu_gate[skinny]")
+           "gemm_bounded_gate[skinny]" if shape is not None and shape.bounded else "gemm_silu_gate[skinny]")
     return out

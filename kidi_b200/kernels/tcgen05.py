@@ -16,6 +16,7 @@ from 17 rows on, except weights as tall as an output head (KIDI_B200_TCGEN05_MAX
 """
 from __future__ import annotations
 
+import ctypes
 import os
 from typing import Dict, Optional
 
@@ -54,7 +55,7 @@ def _library():
                                           c_void_p, c_void_p]
         lib.kidi_gemm_tcgen05.restype = c_int
         lib.kidi_gemm_tcgen05_grouped.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong,
-                                                  c_int, c_int, c_void_p, c_void_p, c_void_p]
+                                                  c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p]
         lib.kidi_gemm_tcgen05_grouped.restype = c_int
         lib.kidi_gemm_tcgen05_token_tile.argtypes = [c_int]
         lib.kidi_gemm_tcgen05_token_tile.restype = c_int
@@ -147,10 +148,11 @@ def gemm_silu_gate(x: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Te
 GROUP_TILE = 128                        # rows of a tile of a grouped product
 
 
-def gemm_grouped(x: torch.Tensor, weight: torch.Tensor, group_of_tile: torch.Tensor, gated: bool) -> torch.Tensor:
+def gemm_grouped(x: torch.Tensor, weight: torch.Tensor, group_of_tile: torch.Tensor, gated: bool,
+                 shape: Optional[ops.GateShape] = None) -> torch.Tensor:
     """A product with weights in groups: rows 128 i .. 128 i + 127 of x [rows, K] take weight[group_of_tile[i]] of
     weight [groups, features, K] (`gated`: [groups, 2 * features, K], gate rows first, and the result is silu(gate) * up);
-    bfloat16. Rows of tiles whose group (int32) is negative are not written."""
+    bfloat16. Rows of tiles whose group (int32) is negative are not written. `shape`: another activation than SiLU."""
     _need_cuda(x, weight, group_of_tile)
     groups, height, K = weight.shape
     rows = x.shape[0]
@@ -163,6 +165,7 @@ def gemm_grouped(x: torch.Tensor, weight: torch.Tensor, group_of_tile: torch.Ten
     _, _, error = _device_state(x.device)
     _check(_library().kidi_gemm_tcgen05_grouped(
         _ptr(x), _ptr(weight), _ptr(out), rows, features, K, x.stride(0), out.stride(0), 1 if gated else 0, groups,
-        _ptr(group_of_tile), _ptr(error), _stream()),
-        "gemm_silu_gate[tcgen05, groups]" if gated else "gemm_tcgen05[groups]")
+        _ptr(group_of_tile), _ptr(error), ctypes.byref(shape) if shape is not None else None, _stream()),
+        "gemm_bounded_gate[tcgen05, groups]" if gated and shape is not None and shape.bounded
+        else "gemm_silu_gate[tcgen05, groups]" if gated else "gemm_tcgen05[groups]")
     return out

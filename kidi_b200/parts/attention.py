@@ -44,6 +44,13 @@ of those sizes, float32 arithmetic, tensors q_norm_name and k_norm_name); weight
 the weight of a key is sigmoid(score + b), b a number per head from the tensor `weight_bias_name`, and the weights are
 not normalised over the keys); out_scale (a factor on the concatenated heads, default 1).
 
+And: values_from_keys (bool): there is no value projection, a value is its key as projected (bias included) before the key
+norm (with qk_norm per head, without a rotation). The cache then keeps one row per token and key/value head, the key before
+its norm: with r_u = 1 / sqrt(mean(k_u^2) + eps) a score is r_u ((w_q w_k N(q)) . k_u) scale, so both norms' weights ride in
+q, and the attention kernels form r_u themselves from the row they read anyway. distance_bias_reach (None: none): the
+tensor `distance_bias_name` [buckets, num_heads] (its height is the checkpoint's choice) holds a number per bucket of
+distance (`distance_buckets`) that is added to a score after the scale. sink_score (None: none): a sink as above whose score is that number for every head, without a tensor.
+
 The part can also run on projections that another part holds (`joint_input`, `mix`, `joint_output`; see
 `parallel_mixers`).
 """
@@ -60,6 +67,7 @@ from ..kernels import ops
 from ..kernels.attention import AttentionLauncher, reach_of
 from .base import Part
 from .linear import Linear
+from .position import distance_buckets
 from .registry import register_part
 from .spec import ParamSpec
 
@@ -93,7 +101,12 @@ class Attention(Part):
             ("q", "q_proj.weight"), ("k", "k_proj.weight"), ("v", "v_proj.weight"), ("o", "o_proj.weight"),
             ("sink", "sinks"), ("gate", "gate_proj.weight"), ("q_bias", "q_proj.bias"), ("k_bias", "k_proj.bias"),
             ("v_bias", "v_proj.bias"), ("q_norm", "q_norm.weight"), ("k_norm", "k_norm.weight"),
-            ("weight_bias", "weight_bias"))}
+            ("weight_bias", "weight_bias"), ("distance_bias", "distance_bias"))}
+        self.tied = bool(spec.param("values_from_keys", False))
+        self.bias_reach = spec.param("distance_bias_reach", None)
+        self.bias_buckets = int(spec.param("distance_bias_buckets", 32))      # what random weights get
+        self.distance_bias: Optional[ops.DistanceBias] = None
+        self.sink_score = spec.param("sink_score", None)
         self.chunk = spec.param("chunk", None)
         self.wide_norm = self.qk_norm and spec.param("qk_norm_scope", "head") == "rows"
         if spec.param("qk_norm_scope", "head") not in ("head", "rows"):
@@ -116,13 +129,23 @@ class Attention(Part):
             raise unsupported("sigmoid weights with a sink or a gate per head are not built")
         if self.wide_norm and not (self.own_kv and self.norm_weight):
             raise unsupported("a norm over whole rows of queries and keys needs both projections and both weights")
+        if self.sink_score is not None and self.has_sink:
+            raise invalid_argument("a sink has a number per head from a tensor or one fixed number, not both")
+        if self.sigmoid and self.sink_score is not None:
+            raise unsupported("sigmoid weights with a sink are not built")
+        if self.tied and (not self.own_kv or self.value_dim != self.head_dim or not self.qk_norm or self.wide_norm
+                          or spec.param("position", None) is not None or spec.param("query_scale", None) is not None):
+            raise unsupported("values that are keys before their norm need a norm per head of queries and keys, values as wide "
+                              "as keys and no rotation")
+        if self.bias_reach is not None and int(self.bias_reach) <= 0:
+            raise invalid_argument("the reach of a distance bias must be positive")
         name = spec.param("position", None)
         self.position = env.positions[name] if name is not None else None
         if self.position is not None and self.position.head_dim != self.head_dim:
             raise invalid_argument("the rotary encoding was built for another head width")
         self.q_width = self.heads * self.head_dim
         self.kv_width = self.kv_heads * self.head_dim
-        self.v_width = self.kv_heads * self.value_dim
+        self.v_width = 0 if self.tied else self.kv_heads * self.value_dim
         self.out_width = self.heads * self.value_dim
         # The fused projection's rows: q, k, v, then one gate row a head, then zero rows up to a multiple of 8
         # (so that the rows of its result start on 16-byte boundaries).
@@ -131,7 +154,8 @@ class Attention(Part):
         self.fused_width = self.gate_begin + self.gate_width
         scale_name = spec.param("query_scale", None)
         self.query_scale = env.positions[scale_name] if scale_name is not None else None
-        self.sinks = None
+        self.sinks = torch.full((self.heads,), float(self.sink_score), dtype=torch.float32, device=env.device) \
+            if self.sink_score is not None else None
         self.qkv: Optional[Linear] = None
         self.out: Optional[Linear] = None
         self.q_norm = self.k_norm = None
@@ -148,15 +172,19 @@ class Attention(Part):
         self.launcher = AttentionLauncher(heads=self.heads, kv_heads=self.kv_heads, head_dim=self.head_dim,
                                           scale=self.scale, window=self.window, softcap=self.softcap,
                                           slopes=self.slopes, chunk=self.chunk,
-                                          out_scale=float(spec.param("out_scale", 1.0)))
+                                          out_scale=float(spec.param("out_scale", 1.0)), tied=self.tied,
+                                          biased=self.bias_reach is not None, key_eps=self.eps)
 
     def parameter_specs(self) -> List[ParamSpec]:
         n = self.names
         sources = [(n["q"], (self.q_width, self.hidden))]
         biases = [(n["q_bias"], (self.q_width,))]
         if self.own_kv:
-            sources += [(n["k"], (self.kv_width, self.hidden)), (n["v"], (self.v_width, self.hidden))]
-            biases += [(n["k_bias"], (self.kv_width,)), (n["v_bias"], (self.v_width,))]
+            sources.append((n["k"], (self.kv_width, self.hidden)))
+            biases.append((n["k_bias"], (self.kv_width,)))
+        if self.own_kv and not self.tied:
+            sources.append((n["v"], (self.v_width, self.hidden)))
+            biases.append((n["v_bias"], (self.v_width,)))
         if self.gate_width:
             sources.append((n["gate"], (self.gate_width, self.hidden)))
         specs = [
@@ -175,6 +203,8 @@ class Attention(Part):
             specs.append(ParamSpec(n["weight_bias"], (self.heads,), init=("normal", 1.0)))
         if self.has_sink:
             specs.append(ParamSpec(n["sink"], (self.heads,), init=("normal", 1.0)))
+        if self.bias_reach is not None:
+            specs.append(ParamSpec(n["distance_bias"], (self.bias_buckets, self.heads), init=("normal", 0.5), open_axes=(0,)))
         return specs
 
     def bind(self, tensors) -> None:
@@ -194,6 +224,13 @@ class Attention(Part):
             self.q_norm, self.k_norm = tensors[self.names["q_norm"]], tensors[self.names["k_norm"]]
             if self.wide_norm or self.q_norm.dtype != self.k_norm.dtype:
                 self.q_norm, self.k_norm = self.q_norm.float(), self.k_norm.float()
+        if self.tied:                  # both weights ride in q (formed once, in 32-bit)
+            self.q_norm, self.k_norm = (self.q_norm.float() * self.k_norm.float()).contiguous(), None
+        if self.bias_reach is not None:
+            by_bucket = tensors[self.names["distance_bias"]]
+            reach, seen = int(self.bias_reach), reach_of(self.window, self.chunk) or self.env.max_positions
+            buckets = distance_buckets(min(seen, reach + 1), by_bucket.shape[0], reach)
+            self.distance_bias = ops.DistanceBias(by_bucket.float()[buckets.to(by_bucket.device)])
         if self.has_sink:
             self.sinks = tensors[self.names["sink"]].float().contiguous()
         if self.sigmoid:
@@ -201,6 +238,8 @@ class Attention(Part):
 
     def cache_requests(self) -> list:
         window = reach_of(self.window, self.chunk) if self.ring else None
+        if self.tied:                  # the keys before their norm are all that is kept
+            return [KVRequest(self.kv_heads, self.head_dim, window, value_dim=0)]
         return [KVRequest(self.kv_heads, self.head_dim, window,
                           value_dim=self.value_dim if self.value_dim != self.head_dim else None)]
 
@@ -245,8 +284,10 @@ class Attention(Part):
                       value_dim=self.value_dim)
         ring = view.ring_pages > 0
         extras = {}
-        if self.has_sink:
+        if self.sinks is not None:
             extras["sinks"] = self.sinks
+        if self.distance_bias is not None:
+            extras["distance_bias"] = self.distance_bias
         if self.has_gate:
             extras["gate"] = qkv[:, self.gate_begin:self.gate_begin + self.heads]
         if self.value_dim != self.head_dim:
@@ -264,6 +305,16 @@ class Attention(Part):
         fused = owns_cache and store_first and self.value_dim == self.head_dim and self.query_scale is None \
             and not self.wide_norm \
             and self.launcher.fuses_rotation(plan, qkv, kv_view=view, q_norm=self.q_norm, k_norm=self.k_norm, **rotate)
+        # Whether the attention kernel multiplies by the gate itself.
+        gate = qkv[:, self.gate_begin:self.gate_begin + self.out_width] if self.output_gate else None
+        gated_inside = gate is not None and (self.tied or self.distance_bias is not None)
+        if gated_inside:
+            extras["element_gate"] = gate
+        if self.tied:
+            common["tied"] = True
+            if not fused and self.launcher.wants_normed_keys(plan, qkv, kv_view=view):
+                common["k_normed"] = extras["k_normed"] = torch.empty((qkv.shape[0], self.kv_width), dtype=qkv.dtype,
+                                                                      device=qkv.device)
         if self.wide_norm:
             plain = position is None and self.query_scale is None
             ops.wide_norm_store(qkv, q_norm=self.q_norm, k_norm=self.k_norm, eps=self.eps, tables=ctx.tables, kv_view=view,
@@ -283,7 +334,8 @@ class Attention(Part):
                           step_rows_cached=store_first and not fused, q_only=not self.own_kv, **extras)
         if owns_cache and not store_first:
             ops.rope_store(qkv, q_norm=None, k_norm=None, eps=self.eps, tables=ctx.tables, kv_view=view, store=True,
-                           transform=False, cos=None, sin=None, rotary_dim=0, **common)
-        if self.output_gate:
-            ops.sigmoid_gate(attended, qkv[:, self.gate_begin:self.gate_begin + self.out_width])
+                           transform=False, cos=None, sin=None, rotary_dim=0,
+                           **{name: value for name, value in common.items() if name != "k_normed"})
+        if gate is not None and not gated_inside:
+            ops.sigmoid_gate(attended, gate)
         return attended

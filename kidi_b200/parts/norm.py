@@ -8,7 +8,8 @@ stream takes its pending delta: sum and normalisation run in one kernel, in 32-b
 Parameters of `rms_norm`: size, eps, weight_name (the tensor's name under the prefix, default "weight") and
 weight_offset (default 0): the stored tensor plus this number is the weight, so a weight that a model stores
 around zero has weight_offset 1: y = x / sqrt(mean(x^2) + eps) * (1 + w). `groups` (default 1): the row is split into
-that many equal consecutive parts and each is divided by its own root mean square before the weight.
+that many equal consecutive parts and each is divided by its own root mean square before the weight. `fold` (default: true
+without a weight_offset): whether the product before the norm may prepare its rows (`prepared_weight`).
 
 The norm can also stand behind a sublayer, x <- x + norm(sublayer(...)): what reads the stream next normalises the
 sublayer's result and adds it in its own kernel (`delta_parts`, `apply_delta`).
@@ -35,6 +36,7 @@ class RMSNorm(Part):
         self.weight_name = spec.param("weight_name", "weight")
         self.offset = float(spec.param("weight_offset", 0.0))
         self.groups = int(spec.param("groups", 1))
+        self.fold = bool(spec.param("fold", not self.offset))
         if self.groups < 1 or self.size % self.groups:
             raise invalid_argument("a norm's rows split into equal parts")
         self.weight: Optional[torch.Tensor] = None
@@ -64,7 +66,7 @@ class RMSNorm(Part):
     def prepared_weight(self) -> Optional[torch.Tensor]:
         """The weight vector a product needs to prepare rows for this norm (`ResidualSink`), or
         None when this norm does not take prepared rows."""
-        return self.weight if self.env.dtype == torch.bfloat16 and not self.offset and self.groups == 1 else None
+        return self.weight if self.env.dtype == torch.bfloat16 and self.fold and self.groups == 1 else None
 
     reads_lanes = True            # a stream kept as several lanes is read as a weighted sum of them
 

@@ -14,6 +14,9 @@ over that length; pairs that turn more often than `fast` keep their frequency, p
     ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1),   f_i <- f_i / factor * ramp_i + f_i (1 - ramp_i)
 and cosine and sine are both multiplied by 0.1 ln(factor) + 1.
 
+With `angles64` the frequencies and angles are 64-bit and only the cosines and sines are rounded to 32-bit (a 32-bit angle is
+off by 6e-5 at a thousand turns' worth of position).
+
 `learned_positions` is a table with a vector per position that is added to the embeddings
 (times `scale`, default 1), in 32-bit; mixers read nothing from it. Parameters: hidden_size,
 max_positions, scale, name (the table's tensor name under the prefix, default "weight").
@@ -22,11 +25,16 @@ max_positions, scale, name (the table's tensor name under the prefix, default "w
 layer's `query_scale`): 1 + coef * ln(floor((p + 1) / every) + 1) at position p, so that scores sharpen step by
 step as a sequence grows. Parameters: coef, every, max_positions. The table is 32-bit, built once.
 
+`distance_buckets` is no part but a function: the bucket of every distance for a learned bias of B numbers, the first half
+of them one distance each, the second half spread over the logarithm of the distance up to a `reach`.
+
 Interface of a position encoding: `on_embeddings(stream, ctx)` (may change the
 embeddings; rotary does nothing there) and whatever its mixers agree to read from it
 (`cos`, `sin`, `rotary_dim` here).
 """
 from __future__ import annotations
+
+import math
 
 import torch
 
@@ -37,6 +45,23 @@ from .registry import register_part
 from .spec import ParamSpec
 
 
+def distance_buckets(count: int, buckets: int, reach: int) -> torch.Tensor:
+    """int64 [count]: the bucket of distances 0 .. count - 1. With B buckets and h = B // 2 a distance n < h has bucket n, any
+    other min(B - 1, h + floor(ln(n / h) / ln(reach / h) (B - h))). The logarithms are 64-bit; where n is an exact power the
+    quotient is the whole number it stands for, whatever the logarithms round to."""
+    half = buckets // 2
+    if buckets < 1 or not reach > half:
+        raise invalid_argument(f"{buckets} distance buckets must reach further than {half} positions, not {reach}")
+    if half == 0:
+        return torch.zeros(count, dtype=torch.int64)
+    distance = torch.arange(count, dtype=torch.float64)
+    place = torch.log(distance.clamp(min=half) / half) / math.log(reach / half) * (buckets - half)
+    whole = torch.round(place)
+    place = torch.where((place - whole).abs() < 1e-9, whole, torch.floor(place))
+    far = (half + place).clamp(max=buckets - 1)
+    return torch.where(distance < half, distance, far).long()
+
+
 @register_part("position", "rotary")
 class RotaryEncoding(Part):
     def __init__(self, spec, env):
@@ -45,6 +70,7 @@ class RotaryEncoding(Part):
         self.rotary_dim = int(spec.param("rotary_dim", self.head_dim))
         self.theta = float(spec.param("theta"))
         self.max_positions = int(spec.param("max_positions"))
+        self.angles64 = bool(spec.param("angles64", False))
         scaling = spec.param("scaling", None)
         self.scaling = {key: float(scaling[key]) for key in ("factor", "original", "fast", "slow")} if scaling else None
         if self.scaling is not None and (self.scaling["factor"] <= 0 or self.scaling["original"] <= 0
@@ -68,7 +94,6 @@ class RotaryEncoding(Part):
             frequency = 1.0 / power
             factor = 1.0
             if self.scaling is not None:
-                import math
                 s, n = self.scaling, float(self.rotary_dim)
                 pair = lambda turns: n * math.log(s["original"] / (2.0 * math.pi * turns)) / (2.0 * math.log(self.theta))
                 lo = max(math.floor(pair(s["fast"])), 0)
@@ -77,6 +102,13 @@ class RotaryEncoding(Part):
                 frequency = (frequency.double() / s["factor"] * ramp + frequency.double() * (1.0 - ramp)).float()
                 factor = 0.1 * math.log(s["factor"]) + 1.0
             angle = torch.arange(self.max_positions, dtype=torch.float32)[:, None] * frequency[None, :]
+            if self.angles64:
+                if self.scaling is not None:
+                    raise invalid_argument("a stretched rotary encoding has 32-bit angles")
+                exact = self.theta ** (-2.0 * torch.arange(half, dtype=torch.float64) / self.rotary_dim)
+                angle = torch.arange(self.max_positions, dtype=torch.float64)[:, None] * exact[None, :]
+                self._tables = tuple(table.float().contiguous().to(self.env.device) for table in (torch.cos(angle), torch.sin(angle)))
+                return self._tables
             self._tables = ((torch.cos(angle) * factor).contiguous().to(self.env.device),
                             (torch.sin(angle) * factor).contiguous().to(self.env.device))
         return self._tables

@@ -21,6 +21,13 @@ first stacked tensor is [experts, expert_size, hidden]; shared_size and shared_n
 of the same form and that width, under `<prefix><shared_name><gate|up|down>`, that every token passes and whose
 result is added with weight 1.
 
+And: correction_name (a tensor [experts] that is added to the scores where experts and groups are chosen, and not to the
+weights); group_score "largest" (the default) or "two_largest" (a group's score is the sum of its two largest);
+weight_scale (the weights are multiplied by it, after the renormalisation; default 1); activation "silu" (the default) or
+"bounded_swish" (a gated expert's form in `gated_mlp`, with limit, alpha and up_shift, and shared_limit for the shared
+expert); shared_gate_name (a tensor [1, hidden] under the shared expert's prefix: its result is multiplied by
+sigmoid(W_sg h), one number a token, computed beside the router's logits in 32-bit).
+
 Steps of few rows, steps inside a captured decode graph, and every step of the 32-bit engine read the
 chosen experts' weights through the choice on the device. Prompts of the bfloat16 engine group the (row,
 choice) pairs by expert on the device, gather the rows and run them through two products over groups of this
@@ -76,6 +83,26 @@ class RoutedExperts(Part):
         shared = spec.param("shared_size", None)
         self.shared_size = int(shared) if shared is not None else None
         self.shared_name = spec.param("shared_name", "shared.")
+        self.correction_name = spec.param("correction_name", None)
+        self.correction: Optional[torch.Tensor] = None
+        self.two_largest = spec.param("group_score", "largest") == "two_largest"
+        if spec.param("group_score", "largest") not in ("largest", "two_largest"):
+            raise invalid_argument("a group of experts is ranked by its largest score or the sum of its two largest")
+        self.weight_scale = float(spec.param("weight_scale", 1.0))
+        self.shared_gate_name = spec.param("shared_gate_name", None) if self.shared_size is not None else None
+        self.shared_gate: Optional[torch.Tensor] = None
+        activation = spec.param("activation", "silu")
+        if activation not in ("silu", "bounded_swish") or (activation != "silu" and not self.gated):
+            raise unsupported(f"expert activation '{activation}' is not built (gated experts: silu and bounded_swish)")
+        self.shape = self.shared_shape = None
+        if activation == "bounded_swish":
+            limits = [float(spec.param("limit"))] + ([float(spec.param("shared_limit", spec.param("limit")))]
+                                                     if self.shared_size is not None else [])
+            if not all(limit > 0 for limit in limits):
+                raise invalid_argument("the bound of a bounded gate must be positive")
+            shapes = [ops.GateShape(1, limit, float(spec.param("alpha", 1.702)), float(spec.param("up_shift", 1.0)))
+                      for limit in limits]
+            self.shape, self.shared_shape = shapes[0], shapes[-1]
         if min(self.hidden, self.inter, self.experts, self.top) <= 0 or self.top > self.experts:
             raise invalid_argument("invalid routed feed-forward dimensions")
         if self.experts > 1024 or self.top > 32:
@@ -106,6 +133,8 @@ class RoutedExperts(Part):
         specs = [ParamSpec(self.router_name, (self.experts, self.hidden)),
                  *([ParamSpec(self.router_bias_name, (self.experts,), init=("normal", 0.1))]
                    if self.router_bias_name is not None else []),
+                 *([ParamSpec(self.correction_name, (self.experts,), init=("normal", 0.1))]
+                   if self.correction_name is not None else []),
                  ParamSpec("experts.gate_up", (self.experts * per, self.hidden), sources=tuple(first)),
                  ParamSpec("experts.down", (self.experts * self.hidden, self.inter), sources=tuple(down))]
         if self.shared_size is not None:
@@ -117,6 +146,8 @@ class RoutedExperts(Part):
             else:
                 specs.append(ParamSpec(name + self.up_name, (self.shared_size, self.hidden)))
             specs.append(ParamSpec(name + self.down_name, (self.hidden, self.shared_size)))
+            if self.shared_gate_name is not None:
+                specs.append(ParamSpec(name + self.shared_gate_name, (1, self.hidden)))
         return specs
 
     def bind(self, tensors) -> None:
@@ -124,6 +155,13 @@ class RoutedExperts(Part):
         self.router = tensors[self.router_name]
         if self.router_bias_name is not None:
             self.router_bias = tensors[self.router_bias_name].float().contiguous()
+        if self.correction_name is not None:
+            self.correction = tensors[self.correction_name].float().contiguous()
+        if self.shared_gate_name is not None:       # (the row joins the router's product: in the router's type)
+            row = tensors[self.shared_name + self.shared_gate_name]
+            if row.dtype != self.router.dtype:
+                row, self.router = row.float(), self.router.float()
+            self.shared_gate = row.contiguous()
         self.gate_up = tensors["experts.gate_up"].view(self.experts, per, self.hidden)
         self.down = tensors["experts.down"].view(self.experts, self.hidden, self.inter)
         self._gate_up = [Linear(self.gate_up[index]) for index in range(self.experts)]
@@ -134,8 +172,10 @@ class RoutedExperts(Part):
             self._shared = (Linear(tensors[name + ("gate_up" if self.gated else self.up_name)]),
                             Linear(tensors[name + self.down_name]))
 
-    def _activate(self, first: torch.Tensor) -> torch.Tensor:
+    def _activate(self, first: torch.Tensor, shape=None) -> torch.Tensor:
         """The experts' activation on the first product's result (in place where it can be)."""
+        if shape is not None:
+            return ops.bounded_gate(first, shape.limit, shape.alpha, shape.shift)
         return ops.silu_gate(first) if self.gated else ops.gelu(first, out=first)
 
     def forward(self, x, ctx) -> torch.Tensor:
@@ -150,29 +190,33 @@ class RoutedExperts(Part):
     def _forward_shared(self, x) -> torch.Tensor:
         up, down = self._shared
         if skinny.fits(x, up.weight) and up.bias is None:            # few rows: the activation in the epilogue
-            mid = skinny.gemm_silu_gate(x, up.weight) if self.gated else skinny.gemm(x, up.weight, x.dtype, activation="gelu")
+            mid = skinny.gemm_silu_gate(x, up.weight, shape=self.shared_shape) if self.gated else skinny.gemm(x, up.weight, x.dtype, activation="gelu")
         else:
-            mid = self._activate(up.forward(x))
+            mid = self._activate(up.forward(x), self.shared_shape)
         return down.forward(mid)
 
     def _forward_routed(self, x, ctx, shared=lambda: None) -> torch.Tensor:
         """`shared()`: the shared expert's result (or None), asked for where the routed sum is formed."""
         rows = x.shape[0]
+        share = torch.empty(rows, dtype=torch.float32, device=x.device) if self.shared_gate is not None else None
         chosen, weight = routed.route(x, self.router, self.top, self.renormalise, self.score, self.groups,
-                                      self.keep_groups, self.renormalise_eps, self.router_bias)
+                                      self.keep_groups, self.renormalise_eps, self.router_bias, correction=self.correction,
+                                      two_largest=self.two_largest, weight_scale=self.weight_scale,
+                                      share_row=self.shared_gate, share=share)
         slots = rows * self.top
         if x.dtype == torch.float32 or self.gate_up.dtype == torch.float32 or ctx.plan.is_decode \
                 or slots <= SLOT_PATH_MAX:
-            return routed.expert_slots(x, self.gate_up, self.down, chosen, weight, self.weight_on_input, self.gated, shared)
+            return routed.expert_slots(x, self.gate_up, self.down, chosen, weight, self.weight_on_input, self.gated, shared,
+                                       shape=self.shape, share=share)
         if GROUPED and self.hidden % 8 == 0 and self.inter % 8 == 0 \
                 and 0 < routed.group_rows(slots, self.experts) <= 4 * slots:
             source, place, tiles = routed.group_slots(chosen, self.experts)
             gathered = routed.gather_slots(x, source, weight, self.top, self.weight_on_input)
-            mid = tcgen05.gemm_grouped(gathered, self.gate_up, tiles, self.gated)
+            mid = tcgen05.gemm_grouped(gathered, self.gate_up, tiles, self.gated, shape=self.shape)
             if not self.gated:
                 mid = self._activate(mid)
             result = tcgen05.gemm_grouped(mid, self.down, tiles, False)
-            return routed.combine_slots(result, place, weight, rows, self.top, self.weight_on_input, shared())
+            return routed.combine_slots(result, place, weight, rows, self.top, self.weight_on_input, shared(), share)
         # Many rows: (row, choice) pairs in the order of their experts (a stable sort, so a row's place among
         # its expert's rows follows its place in the step), one host round trip for the counts.
         picked = chosen.reshape(-1).cpu().numpy()
@@ -212,11 +256,11 @@ class RoutedExperts(Part):
             ops.note("library_bmm")
         for index, begin, end in spans:
             self._gate_up[index].forward(gathered[begin:end], out=first[begin:end])
-        mid = self._activate(first)                  # one activation kernel for the rows of all experts
+        mid = self._activate(first, self.shape)      # one activation kernel for the rows of all experts
         if cap:
             torch.bmm(mid[:batch].view(self.experts, cap, self.inter), self.down.transpose(1, 2),
                       out=result[:batch].view(self.experts, cap, self.hidden))
             ops.note("library_bmm")
         for index, begin, end in spans:
             self._down[index].forward(mid[begin:end], out=result[begin:end])
-        return routed.combine_slots(result, tables[total:], weight, rows, self.top, self.weight_on_input, shared())
+        return routed.combine_slots(result, tables[total:], weight, rows, self.top, self.weight_on_input, shared(), share)

@@ -143,7 +143,8 @@ class ParamSpec:
     gate/up -> gate_up rule (src/kidi/model/qwen3.cpp:113-132).
     `init` names the random-weights distribution: ("normal", std), ("one_plus_normal", std),
     ("uniform", high) on [0, high), ("eye_plus_normal", std): the identity plus N(0, std), or ("last_one", std): N(0, std) with 1 added to the last entry. `storage` is "float" (bfloat16, or 32-bit when the
-    file stores 32-bit) or "int32".
+    file stores 32-bit) or "int32". `open_axes`: axes whose extent is the checkpoint's to choose (the file's tensor is
+    taken as it is; `shape` says what random weights get).
     """
 
     name: str
@@ -153,6 +154,7 @@ class ParamSpec:
     storage: str = "float"
     alias_of: Optional[str] = None  # full name of a tensor this one shares storage with when absent
     rules: Tuple[WeightRule, ...] = ()
+    open_axes: Tuple[int, ...] = ()
 
     def alternatives(self) -> Tuple[WeightRule, ...]:
         """The rules that can fill this parameter when its own name is absent."""

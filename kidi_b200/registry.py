@@ -95,3 +95,4 @@ def _load_builtin() -> None:
         from .models import gazezen  # noqa: F401
         from .models import biropel  # noqa: F401
         from .models import dibesun  # noqa: F401
+        from .models import bimolix  # noqa: F401

@@ -210,6 +210,8 @@ def bind_parameters(params: Sequence[Tuple[str, ParamSpec]], source, *, engine_d
             continue
         for name, (_, shape) in zip(names, rule.sources):
             found = tuple(source.shape(name))
+            if spec.open_axes and len(names) == 1 and len(found) == len(shape) and min(found) > 0:
+                shape = tuple(have if axis in spec.open_axes else want for axis, (have, want) in enumerate(zip(found, shape)))
             if found != tuple(shape):
                 wrong.append(f"{name}: shape {list(found)} in the file, {list(shape)} expected")
             if _stored_dtype(source.dtype(name), spec.storage, engine_dtype) is None:
