@@ -2,7 +2,7 @@
 """Decode and prefill throughput of the library on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch B] [--model 8b|14b|32b] [--impl ours|reference]
-    python bench.py --design sanozen|gakenex|gazezen|biropel|dibesun [--widths 2048,4096] [--layers 4]     (another record; see `design_comparison`)
+    python bench.py --design sanozen|gakenex|gazezen|biropel|dibesun|bimolix [--widths 2048,4096] [--layers 4]     (another record; see `design_comparison`)
 
 A step is one decode step of the batch. The default run is the Qwen3-8B shape (every
 layer size, all 36 layers) with random bfloat16 weights drawn on the device from a
@@ -404,8 +404,29 @@ def dibesun_shape(width: int, layers: int = 4) -> dict:
             "norm": {"eps": 1e-5, "groups": 8}, "embedding": {"scale": 2.0}, "layers": stack}
 
 
+def bimolix_shape(width: int, layers: int = 4) -> dict:
+    """A Bimolix stack at the layer sizes of a model of `width`: retention (heads of 128 x 128, whole heads rotated) with a
+    dense SiLU-gated feed-forward of the Qwen3 layers' size in turn with attention whose values are its keys (as many heads
+    of 128, a key/value head for four heads, runs of 4,096 positions, 32 distance buckets up to 1,024) with sixteen routed
+    experts of a quarter of that size in four groups of which two are kept, two experts a token, plus a shared one of half of
+    it (a token uses as many feed-forward weights)."""
+    heads = width // 128
+    inter = (8 * width // 3 + 127) // 128 * 128
+    retention = {"heads": heads, "dim": 128, "vdim": 128, "rot": {"base": 10000.0, "dims": 128},
+                 "decay": [1.0 - 2.0 ** (-2.0 - 8.0 * index / max(1, heads - 1)) for index in range(heads)]}
+    attention = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                 "bias_max": 1024, "mask": {"size": 4096}}
+    routed = {"kind": "moe", "expert": {"ff": inter // 4, "limit": 7.0},
+              "router": {"experts": 16, "top": 2, "groups": {"count": 4, "keep": 2}, "scale": 1.5},
+              "shared": {"ff": inter // 2, "limit": 7.0}}
+    stack = [{"type": "retention", "mixer": retention, "mlp": {"kind": "dense", "ff": inter}} if index % 2 == 0 else
+             {"type": "attention", "mixer": attention, "mlp": routed} for index in range(layers)]
+    return {"architecture": "Bimolix", "vocab": 32768, "width": width, "max_positions": 8192, "norm": {"eps": 1e-5},
+            "layers": stack}
+
+
 DESIGN_SHAPES = {"sanozen": sanozen_shape, "gakenex": gakenex_shape, "gazezen": gazezen_shape, "biropel": biropel_shape,
-                 "dibesun": dibesun_shape}
+                 "dibesun": dibesun_shape, "bimolix": bimolix_shape}
 
 
 def qwen3_shape(width: int, layers: int = 4) -> dict:
@@ -421,7 +442,7 @@ KERNEL_CLASSES = (
     ("products", ("gemm_", "library_mm", "library_bmm", "gemm_heads")),
     ("prompt attention", ("attention_prefill",)),
     ("decode attention", ("attention_decode", "latent_attention")),
-    ("recurrence", ("gated_recurrence", "scalar_recurrence", "linear_attention")),
+    ("recurrence", ("gated_recurrence", "scalar_recurrence", "linear_attention", "retention")),
     ("stream norm", ("add_rmsnorm", "add_layernorm", "lanes_", "add_parts_norm")),
     ("activation", ("silu_gate", "poly_norm", "bounded_gate", "gelu", "relu_squared", "silu_columns")),
     ("experts through the choice", ("expert_slots",)),
@@ -587,6 +608,41 @@ def class_work(design: str, config: dict, rows: int, context: int, decode: bool)
             else:
                 weights += used
                 act_width += 3 * ff * router["top"]
+        work["prompt attention"] = ("flops", attention)
+        work["decode attention"] = ("bytes", cache)
+        work["recurrence"] = ("bytes", scan)
+        if decode:
+            work["experts through the choice"] = ("bytes", chosen)
+    elif design == "bimolix":
+        width, layers = config["width"], config["layers"]
+        weights, norms, act_width, attention, cache, chosen, scan = config["vocab"] * width, 2, 0, 0.0, 0.0, 0.0, 0.0
+        for layer in layers:
+            m, mlp = layer["mixer"], layer["mlp"]
+            heads, dim, vdim = m["heads"], m["dim"], m["vdim"]
+            norms += 2
+            if layer["type"] == "retention":
+                keys, values = heads * dim, heads * vdim
+                weights += width * (2 * keys + 2 * values) + values * width
+                # q, k, v and the gate read, the gated result written; the state read and written
+                scan += rows * (2 * keys + 3 * values) * 2.0 + (rows if decode else 1) * 2.0 * heads * dim * vdim * 4
+            else:
+                groups, chunk = m["kv_heads"], m["mask"]["size"]
+                weights += width * (2 * heads * dim + groups * dim) + heads * dim * width
+                whole, rest = divmod(rows, chunk)
+                attention += 4.0 * heads * dim * (whole * chunk * (chunk + 1) / 2 + rest * (rest + 1) / 2)
+                cache += rows * ((context - 1) % chunk + 1) * groups * dim * 2.0         # a key is its value
+            if mlp["kind"] == "dense":
+                weights += 3 * width * mlp["ff"]
+                act_width += 0 if decode else 3 * mlp["ff"]
+                continue
+            router, ff, shared = mlp["router"], mlp["expert"]["ff"], mlp["shared"]["ff"]
+            weights += (router["experts"] + 1) * width + 3 * width * shared
+            used = 3 * width * ff * router["top"]                                    # per token
+            act_width += 0 if decode else 3 * shared                                 # (the routed gate: in the epilogue)
+            if decode:         # each (row, choice) streams its expert's weights
+                chosen += rows * used * 2.0
+            else:
+                weights += used
         work["prompt attention"] = ("flops", attention)
         work["decode attention"] = ("bytes", cache)
         work["recurrence"] = ("bytes", scan)

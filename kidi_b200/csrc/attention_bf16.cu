@@ -923,17 +923,19 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
             for (int i = 0; i < 2; ++i)
                 if (2 * t + i < group) bias[i] = a.weight_bias[head0 + 2 * t + i] * LOG2E;
         }
+        // What is added to the scores of a tile (asked for a tile ahead).
+        float distance[4] = {0.f, 0.f, 0.f, 0.f};
+        auto ask_distances = [&](int tile) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+                distance[i] = bias_of(a, head0 + min(2 * t + (i & 1), group - 1),
+                                      position - (tile * TILE + warp * 16 + g + (i >> 1) * 8));
+        };
+        if constexpr (BIASED) ask_distances(tile_first);
         for (int index = 0; index < tiles; ++index) {
             const int tile = tile_first + index, buffer = index % STAGES;
             const int k_load = 2 * index, v_load = 2 * index + 1;                 // the ring's loads of this tile
             const bool newest = has_new && tile == new_tile;
-            float distance[4] = {0.f, 0.f, 0.f, 0.f};      // what is added to the scores (asked for before the tile is waited for)
-            if constexpr (BIASED) {
-#pragma unroll
-                for (int i = 0; i < 4; ++i)
-                    distance[i] = bias_of(a, head0 + min(2 * t + (i & 1), group - 1),
-                                          position - (tile * TILE + warp * 16 + g + (i >> 1) * 8));
-            }
             if (RING) {
                 wait_tile(&tile_bar[k_load % 3], (k_load / 3) & 1);
                 if (newest) wait_tile(&tile_bar[v_load % 3], (v_load / 3) & 1);   // the step's value goes into the value tile
@@ -1030,7 +1032,7 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
                     const int holder = (lane & ~3) | (g >> 1);
                     const float square0 = __shfl_sync(0xffffffffu, (g & 1) ? low_square[1] : low_square[0], holder);
                     const float square1 = __shfl_sync(0xffffffffu, (g & 1) ? high_square[3] : high_square[2], holder);
-                    const float factor0 = 1.0f / sqrtf(square0 / (float)D + a.eps), factor1 = 1.0f / sqrtf(square1 / (float)D + a.eps);
+                    const float factor0 = rsqrtf(fmaf(square0, 1.0f / D, a.eps)), factor1 = rsqrtf(fmaf(square1, 1.0f / D, a.eps));
                     s[0] *= factor0; s[1] *= factor0; s[2] *= factor1; s[3] *= factor1;
                 }
 #pragma unroll
@@ -1077,6 +1079,9 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
                 p0 = transpose_8x8(pack_bf16(s[0], s[1]));   // keys 2t, 2t+1 of head g
                 p1 = transpose_8x8(pack_bf16(s[2], s[3]));   // keys 2t+8, 2t+9
             }
+            if constexpr (BIASED) {
+                if (index + 1 < tiles) ask_distances(tile + 1);
+            }
             if (RING) {
                 __syncthreads();                            // the keys are read: their buffer takes the next values
                 if (v_load + 2 < 2 * tiles) issue_load(v_load + 2);
@@ -1104,6 +1109,28 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
         denom[i] += __shfl_xor_sync(0xffffffffu, denom[i], 8);
         denom[i] += __shfl_xor_sync(0xffffffffu, denom[i], 16);
     }
+
+    // What the end of the kernel multiplies the result by is asked for here: the gate of the first four elements that this
+    // thread finishes (from four elements a thread on), and their head's sink.
+    const int share = CLUSTER ? ((group * D + a.splits - 1) / a.splits + 3) & ~3 : 0;
+    const int early = (CLUSTER && a.splits > 1 ? split * share : 0) + threadIdx.x * 4;      // the element's place in the group's heads
+    uint2 early_gate = make_uint2(0u, 0u);
+    if (a.element_gate && early < group * D)
+        early_gate = __ldg(reinterpret_cast<const uint2*>(a.element_gate + row * a.ld_element_gate + (long long)head0 * D + early));
+    // Four finished elements of a head to the output, times their gate (`first`: the ones asked for above).
+    auto store_four = [&](const float4& value, float scale, int head, int c, bool first) {
+        float4 factor = make_float4(scale, scale, scale, scale);
+        if (a.element_gate) {
+            const uint2 raw = first ? early_gate : *reinterpret_cast<const uint2*>(a.element_gate + row * a.ld_element_gate + (long long)head * D + c);
+            const float2 z0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+            const float2 z1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+            factor.x /= 1.0f + expf(-z0.x); factor.y /= 1.0f + expf(-z0.y);
+            factor.z /= 1.0f + expf(-z1.x); factor.w /= 1.0f + expf(-z1.y);
+        }
+        bf16* out = a.out + (long long)row * a.ldo + (long long)head * D + c;
+        *reinterpret_cast<__nv_bfloat162*>(out) = __floats2bfloat162_rn(value.x * factor.x, value.y * factor.y);
+        *reinterpret_cast<__nv_bfloat162*>(out + 2) = __floats2bfloat162_rn(value.z * factor.z, value.w * factor.w);
+    };
 
     // Merge the four warps in warp order through shared memory (the tiles are free now). Rows of
     // the partial results are padded by four floats: the 32 lanes of a store hit 32 banks.
@@ -1170,7 +1197,6 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
     // the splits are merged. A cluster's blocks share the output elements in pieces of `share`
     // elements (a multiple of four), and each sends its partial values to the block that merges
     // them (distributed shared memory, 16 bytes a store).
-    const int share = CLUSTER ? ((group * D + a.splits - 1) / a.splits + 3) & ~3 : 0;
     for (int item = threadIdx.x * 4; item < group * D; item += THREADS * 4) {
         const int r = item / D, c = item - r * D;
         float4 value = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -1183,9 +1209,7 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
         const int head = head0 + r;
         if (a.splits == 1) {
             const float scale = finish_factor(a, row, head, merge_weight[32 + r * 2], merge_weight[32 + r * 2 + 1]);
-            bf16* out = a.out + (long long)row * a.ldo + (long long)head * D + c;
-            *reinterpret_cast<__nv_bfloat162*>(out) = __floats2bfloat162_rn(value.x * scale * gate_of(a, row, head, c), value.y * scale * gate_of(a, row, head, c + 1));
-            *reinterpret_cast<__nv_bfloat162*>(out + 2) = __floats2bfloat162_rn(value.z * scale * gate_of(a, row, head, c + 2), value.w * scale * gate_of(a, row, head, c + 3));
+            store_four(value, scale, head, c, item == threadIdx.x * 4);
         } else if (CLUSTER) {
             const int target = item / share;
             *reinterpret_cast<float4*>(cluster.map_shared_rank(recv_out, target) + split * share + item - target * share) = value;
@@ -1220,10 +1244,7 @@ attention_decode_narrow_kernel(const __grid_constant__ CUtensorMap k_map, const 
                 value.x += part.x * factor; value.y += part.y * factor; value.z += part.z * factor; value.w += part.w * factor;
             }
             const float scale = finish_factor(a, row, head0 + r, top, total);
-            const int head = head0 + r;
-            bf16* out = a.out + (long long)row * a.ldo + (long long)head * D + c;
-            *reinterpret_cast<__nv_bfloat162*>(out) = __floats2bfloat162_rn(value.x * scale * gate_of(a, row, head, c), value.y * scale * gate_of(a, row, head, c + 1));
-            *reinterpret_cast<__nv_bfloat162*>(out + 2) = __floats2bfloat162_rn(value.z * scale * gate_of(a, row, head, c + 2), value.w * scale * gate_of(a, row, head, c + 3));
+            store_four(value, scale, head0 + r, c, i == threadIdx.x * 4);
         }
         return;
     }
@@ -1336,7 +1357,7 @@ int page_map(CUtensorMap* map, const void* base, long long rows) {
 }
 
 bool aligned(const Args& a) {
-    return !((uintptr_t)a.element_gate & 1) && !((uintptr_t)a.q & 15) && !((uintptr_t)a.k_step & 15) && !((uintptr_t)a.v_step & 15) &&
+    return !((uintptr_t)a.element_gate & 7) && !(a.ld_element_gate & 3) && !((uintptr_t)a.q & 15) && !((uintptr_t)a.k_step & 15) && !((uintptr_t)a.v_step & 15) &&
            !((uintptr_t)a.k_cache & 15) && !((uintptr_t)a.v_cache & 15) && !((uintptr_t)a.out & 3) && !(a.ldq & 7) &&
            !(a.ldkv & 7) && !(a.ldo & 1);
 }

@@ -270,8 +270,12 @@ struct Params {
     int chunk;              // > 0: only keys of the query's own run of `chunk` positions are seen
     float out_scale;        // the result is multiplied by it
     SigmoidShape shape;
-    const float* distance_bias;   // biased build only: [heads, bias_stride] in base-2 exponent units, readable from entry -128
-    int bias_stride, bias_last;   // to bias_last + 384 of a row; distances beyond bias_last take that entry
+    // Biased build only: what is added to a score, in base-2 exponent units, by descending distance: entry j of head h is
+    // that of distance bias_origin - j (distances beyond bias_last, and below zero, are filled in). Four copies of a head's
+    // row follow one another, copy c moved c entries to the right, so that any four entries in a row are an aligned 16-byte
+    // piece of one of them: [heads, 4, bias_copy].
+    const float* distance_bias;
+    int bias_copy, bias_origin, bias_last;
     const bf16* element_gate;     // [rows, ld_element_gate] or null: the result is multiplied by sigmoid of it
     long long ld_element_gate;
     int keys_apart;         // the keys are a matrix of their own (k_map); the rows hold query heads, then value heads
@@ -644,7 +648,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map, const 
             const int last_first_seen = first_visible(at.start + q0 + BM - 1, p.window, p.chunk);
             const float scale_log2 = p.scale * LOG2E;
             const float bias_log2 = SIGMOID ? -p.weight_bias[head0 + h] * LOG2E : 0.f;
-            const float* bias_row = BIASED ? p.distance_bias + (long long)(head0 + h) * p.bias_stride : nullptr;
+            const float* bias_row = BIASED ? p.distance_bias + (long long)(head0 + h) * 4 * p.bias_copy : nullptr;
             float reference = -INFINITY;                            // what the exponentials are taken against
             float denom = 0.f;                                      // this thread's part of the row sum
             unsigned exchanges = 0;                                 // uses of row_shared so far
@@ -694,11 +698,18 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map, const 
                 float unit = scale_log2, shift = 0.f;       // a score in base-2 exponent units: s * unit + shift
                 if constexpr (BIASED) {
                     if (at.start + q0 - (key0 + BN - 1) >= p.bias_last) {
-                        shift = __ldg(bias_row + p.bias_last);
+                        shift = __ldg(bias_row + (p.bias_origin - p.bias_last));
                     } else {                                // (distance of the thread's i-th key: last - i)
-                        const float* entry = bias_row + last;
+                        const int first_entry = p.bias_origin - last, copy = -first_entry & 3;
+                        const float4* entry = reinterpret_cast<const float4*>(bias_row + copy * p.bias_copy + first_entry + copy);
 #pragma unroll
-                        for (int i = 0; i < SHARE; ++i) s[i] = fmaf(s[i], scale_log2, __ldg(entry - i));
+                        for (int i = 0; i < SHARE; i += 4) {
+                            const float4 four = __ldg(entry + i / 4);
+                            s[i] = fmaf(s[i], scale_log2, four.x);
+                            s[i + 1] = fmaf(s[i + 1], scale_log2, four.y);
+                            s[i + 2] = fmaf(s[i + 2], scale_log2, four.z);
+                            s[i + 3] = fmaf(s[i + 3], scale_log2, four.w);
+                        }
                         unit = 1.f;
                     }
                 }
@@ -753,6 +764,18 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map, const 
                 asm volatile("fence.proxy.async.shared::cta;" ::: "memory");   // P is read by the tensor core
                 mbarrier_arrive(&ctl.p_ready[h]);
             }
+            // The row's gate is asked for while the last product runs.
+            constexpr int PIECES = D / (32 * GROUPS);       // of 32 columns, this thread's
+            uint4 gate[SIGMOID ? 1 : PIECES][4];
+            const bool gated = !SIGMOID && p.element_gate != nullptr;
+            if (gated && r < q_rows) {
+                const bf16* from = p.element_gate + (long long)(row0 + q0 + r) * p.ld_element_gate + (long long)(head0 + h) * D;
+#pragma unroll
+                for (int piece = 0; piece < (SIGMOID ? 1 : PIECES); ++piece)
+#pragma unroll
+                    for (int i = 0; i < 4; ++i)
+                        gate[piece][i] = __ldg(reinterpret_cast<const uint4*>(from + 32 * (group + GROUPS * piece)) + i);
+            }
             if (ok) ok = mbarrier_wait(&ctl.pv_done[h], (tiles - 1) & 1, abort_flag);
             if (ok) {
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -772,17 +795,16 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map, const 
                     inverse *= 1.0f / (1.0f + expf(-__bfloat162float(p.gate[(long long)(row0 + q0 + r) * p.ldg + head0 + h])));
                 }
                 bf16* out = p.out + (long long)(row0 + q0 + r) * p.ldo + (long long)(head0 + h) * D;
-                const bf16* gate = !SIGMOID && p.element_gate ? p.element_gate + (long long)(row0 + q0 + r) * p.ld_element_gate +
-                                                        (long long)(head0 + h) * D : nullptr;
-#pragma unroll 1
-                for (int c = 32 * group; c < D && ok; c += 32 * GROUPS) {
+#pragma unroll
+                for (int piece = 0; piece < PIECES; ++piece) {
+                    const int c = 32 * (group + GROUPS * piece);
                     float o[32];
                     tmem_load_32(tmem_o + c, o);
                     if (r < q_rows) {
 #pragma unroll
                         for (int i = 0; i < 32; i += 8) {
-                            if (gate) {
-                                const uint4 raw = *reinterpret_cast<const uint4*>(gate + c + i);
+                            if (gated) {
+                                const uint4 raw = gate[SIGMOID ? 0 : piece][i / 8];
                                 const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&raw);
 #pragma unroll
                                 for (int t = 0; t < 4; ++t) {
@@ -876,7 +898,7 @@ struct KidiHeadExtras {      // what a head's result passes beside the plain sof
     int chunk;               // > 0: only keys of the query's own run of `chunk` positions are seen
     float out_scale;         // the result is multiplied by it
     const float* distance_bias;      // biased build only (and there needed): see Params
-    int bias_stride, bias_last;
+    int bias_copy, bias_origin, bias_last;
     const void* element_gate;        // [rows, ld_element_gate] bfloat16, 16-byte pieces: a gate per element of the result
     long long ld_element_gate;
     const void* keys;                // [rows, ld_keys] bfloat16: the step's keys, where qkv holds queries and values only
@@ -973,12 +995,14 @@ KIDI_API int kidi_attention_prefill_tcgen05(const void* qkv, long long ld, int r
         p.chunk = extras->chunk;
         p.out_scale = extras->out_scale;
         p.distance_bias = extras->distance_bias;
-        p.bias_stride = extras->bias_stride;
+        p.bias_copy = extras->bias_copy;
+        p.bias_origin = extras->bias_origin;
         p.bias_last = extras->bias_last;
         p.element_gate = (const bf16*)extras->element_gate;
         p.ld_element_gate = extras->ld_element_gate;
     }
-    if (BIASED != (p.distance_bias != nullptr) || (BIASED && (p.bias_last < 0 || p.bias_stride <= p.bias_last)) ||
+    if (BIASED != (p.distance_bias != nullptr) || (BIASED && (p.bias_last < 0 || p.bias_origin < p.bias_last + 2 * BN || p.bias_copy < p.bias_origin + 2 * BN + 4 ||
+                    (p.bias_copy & 3) || ((uintptr_t)p.distance_bias & 15))) ||
         ((uintptr_t)p.element_gate & 15) || (p.ld_element_gate & 7) || (SIGMOID && p.element_gate))
         return KIDI_REFUSED_SIZE;
     p.shape = sigmoid_shape(p.scale, p.softcap);

@@ -73,12 +73,16 @@ constexpr int DP = D + 8, EP = E + 8;               // row pitches: ldmatrix wit
 #endif
 constexpr bool WIDE = KIDI_LINEAR_WIDE != 0;
 constexpr int SCORE_PITCH = CHUNK + 8;
-// Shared memory of the wide read-out with slices of `slice` rows of the state: q and k in three parts, v, the slices (later
-// the scores in three parts), the decay's powers and the rows' sums of squares.
+// Shared memory of the wide read-out with slices of `slice` rows of the state: two regions, one for q in three parts and
+// later the scores in three parts, one for the slices, then k in three parts, then v; the decay's powers and the rows' sums
+// of squares. (Two blocks of head widths 128 x 128 fit an SM.)
+__host__ __device__ constexpr size_t larger(size_t x, size_t y) { return x > y ? x : y; }
+__host__ __device__ constexpr size_t wide_first_region() { return larger((size_t)3 * CHUNK * DP, (size_t)3 * CHUNK * SCORE_PITCH); }
+__host__ __device__ constexpr size_t wide_second_region(int slice) {
+    return larger(larger((size_t)2 * 3 * slice * EP, (size_t)3 * CHUNK * DP), (size_t)CHUNK * EP);
+}
 __host__ __device__ constexpr size_t wide_read_bytes(int slice) {
-    const size_t slices = (size_t)2 * 3 * slice * EP, scores = (size_t)3 * CHUNK * SCORE_PITCH;
-    return ((size_t)6 * CHUNK * DP + (size_t)CHUNK * EP + (slices > scores ? slices : scores)) * sizeof(bf16) +
-           (size_t)(CHUNK + 4 + 4 * CHUNK) * sizeof(float);
+    return (wide_first_region() + wide_second_region(slice)) * sizeof(bf16) + (size_t)(CHUNK + 4 + 4 * CHUNK) * sizeof(float);
 }
 constexpr size_t MOST_SHARED = 227 * 1024;
 static_assert(!WIDE || wide_read_bytes(16) <= MOST_SHARED, "head widths of the wide build: too large for shared memory");
@@ -152,23 +156,49 @@ struct Chunk {
     }
 };
 
-// The wide build: a chunk's rows of q or k as 32-bit numbers, turned by position and times `scale`, from the bfloat16 tile
-// `raw`; `store(row, column, value)` takes every entry. A thread that takes entry i of a rotated pair takes its partner too.
-template <typename Store>
-__device__ __forceinline__ void widen(const bf16* raw, const LinearChunksArgs& a, int row0, int tokens, float scale, int threads,
-                                      Store store) {
-    const int half = a.cos_table ? a.rotary_dim / 2 : 0, units = D - half;       // pairs, then single entries
-    for (int i = threadIdx.x; i < CHUNK * units; i += threads) {
-        const int r = i / units, c = i - r * units;
-        const bf16* source = raw + r * DP;
-        if (c < half) {
-            const long long at = (long long)a.row_pos[row0 + min(r, tokens - 1)] * half + c;
-            const float cosine = a.cos_table[at], sine = a.sin_table[at];
-            const float u = to_float(source[c]), v = to_float(source[c + half]);
-            store(r, c, scale * (u * cosine - v * sine));
-            store(r, c + half, scale * (v * cosine + u * sine));
-        } else {
-            store(r, c + half, scale * to_float(source[c + half]));
+// The wide build: a chunk's rows of q or k (COUNT tiles at once: they turn by the same angles) as 32-bit numbers, turned by
+// position; `take(tile, row, column, x, y)` gets two neighbouring entries, or, where half the rotary width is odd,
+// `take_one(tile, row, column, x)` every entry. A warp takes a row; a lane that takes entries of rotated pairs has read their
+// partners before it hands any of them on.
+template <int COUNT, typename Take, typename TakeOne>
+__device__ __forceinline__ void widen(const bf16* const (&tiles)[COUNT], const LinearChunksArgs& a, int row0, int tokens,
+                                      int warps, Take take, TakeOne take_one) {
+    const int half = a.cos_table ? a.rotary_dim / 2 : 0, lane = threadIdx.x & 31;
+    for (int r = threadIdx.x >> 5; r < CHUNK; r += warps) {
+        const long long angles = half ? (long long)a.row_pos[row0 + min(r, tokens - 1)] * half : 0;
+        if (half & 1) {
+            for (int c = lane; c < D - half; c += 32) {          // pairs, then single entries
+                const bool pair = c < half;
+                const float cosine = pair ? a.cos_table[angles + c] : 1.f, sine = pair ? a.sin_table[angles + c] : 0.f;
+#pragma unroll
+                for (int tile = 0; tile < COUNT; ++tile) {
+                    const bf16* source = tiles[tile] + r * DP;
+                    const float u = pair ? to_float(source[c]) : 0.f, v = to_float(source[c + half]);
+                    if (pair) take_one(tile, r, c, u * cosine - v * sine);
+                    take_one(tile, r, c + half, pair ? v * cosine + u * sine : v);
+                }
+            }
+            continue;
+        }
+        for (int c = 2 * lane; c < D - half; c += 64) {          // two pairs, then two single entries
+            const bool pair = c < half;
+            float2 cosine = make_float2(1.f, 1.f), sine = make_float2(0.f, 0.f);
+            if (pair) {
+                cosine = *reinterpret_cast<const float2*>(a.cos_table + angles + c);
+                sine = *reinterpret_cast<const float2*>(a.sin_table + angles + c);
+            }
+#pragma unroll
+            for (int tile = 0; tile < COUNT; ++tile) {
+                const bf16* source = tiles[tile] + r * DP + c;
+                const float2 v = unpack(*reinterpret_cast<const unsigned*>(source + half));
+                if (pair) {
+                    const float2 u = unpack(*reinterpret_cast<const unsigned*>(source));
+                    take(tile, r, c, u.x * cosine.x - v.x * sine.x, u.y * cosine.y - v.y * sine.y);
+                    take(tile, r, c + half, v.x * cosine.x + u.x * sine.x, v.y * cosine.y + u.y * sine.y);
+                } else {
+                    take(tile, r, c + half, v.x, v.y);
+                }
+            }
         }
     }
 }
@@ -193,8 +223,12 @@ __global__ void __launch_bounds__(THREADS) chunk_sums_kernel(LinearChunksArgs a)
     copy_async_wait<0>();
     __syncthreads();
     if constexpr (WIDE) {
-        widen(k_tile, a, chunk.row, chunk.tokens, a.key_scale, THREADS,
-              [&](int r, int c, float value) { wide_keys[r * (D + 4) + c] = value; });
+        const bf16* const tiles[1] = {k_tile};
+        widen(tiles, a, chunk.row, chunk.tokens, THREADS / 32,
+              [&](int, int r, int c, float x, float y) {
+                  *reinterpret_cast<float2*>(wide_keys + r * (D + 4) + c) = make_float2(x * a.key_scale, y * a.key_scale);
+              },
+              [&](int, int r, int c, float x) { wide_keys[r * (D + 4) + c] = x * a.key_scale; });
         __syncthreads();
     }
     constexpr int SPAN = 64, SPANS = (E + SPAN - 1) / SPAN;
@@ -426,7 +460,7 @@ __global__ void __launch_bounds__(THREADS) chunk_read_kernel(LinearChunksArgs a)
 // ---------------------------------------------------------------- the read-out of the wide build
 // Sixteen warps: four times 16 tokens by four sides (a side takes every fourth pair of 8-column tiles). q and k are widened
 // and split in shared memory once; the scores of 16 tokens against 16 keys are one warp's (side = key tile), which leaves
-// them, decayed and split, where the slices of the state were.
+// them, decayed and split, where q was.
 constexpr int WIDE_THREADS = 512, SIDES = 4, WIDE_MINE = (PAIRS + SIDES - 1) / SIDES;
 
 // Three parts of x, the largest first.
@@ -439,15 +473,15 @@ __device__ __forceinline__ void split_store(bf16* at, int plane, float x) {
     at[2 * plane] = __float2bfloat16_rn(x - __bfloat162float(second));
 }
 
-__global__ void __launch_bounds__(WIDE_THREADS) chunk_read_wide_kernel(LinearChunksArgs a) {
+__global__ void __launch_bounds__(WIDE_THREADS, 2) chunk_read_wide_kernel(LinearChunksArgs a) {
     extern __shared__ __align__(16) unsigned char raw[];
     constexpr int PLANE = CHUNK * DP, SCORE_PLANE = CHUNK * SCORE_PITCH;
     bf16* q_parts = reinterpret_cast<bf16*>(raw);           // [3][64][DP] (the bfloat16 rows first stand in the first plane)
-    bf16* k_parts = q_parts + 3 * PLANE;                    // [3][64][DP]
-    bf16* v_tile = k_parts + 3 * PLANE;                     // [64][EP]
-    bf16* s_tile = v_tile + CHUNK * EP;                     // [2][3][SLICE][EP], then the scores [3][64][SCORE_PITCH]
-    constexpr int SHARED_TILE = 2 * 3 * SLICE * EP > 3 * SCORE_PLANE ? 2 * 3 * SLICE * EP : 3 * SCORE_PLANE;
-    float* power = reinterpret_cast<float*>(s_tile + SHARED_TILE);      // [65]: a^0 .. a^64
+    bf16* score_parts = q_parts;                            // then [3][64][SCORE_PITCH]
+    bf16* s_tile = q_parts + wide_first_region();           // [2][3][SLICE][EP]
+    bf16* k_parts = s_tile;                                 // then [3][64][DP]
+    bf16* v_tile = s_tile;                                  // then [64][EP]
+    float* power = reinterpret_cast<float*>(s_tile + wide_second_region(SLICE));      // [65]: a^0 .. a^64
     float* squares = power + CHUNK + 4;                     // [SIDES][64]
     const Chunk chunk(a, blockIdx.z, blockIdx.x);
     if (!chunk.live) return;
@@ -472,18 +506,24 @@ __global__ void __launch_bounds__(WIDE_THREADS) chunk_read_wide_kernel(LinearChu
         copy_async_commit();
     };
     load_rows_wide(q_parts, a.q + chunk.row * a.ldq + (long long)head * D, a.ldq, D, DP);
-    load_rows_wide(k_parts, a.k + chunk.row * a.ldk + (long long)head * D, a.ldk, D, DP);
-    load_rows_wide(v_tile, a.v + chunk.row * a.ldv + (long long)head * E, a.ldv, E, EP);
     copy_async_commit();
     load_slice(0);
     for (int i = threadIdx.x; i <= CHUNK; i += WIDE_THREADS) power[i] = powf(a.decay[head], (float)i);
     copy_async_wait<1>();
     __syncthreads();
     // (In place: a thread reads an entry and its partner before it writes either, and nobody else reads them.)
-    widen(q_parts, a, chunk.row, chunk.tokens, 1.f, WIDE_THREADS,
-          [&](int r, int c, float value) { split_store(q_parts + r * DP + c, PLANE, value); });
-    widen(k_parts, a, chunk.row, chunk.tokens, a.key_scale, WIDE_THREADS,
-          [&](int r, int c, float value) { split_store(k_parts + r * DP + c, PLANE, value); });
+    auto widen_in_place = [&](bf16* planes, float scale) {
+        const bf16* const tiles[1] = {planes};
+        widen(tiles, a, chunk.row, chunk.tokens, WIDE_THREADS / 32,
+              [&](int, int r, int c, float x, float y) {
+                  unsigned parts[3];
+                  split_pair(x * scale, y * scale, parts[0], parts[1], parts[2]);
+#pragma unroll
+                  for (int part = 0; part < 3; ++part) *reinterpret_cast<unsigned*>(planes + part * PLANE + r * DP + c) = parts[part];
+              },
+              [&](int, int r, int c, float x) { split_store(planes + r * DP + c, PLANE, x * scale); });
+    };
+    widen_in_place(q_parts, 1.f);
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     const int matrix = lane >> 3, within = lane & 7;
@@ -527,6 +567,8 @@ __global__ void __launch_bounds__(WIDE_THREADS) chunk_read_wide_kernel(LinearChu
         }
         __syncthreads();                                    // the slice is read: its buffer takes the one after next
     }
+    load_rows_wide(k_parts, a.k + chunk.row * a.ldk + (long long)head * D, a.ldk, D, DP);
+    copy_async_commit();
     const float below = power[row + g + 1], above = power[row + g + 9];
 #pragma unroll
     for (int j = 0; j < 2 * WIDE_MINE; ++j) {
@@ -534,9 +576,12 @@ __global__ void __launch_bounds__(WIDE_THREADS) chunk_read_wide_kernel(LinearChu
         o[j][2] *= above; o[j][3] *= above;
     }
     // Scores: this warp's 16 tokens against key tile `side`, where it holds a key at or before the last of them.
-    bf16* score_parts = s_tile;
+    copy_async_wait<0>();
+    __syncthreads();
+    widen_in_place(k_parts, a.key_scale);
+    __syncthreads();
+    float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
     if (side <= (warp & 3)) {
-        float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
 #pragma unroll
         for (int kk = 0; kk < D / 16; ++kk) {
             unsigned q[3][4], k[3][4];
@@ -553,6 +598,11 @@ __global__ void __launch_bounds__(WIDE_THREADS) chunk_read_wide_kernel(LinearChu
                     mma_bf16(s[1], q[part], k[order - part][2], k[order - part][3]);
                 }
         }
+    }
+    __syncthreads();                                        // q and k are read: the scores and v take their places
+    load_rows_wide(v_tile, a.v + chunk.row * a.ldv + (long long)head * E, a.ldv, E, EP);
+    copy_async_commit();
+    if (side <= (warp & 3)) {
 #pragma unroll
         for (int j = 0; j < 2; ++j)
 #pragma unroll
@@ -566,6 +616,7 @@ __global__ void __launch_bounds__(WIDE_THREADS) chunk_read_wide_kernel(LinearChu
                     *reinterpret_cast<unsigned*>(score_parts + part * SCORE_PLANE + r * SCORE_PITCH + key) = parts[part];
             }
     }
+    copy_async_wait<0>();
     __syncthreads();
     for (int kt = 0; kt <= (warp & 3); ++kt) {
         unsigned parts[3][4];

@@ -58,7 +58,7 @@ __device__ __forceinline__ float dot1<bf16, bf16>(const bf16* __restrict__ w, co
 // A block a row: its sixteen warps share the experts (a warp a router row at a time, 32-bit sums in an order
 // that depends on the width only), then the first warp takes the `top` largest scores, one after the other.
 template <typename T, typename TW>
-__global__ void __launch_bounds__(512) route_kernel(const T* __restrict__ x, const TW* __restrict__ router,
+__global__ void __launch_bounds__(544) route_kernel(const T* __restrict__ x, const TW* __restrict__ router,
                                                     int* __restrict__ chosen, float* __restrict__ weight, int hidden,
                                                     int experts, int top, int renormalise, int softmax, int groups,
                                                     int keep, float renormalise_eps, const float* __restrict__ bias,
@@ -68,11 +68,11 @@ __global__ void __launch_bounds__(512) route_kernel(const T* __restrict__ x, con
     float* open = score + experts;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long row = blockIdx.x;
-    if (share && warp == 15) {             // the gate of the expert that every row passes
+    if (warp == 16) {                      // (launched where it is asked for) the gate of the expert that every row passes
         const float z = warp_sum(dot1<T, TW>(share_row, x + row * hidden, hidden, lane));
         if (lane == 0) share[row] = 1.0f / (1.0f + expf(-z));
     }
-    for (int e = warp; e < experts; e += 16) {
+    for (int e = warp; warp < 16 && e < experts; e += 16) {
         float z = warp_sum(dot1<T, TW>(router + (long long)e * hidden, x + row * hidden, hidden, lane));
         if (bias) z += bias[e];
         if (lane == 0) score[e] = softmax ? z : 1.0f / (1.0f + expf(-z));
@@ -176,7 +176,7 @@ KIDI_API int kidi_route(const void* x, int dtype, const void* router, int weight
     const size_t shared = (size_t)experts * 2 * sizeof(float);
 #define KIDI_CASE(D, T, W, TW)                                                                                        \
     if (dtype == D && weight_dtype == W)                                                                              \
-        return kidi_launch(route_kernel<T, TW>, (unsigned)rows, 512, shared, stream, (const T*)x, (const TW*)router,  \
+        return kidi_launch(route_kernel<T, TW>, (unsigned)rows, share ? 544 : 512, shared, stream, (const T*)x, (const TW*)router,  \
                            chosen, weight, hidden, experts, top, renormalise, softmax, groups, keep, renormalise_eps, \
                            bias, correction, two_largest, weight_scale, (const TW*)share_row, share);
     KIDI_CASE(KIDI_F32, float, KIDI_F32, float)

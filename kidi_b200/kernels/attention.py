@@ -126,8 +126,8 @@ class HeadExtras(ctypes.Structure):
     distance, a sigmoid gate per element, keys that lie apart from the values."""
     _fields_ = [("sinks", c_void_p), ("gate", c_void_p), ("ldg", c_longlong), ("softcap", c_float),
                 ("weight_bias", c_void_p), ("chunk", c_int), ("out_scale", c_float), ("distance_bias", c_void_p),
-                ("bias_stride", c_int), ("bias_last", c_int), ("element_gate", c_void_p), ("ld_element_gate", c_longlong),
-                ("keys", c_void_p), ("ld_keys", c_longlong)]
+                ("bias_copy", c_int), ("bias_origin", c_int), ("bias_last", c_int), ("element_gate", c_void_p),
+                ("ld_element_gate", c_longlong), ("keys", c_void_p), ("ld_keys", c_longlong)]
 
 
 def extras_fit(sinks: Optional[torch.Tensor], gate: Optional[torch.Tensor], heads: int) -> bool:
@@ -163,7 +163,7 @@ def prefill_tensor_memory(qkv: torch.Tensor, out: torch.Tensor, seq_len: torch.T
         extras = HeadExtras(sinks.data_ptr() if sinks is not None else 0, gate.data_ptr() if gate is not None else 0,
                             gate.stride(0) if gate is not None else 0, float(softcap or 0.0),
                             weight_bias.data_ptr() if weight_bias is not None else 0, int(chunk or 0), float(out_scale),
-                            *(distance_bias.fields(heads, log2=True) if distance_bias is not None else (0, 0, 0)),
+                            *(distance_bias.descending(heads) if distance_bias is not None else (0, 0, 0, 0)),
                             element_gate.data_ptr() if element_gate is not None else 0,
                             element_gate.stride(0) if element_gate is not None else 0,
                             k_normed.data_ptr() if k_normed is not None else 0,

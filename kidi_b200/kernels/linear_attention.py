@@ -75,9 +75,10 @@ def chunks_fit(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, dim: int, vdim
 
 
 def wide_chunks_fit(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, dim: int, vdim: int, longest: int) -> bool:
-    """The same for the form with 32-bit queries and keys, whose three parts of each must fit shared memory."""
-    rows = 6 * CHUNK * (dim + 8) + CHUNK * (vdim + 8) + max(2 * 3 * 16 * (vdim + 8), 3 * CHUNK * (CHUNK + 8))
-    return chunks_fit(q, k, v, dim, vdim, longest) and 2 * rows + 4 * (CHUNK + 4 + 4 * CHUNK) <= 227 * 1024
+    """The same for the form with 32-bit queries and keys, of which a block keeps three parts in shared memory."""
+    parts = 3 * CHUNK * (dim + 8)
+    first, second = max(parts, 3 * CHUNK * (CHUNK + 8)), max(2 * 3 * 16 * (vdim + 8), parts, CHUNK * (vdim + 8))
+    return chunks_fit(q, k, v, dim, vdim, longest) and 2 * (first + second) + 4 * (CHUNK + 4 + 4 * CHUNK) <= 227 * 1024
 
 
 def library():
