@@ -163,13 +163,15 @@ def routed(h: torch.Tensor, w: Mapping[str, torch.Tensor], prefix: str, mlp: Map
     groups = router.get("groups") or {"count": 1, "keep": 1}
     scores = torch.sigmoid(lin(w[prefix + "router"], h))
     choice = scores + w[prefix + "correction"].to(h.dtype)
-    out = torch.zeros_like(h)
+    share = torch.zeros(h.shape[0], int(router["experts"]), dtype=h.dtype)          # of every expert in every token
     for t in range(h.shape[0]):
         chosen = chosen_or_given(choice[t], int(router["top"]), int(groups["count"]), int(groups["keep"]),
                                  given[t] if given is not None else None, margin)
-        weights = scores[t, chosen] / (scores[t, chosen].sum() + 1e-20) * float(router["scale"])
-        for weight, index in zip(weights, chosen.tolist()):
-            out[t] += weight * bounded_expert(h[t:t + 1], w, f"{prefix}e{index}.", float(mlp["expert"]["limit"]))[0]
+        share[t, chosen] = scores[t, chosen] / (scores[t, chosen].sum() + 1e-20) * float(router.get("scale", 1.0))
+    out = torch.zeros_like(h)
+    for index in range(share.shape[1]):
+        users = (share[:, index] != 0).nonzero().flatten()
+        out[users] += share[users, index, None] * bounded_expert(h[users], w, f"{prefix}e{index}.", float(mlp["expert"]["limit"]))
     shared = mlp.get("shared")
     if shared:
         out = out + torch.sigmoid(lin(w[prefix + "shared.sg"], h)) \
