@@ -229,7 +229,8 @@ class Attention(Part):
         if self.bias_reach is not None:
             by_bucket = tensors[self.names["distance_bias"]]
             reach, seen = int(self.bias_reach), reach_of(self.window, self.chunk) or self.env.max_positions
-            buckets = distance_buckets(min(seen, reach + 1), by_bucket.shape[0], reach)
+            last = max(reach, by_bucket.shape[0] // 2)          # from here on it is the last bucket's
+            buckets = distance_buckets(min(seen, last + 1), by_bucket.shape[0], reach)
             self.distance_bias = ops.DistanceBias(by_bucket.float()[buckets.to(by_bucket.device)])
         if self.has_sink:
             self.sinks = tensors[self.names["sink"]].float().contiguous()

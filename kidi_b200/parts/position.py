@@ -48,13 +48,14 @@ from .spec import ParamSpec
 def distance_buckets(count: int, buckets: int, reach: int) -> torch.Tensor:
     """int64 [count]: the bucket of distances 0 .. count - 1. With B buckets and h = B // 2 a distance n < h has bucket n, any
     other min(B - 1, h + floor(ln(n / h) / ln(reach / h) (B - h))). The logarithms are 64-bit; where n is an exact power the
-    quotient is the whole number it stands for, whatever the logarithms round to."""
+    quotient is the whole number it stands for, whatever the logarithms round to. (With a reach that the first half covers
+    already, everything beyond that half has the last bucket.)"""
     half = buckets // 2
-    if buckets < 1 or not reach > half:
-        raise invalid_argument(f"{buckets} distance buckets must reach further than {half} positions, not {reach}")
-    if half == 0:
-        return torch.zeros(count, dtype=torch.int64)
+    if buckets < 1 or reach < 1:
+        raise invalid_argument("a distance bias has at least one bucket and a positive reach")
     distance = torch.arange(count, dtype=torch.float64)
+    if half == 0 or reach <= half:
+        return torch.where(distance < half, distance, float(buckets - 1)).long()
     place = torch.log(distance.clamp(min=half) / half) / math.log(reach / half) * (buckets - half)
     whole = torch.round(place)
     place = torch.where((place - whole).abs() < 1e-9, whole, torch.floor(place))

@@ -86,6 +86,8 @@ def distance_bucket(n: int, rows: int, reach: int) -> int:
     half = rows // 2
     if n < half:
         return n
+    if reach <= half:
+        return rows - 1
     place = math.log(n / half) / math.log(reach / half) * (rows - half)
     if abs(place - round(place)) < 1e-9:            # an exact power, whatever the logarithms rounded to
         place = round(place)

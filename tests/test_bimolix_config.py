@@ -127,7 +127,6 @@ def test_what_the_cache_is_asked_for():
 def test_distance_buckets(buckets, reach):
     """Against the definition in exact arithmetic: floor(ln(n / h) / ln(r / h) (B - h)) >= m as (n / h)^(B - h) >= (r / h)^m
     in whole numbers, so that exact powers fall where they belong."""
-    from kidi_b200.errors import KidiError
     from kidi_b200.parts.position import distance_buckets
     half, count = buckets // 2, min(2 * reach + 3, 2000)
     got = distance_buckets(count, buckets, reach).tolist()
@@ -144,8 +143,8 @@ def test_distance_buckets(buckets, reach):
     assert got == [exact(n) for n in range(count)]
     if half:
         assert got == [plain.distance_bucket(n, buckets, reach) for n in range(count)]
-        with pytest.raises(KidiError):
-            distance_buckets(10, buckets, half)
+        # a reach within the first half: what lies beyond that half has the last bucket
+        assert distance_buckets(half + 5, buckets, half).tolist() == list(range(half)) + [buckets - 1] * 5
 
 
 def test_a_random_model_folder_through_the_command_line(tmp_path, capsys):
