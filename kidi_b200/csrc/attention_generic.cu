@@ -53,11 +53,12 @@ template <typename T, typename TW>
 __global__ void __launch_bounds__(128) rope_store_kernel(RopeStoreArgs a) {
     __shared__ float normed[4][256];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int total_heads = a.heads + (a.tied ? 1 : 2) * a.kv_heads;
+    const int first_head = a.transform ? 0 : a.heads;         // copying alone: the k (and v) heads only
+    const int total_heads = a.heads - first_head + (a.tied ? 1 : 2) * a.kv_heads;
     const long long item = (long long)blockIdx.x * 4 + warp;
     if (item >= (long long)a.rows * total_heads) return;
     const int row = (int)(item / total_heads);
-    const int head = (int)(item - (long long)row * total_heads);
+    const int head = first_head + (int)(item - (long long)row * total_heads);
     const int seq = a.row_seq[row];
     if (seq < 0) return;
     const int position = a.row_pos[row];
@@ -163,7 +164,8 @@ __device__ __forceinline__ void load8(const bf16* p, float (&w)[8]) {
 template <typename TW>
 __global__ void __launch_bounds__(128) rope_store_bf16_kernel(RopeStoreArgs a, int group_lanes) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int total_heads = a.heads + (a.tied ? 1 : 2) * a.kv_heads;
+    const int first_head = a.transform ? 0 : a.heads;         // copying alone: the k (and v) heads only
+    const int total_heads = a.heads - first_head + (a.tied ? 1 : 2) * a.kv_heads;
     const int per_warp = 32 / group_lanes;
     const int group = lane / group_lanes, l = lane - group * group_lanes;
     const int item = (blockIdx.x * 4 + warp) * per_warp + group;   // the launcher keeps the count below 2^31
@@ -171,7 +173,7 @@ __global__ void __launch_bounds__(128) rope_store_bf16_kernel(RopeStoreArgs a, i
     // group has a (row, head) to work on.
     bool alive = item < a.rows * total_heads;
     const int row = alive ? item / total_heads : 0;
-    const int head = alive ? item - row * total_heads : 0;
+    const int head = alive ? first_head + item - row * total_heads : first_head;
     const int d = a.head_dim, c0 = 8 * l;
     bf16* vector = (bf16*)a.qkv + (long long)row * a.ld + head * d;
     // The row's elements are asked for together with its sequence and position (a padding
@@ -272,7 +274,8 @@ KIDI_API int kidi_rope_store(const RopeStoreArgs* args, int dtype, int norm_dtyp
         return KIDI_REFUSED_SIZE;
     if (a.tied && (a.cos_table || a.v_cache || !a.q_norm || (a.value_dim && a.value_dim != a.head_dim)) && a.transform)
         return KIDI_REFUSED_SIZE;
-    const long long items = (long long)a.rows * (a.heads + (a.tied ? 1 : 2) * a.kv_heads);
+    const long long items = (long long)a.rows * ((a.transform ? a.heads : 0) + (a.tied ? 1 : 2) * a.kv_heads);
+    if (items <= 0) return 0;
     const unsigned blocks = (unsigned)((items + 3) / 4);
     const bool vectors = dtype == KIDI_BF16 && items < (1LL << 30) && (!a.value_dim || a.value_dim == a.head_dim) && !((uintptr_t)a.q_norm & 15) &&
                          !((uintptr_t)a.k_norm & 15) && !(a.head_dim & 7) && !(a.ld & 7) && !((uintptr_t)a.qkv & 15) &&

@@ -297,8 +297,9 @@ class Attention(Part):
             extras["weight_bias"] = self.weight_bias
         # A ring that is written before attention would lose keys that the step's
         # earlier rows still need; it is written afterwards unless the step is one
-        # token per sequence. A full-history cache is written first.
-        store_first = owns_cache and (not ring or plan.is_decode)
+        # token per sequence or starts every sequence (then the ring holds nothing yet and every
+        # key is a row of the step). A full-history cache is written first.
+        store_first = owns_cache and (not ring or plan.is_decode or int(plan.seq_start.max()) == 0)
         if not owns_cache and ring and not plan.is_decode:
             raise unsupported("a layer that reads another layer's windowed cache takes one token per step")
         # One token per sequence on the tensor-core path: the attention kernel takes the rows as
