@@ -134,6 +134,17 @@ __device__ __forceinline__ void tmem_load_16(unsigned address, float (&v)[16]) {
     for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(r[i]);
 }
 
+// gate_value with the fast exponential and division (a few units in the last place; the results are rounded to bfloat16;
+// far below zero the exponential is held at 2^115, so that the quotient stays a number).
+__device__ __forceinline__ float gate_value_near(const GateShape& shape, float g, float u) {
+    const float slope = shape.bounded ? shape.alpha : 1.f;
+    if (shape.bounded) {
+        g = fminf(g, shape.limit);
+        u = fminf(fmaxf(u, -shape.limit), shape.limit) + shape.shift;
+    }
+    return __fdividef(g, 1.0f + __expf(fminf(-slope * g, 80.f))) * u;
+}
+
 // 16 or 32 columns at once: every load is issued before the wait.
 template <int N>
 __device__ __forceinline__ void tmem_load(unsigned address, float (&v)[N]) {
@@ -407,17 +418,24 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                     else
 #pragma unroll
                         for (int i = 0; i < CW; ++i) v[i] = 0.f;
-                    bool mine = f0 + row < p.features;    // this thread has results of this chunk
+                    // The thread's feature within the tile and its columns of the chunk (gated: half of them).
+                    const int feature = GATED ? row & 63 : row;
+                    const int first = GATED && row >= 64 ? CW / 2 : 0;
+                    constexpr int COUNT = GATED ? CW / 2 : CW;
+                    const bool mine = f0 + feature < p.features;
                     if (GATED) {
-                        // Rows 64..127 hold the up projection of the features in rows 0..63.
-                        if (row >= 64)
+                        // Rows 64..127 hold the up projection of the features in rows 0..63. The two threads of a feature
+                        // share its columns: one takes the first half and gets their up values, the other takes the second
+                        // half and gets their gates.
+                        float* shared_row = exchange + feature * (CW + 1);
 #pragma unroll
-                            for (int i = 0; i < CW; ++i) exchange[(row - 64) * (CW + 1) + i] = v[i];
+                        for (int i = 0; i < CW / 2; ++i) shared_row[(CW / 2 - first) + i] = row < 64 ? v[CW / 2 + i] : v[i];
                         asm volatile("bar.sync 1, 128;" ::: "memory");
-                        mine = mine && row < 64;
-                        if (row < 64)
 #pragma unroll
-                            for (int i = 0; i < CW; ++i) v[i] = gate_value(p.gate, v[i], exchange[row * (CW + 1) + i]);
+                        for (int i = 0; i < CW / 2; ++i) {
+                            const float other = shared_row[first + i];
+                            v[i] = row < 64 ? gate_value_near(p.gate, v[i], other) : gate_value_near(p.gate, other, v[CW / 2 + i]);
+                        }
                         asm volatile("bar.sync 1, 128;" ::: "memory");
                     } else if (p.bias && mine) {
                         const float shift = p.bias[f0 + row];
@@ -429,9 +447,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                         // The copy that read this buffer two chunks ago must be through with it.
                         if (threadIdx.x == 64 && staged_chunks >= 2) asm volatile("cp.async.bulk.wait_group.read 1;" ::: "memory");
                         asm volatile("bar.sync 1, 128;" ::: "memory");
-                        if (row < SPAN)
 #pragma unroll
-                            for (int i = 0; i < CW; ++i) out[i * SPAN + row] = __float2bfloat16_rn(v[i]);
+                        for (int i = 0; i < COUNT; ++i) out[(first + i) * SPAN + feature] = __float2bfloat16_rn(v[i]);
                         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");   // the copy reads what these threads wrote
                         asm volatile("bar.sync 1, 128;" ::: "memory");
                         if (threadIdx.x == 64) {
@@ -442,9 +459,9 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                         ++staged_chunks;
                     } else if (mine) {
 #pragma unroll
-                        for (int i = 0; i < CW; ++i) {
-                            const int token = t0 + c + i;
-                            if (token < p.tokens) y[token * p.ldy + f0 + row] = from_float<TY>(v[i]);
+                        for (int i = 0; i < COUNT; ++i) {
+                            const int token = t0 + c + first + i;
+                            if (token < p.tokens) y[token * p.ldy + f0 + feature] = from_float<TY>(v[i]);
                         }
                     }
                 }
@@ -513,7 +530,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                         for (int j = 0; j < 16; ++j)
                             if (j0 + j < count)
                                 y[(long long)(t0 + first + j0 + j) * p.ldy + f0 + row] =
-                                    from_float<TY>(gate_value(p.gate, sum[j], exchange[row * 17 + j]));
+                                    from_float<TY>(gate_value_near(p.gate, sum[j], exchange[row * 17 + j]));
                     asm volatile("bar.sync 1, 128;" ::: "memory");
                 } else if (f0 + row < p.features) {
 #pragma unroll
