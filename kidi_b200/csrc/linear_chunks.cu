@@ -160,12 +160,15 @@ struct Chunk {
 // position; `take(tile, row, column, x, y)` gets two neighbouring entries, or, where half the rotary width is odd,
 // `take_one(tile, row, column, x)` every entry. A warp takes a row; a lane that takes entries of rotated pairs has read their
 // partners before it hands any of them on.
-template <int COUNT, typename Take, typename TakeOne>
+template <int WARPS, int COUNT, typename Take, typename TakeOne>
 __device__ __forceinline__ void widen(const bf16* const (&tiles)[COUNT], const LinearChunksArgs& a, int row0, int tokens,
-                                      int warps, Take take, TakeOne take_one) {
-    const int half = a.cos_table ? a.rotary_dim / 2 : 0, lane = threadIdx.x & 31;
-    for (int r = threadIdx.x >> 5; r < CHUNK; r += warps) {
-        const long long angles = half ? (long long)a.row_pos[row0 + min(r, tokens - 1)] * half : 0;
+                                      Take take, TakeOne take_one) {
+    const int half = a.cos_table ? a.rotary_dim / 2 : 0, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int position0 = half ? a.row_pos[row0] : 0;            // a sequence's rows of a step follow one another
+#pragma unroll 4
+    for (int i = 0; i < CHUNK / WARPS; ++i) {
+        const int r = warp + i * WARPS;
+        const long long angles = (long long)(position0 + min(r, tokens - 1)) * half;
         if (half & 1) {
             for (int c = lane; c < D - half; c += 32) {          // pairs, then single entries
                 const bool pair = c < half;
@@ -224,7 +227,7 @@ __global__ void __launch_bounds__(THREADS) chunk_sums_kernel(LinearChunksArgs a)
     __syncthreads();
     if constexpr (WIDE) {
         const bf16* const tiles[1] = {k_tile};
-        widen(tiles, a, chunk.row, chunk.tokens, THREADS / 32,
+        widen<THREADS / 32>(tiles, a, chunk.row, chunk.tokens,
               [&](int, int r, int c, float x, float y) {
                   *reinterpret_cast<float2*>(wide_keys + r * (D + 4) + c) = make_float2(x * a.key_scale, y * a.key_scale);
               },
@@ -514,7 +517,7 @@ __global__ void __launch_bounds__(WIDE_THREADS, 2) chunk_read_wide_kernel(Linear
     // (In place: a thread reads an entry and its partner before it writes either, and nobody else reads them.)
     auto widen_in_place = [&](bf16* planes, float scale) {
         const bf16* const tiles[1] = {planes};
-        widen(tiles, a, chunk.row, chunk.tokens, WIDE_THREADS / 32,
+        widen<WIDE_THREADS / 32>(tiles, a, chunk.row, chunk.tokens,
               [&](int, int r, int c, float x, float y) {
                   unsigned parts[3];
                   split_pair(x * scale, y * scale, parts[0], parts[1], parts[2]);

@@ -27,58 +27,77 @@
 #include "common.cuh"
 
 // ---------------------------------------------------------------- choose
-// One row of weights against one row of x, a warp's share; the caller sums over the warp.
-template <typename T, typename TW>
-__device__ __forceinline__ float dot1(const TW* __restrict__ w, const T* __restrict__ x, int K, int lane) {
-    float a = 0.f;
-    for (int k = lane; k < K; k += 32) a = fmaf(to_float(w[k]), to_float(x[k]), a);
-    return a;
-}
-template <>
-__device__ __forceinline__ float dot1<bf16, bf16>(const bf16* __restrict__ w, const bf16* __restrict__ x, int K, int lane) {
-    float a = 0.f;
-    if ((K & 7) || ((uintptr_t)w & 15) || ((uintptr_t)x & 15)) {
-        for (int k = lane; k < K; k += 32) a = fmaf(to_float(w[k]), to_float(x[k]), a);
-        return a;
-    }
-    for (int k = lane * 8; k < K; k += 256) {
-        const uint4 rw = *reinterpret_cast<const uint4*>(w + k), rx = *reinterpret_cast<const uint4*>(x + k);
-        const __nv_bfloat162* pw = reinterpret_cast<const __nv_bfloat162*>(&rw);
-        const __nv_bfloat162* px = reinterpret_cast<const __nv_bfloat162*>(&rx);
+// One row of weights against ROWS rows of x (the first `here` of them; `hidden` apart), a warp's share; the caller sums over
+// the warp. A row's sum runs in the same order whatever ROWS is.
+template <int ROWS, typename T, typename TW>
+__device__ __forceinline__ void dots(const TW* __restrict__ w, const T* __restrict__ x, int K, int lane, int here, float (&a)[ROWS]) {
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const float2 fw = __bfloat1622float2(pw[i]), fx = __bfloat1622float2(px[i]);
-            a = fmaf(fw.x, fx.x, a);
-            a = fmaf(fw.y, fx.y, a);
+    for (int r = 0; r < ROWS; ++r) a[r] = 0.f;
+    if constexpr (sizeof(T) == 2 && sizeof(TW) == 2) {
+        if (!(K & 7) && !((uintptr_t)w & 15) && !((uintptr_t)x & 15)) {
+            for (int k = lane * 8; k < K; k += 256) {
+                const uint4 rw = *reinterpret_cast<const uint4*>(w + k);
+                const __nv_bfloat162* pw = reinterpret_cast<const __nv_bfloat162*>(&rw);
+                float2 fw[4];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) fw[i] = __bfloat1622float2(pw[i]);
+#pragma unroll
+                for (int r = 0; r < ROWS; ++r) {
+                    const uint4 rx = *reinterpret_cast<const uint4*>(x + (long long)min(r, here - 1) * K + k);
+                    const __nv_bfloat162* px = reinterpret_cast<const __nv_bfloat162*>(&rx);
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        const float2 fx = __bfloat1622float2(px[i]);
+                        a[r] = fmaf(fw[i].x, fx.x, a[r]);
+                        a[r] = fmaf(fw[i].y, fx.y, a[r]);
+                    }
+                }
+            }
+            return;
         }
     }
-    return a;
+    for (int k = lane; k < K; k += 32) {
+        const float value = to_float(w[k]);
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) a[r] = fmaf(value, to_float(x[(long long)min(r, here - 1) * K + k]), a[r]);
+    }
 }
 
-// A block a row: its sixteen warps share the experts (a warp a router row at a time, 32-bit sums in an order
-// that depends on the width only), then the first warp takes the `top` largest scores, one after the other.
-template <typename T, typename TW>
+// A block ROWS rows: its sixteen warps share the experts (a warp a router row at a time, 32-bit sums in an order
+// that depends on the width only), then a warp a row takes the `top` largest scores, one after the other.
+template <int ROWS, typename T, typename TW>
 __global__ void __launch_bounds__(544) route_kernel(const T* __restrict__ x, const TW* __restrict__ router,
                                                     int* __restrict__ chosen, float* __restrict__ weight, int hidden,
                                                     int experts, int top, int renormalise, int softmax, int groups,
                                                     int keep, float renormalise_eps, const float* __restrict__ bias,
                                                     const float* __restrict__ correction, int two_largest, float weight_scale,
-                                                    const TW* __restrict__ share_row, float* __restrict__ share) {
-    extern __shared__ float score[];       // [experts] scores, then [experts] what may still be chosen
-    float* open = score + experts;
+                                                    const TW* __restrict__ share_row, float* __restrict__ share, int rows) {
+    extern __shared__ float scores[];      // for each row: [experts] scores, then [experts] what may still be chosen
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const long long row = blockIdx.x;
+    const int row0 = blockIdx.x * ROWS, here = min(ROWS, rows - row0);
+    const T* block_rows = x + (long long)row0 * hidden;
+    float dot[ROWS];
     if (warp == 16) {                      // (launched where it is asked for) the gate of the expert that every row passes
-        const float z = warp_sum(dot1<T, TW>(share_row, x + row * hidden, hidden, lane));
-        if (lane == 0) share[row] = 1.0f / (1.0f + expf(-z));
+        dots<ROWS, T, TW>(share_row, block_rows, hidden, lane, here, dot);
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) {
+            const float z = warp_sum(dot[r]);
+            if (lane == 0 && r < here) share[row0 + r] = 1.0f / (1.0f + expf(-z));
+        }
     }
     for (int e = warp; warp < 16 && e < experts; e += 16) {
-        float z = warp_sum(dot1<T, TW>(router + (long long)e * hidden, x + row * hidden, hidden, lane));
-        if (bias) z += bias[e];
-        if (lane == 0) score[e] = softmax ? z : 1.0f / (1.0f + expf(-z));
+        dots<ROWS, T, TW>(router + (long long)e * hidden, block_rows, hidden, lane, here, dot);
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) {
+            float z = warp_sum(dot[r]);
+            if (bias) z += bias[e];
+            if (lane == 0) scores[2 * experts * r + e] = softmax ? z : 1.0f / (1.0f + expf(-z));
+        }
     }
     __syncthreads();
-    if (warp) return;
+    if (warp >= here) return;
+    const long long row = row0 + warp;
+    float *score = scores + 2 * experts * warp, *open = score + experts;
     if (softmax) {                         // over all experts, the sum in lane order and then across the lanes
         float most = -INFINITY;
         for (int e = lane; e < experts; e += 32) most = fmaxf(most, score[e]);
@@ -174,11 +193,15 @@ KIDI_API int kidi_route(const void* x, int dtype, const void* router, int weight
         (long long)keep * (experts / groups) < top)
         return KIDI_REFUSED_SIZE;
     const size_t shared = (size_t)experts * 2 * sizeof(float);
+    constexpr int ROWS = 4;                  // rows of a block where there are enough of them (experts <= 1,024: 32 KB)
+    const bool many = rows >= 512;
 #define KIDI_CASE(D, T, W, TW)                                                                                        \
     if (dtype == D && weight_dtype == W)                                                                              \
-        return kidi_launch(route_kernel<T, TW>, (unsigned)rows, share ? 544 : 512, shared, stream, (const T*)x, (const TW*)router,  \
-                           chosen, weight, hidden, experts, top, renormalise, softmax, groups, keep, renormalise_eps, \
-                           bias, correction, two_largest, weight_scale, (const TW*)share_row, share);
+        return kidi_launch(many ? route_kernel<ROWS, T, TW> : route_kernel<1, T, TW>,                                 \
+                           (unsigned)(many ? (rows + ROWS - 1) / ROWS : rows), share ? 544 : 512,                     \
+                           many ? ROWS * shared : shared, stream, (const T*)x, (const TW*)router, chosen, weight,     \
+                           hidden, experts, top, renormalise, softmax, groups, keep, renormalise_eps, bias,           \
+                           correction, two_largest, weight_scale, (const TW*)share_row, share, rows);
     KIDI_CASE(KIDI_F32, float, KIDI_F32, float)
     KIDI_CASE(KIDI_F32, float, KIDI_BF16, bf16)
     KIDI_CASE(KIDI_BF16, bf16, KIDI_BF16, bf16)

@@ -523,6 +523,19 @@ def test_the_router_with_a_correction_and_ranked_groups(dtype):
             assert torch.equal(chosen[r].cpu().long(), want)
             assert torch.allclose(weight[r].double().cpu(), s[r, want] / s[r, want].sum() * 1.7, atol=1e-5)
         assert torch.allclose(share.double().cpu(), torch.sigmoid(x.double() @ row[0].double()), atol=1e-5)
+    # many rows (four a block, the last block short of one): what a few rows give, bit for bit
+    x, router = torch.randn(1027, 72, generator=generator).to(dtype).cuda(), (torch.randn(12, 72, generator=generator) * 0.3).to(dtype).cuda()
+    correction, row = (torch.randn(12, generator=generator) * 0.4).cuda(), (torch.randn(1, 72, generator=generator) * 0.3).to(dtype).cuda()
+
+    def route(some):
+        share = torch.empty(some.shape[0]).cuda()
+        chosen, weight = routed.route(some.contiguous(), router, 3, True, "sigmoid", 4, 2, 1e-20, correction=correction,
+                                      two_largest=True, weight_scale=0.7, share_row=row, share=share)
+        return chosen.float(), weight, share
+
+    whole, pieces = route(x), [route(piece) for piece in x.split(100)]
+    for index in range(3):
+        assert torch.equal(whole[index], torch.cat([piece[index] for piece in pieces]))
 
 
 @pytest.mark.parametrize("rows,experts,top,hidden,inter", [(3, 5, 2, 64, 24), (200, 6, 2, 64, 24), (300, 5, 5, 136, 72), (40, 4, 3, 50, 22)])
