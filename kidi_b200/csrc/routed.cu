@@ -14,7 +14,7 @@
 // A (row, choice) pair is a "slot": slot = row * top + choice.
 //
 // Kernels:
-//  * choose: the router's product, the scores, the top choices and their weights, a block a row;
+//  * choose: the router's product, the scores, the top choices and their weights, a block a row (four rows on prompts);
 //  * slots, gate and up: for few rows, and for every row count of the 32-bit engine: a warp per
 //    (slot, feature) reads the chosen expert's two weight rows once and applies the activation; the
 //    input weight is applied to the two products in 32-bit (W (w h) = w (W h));
